@@ -102,13 +102,13 @@ class Group:
 class PagedCache:
     """See the module text. `requests[i]` is the KvRequest of schedule entry i
     (None if that run keeps no keys of its own); `states[i]` its StateRequest or
-    None. `max_tokens` bounds the tokens held by all live sequences together,
+    None; `block_states[i]` what its block's arrangement keeps beside its mixer. `max_tokens` bounds the tokens held by all live sequences together,
     each rounded up to a multiple of 64; `max_seq_len` bounds one sequence;
     `step_tokens` bounds the new tokens of one sequence in one step (it sizes
     the ring of window groups)."""
 
     def __init__(self, requests, states, max_tokens: int, max_seq_len: int, max_slots: int,
-                 dtype, device, step_tokens: int | None = None):
+                 dtype, device, step_tokens: int | None = None, block_states=None):
         self.max_seq_len = max_seq_len
         self.max_slots = max_slots
         self.dtype = dtype
@@ -155,13 +155,12 @@ class PagedCache:
                 shape = (len(group.entries), n_pages.value, group.n_kv_heads, PAGE)
                 group.keys = torch.zeros(shape + (group.head_dim,), dtype=dtype, device=self.device)
                 group.values = torch.zeros(shape + (group.value_dim,), dtype=dtype, device=self.device)
-        self.states = []
-        for request in states:
-            if request is None:
-                self.states.append(None)
-            else:
-                self.states.append(torch.zeros((max_slots, *request.shape), dtype=request.dtype or dtype,
-                                               device=self.device))
+        def tensors_of(wanted):
+            return [None if request is None else
+                    torch.zeros((max_slots, *request.shape), dtype=request.dtype or dtype, device=self.device)
+                    for request in wanted]
+        self.states = tensors_of(states)
+        self.block_states = tensors_of(block_states or [])
 
     def __del__(self):
         handle = getattr(self, "_handle", None)
@@ -175,7 +174,7 @@ class PagedCache:
         """Take a free slot: length 0, no pages, state zeroed."""
         slot = c_int()
         native.check(native.lib().llmh_cache_acquire(self._handle, byref(slot)))
-        for state in self.states:
+        for state in self.states + self.block_states:
             if state is not None:
                 state[slot.value].zero_()
         return slot.value
@@ -238,6 +237,9 @@ class PagedCache:
     def state_view(self, entry: int):
         return self.states[entry]
 
+    def block_state_view(self, entry: int):
+        return self.block_states[entry]
+
     def held_tokens(self) -> int:
         """Tokens held now, each sequence rounded up to whole pages."""
         return native.lib().llmh_cache_held_tokens(self._handle)
@@ -245,7 +247,7 @@ class PagedCache:
     def bytes(self) -> int:
         total = sum(t.numel() * t.element_size() for g in self.groups
                     for t in (g.storage, g.keys, g.values if g.values is not g.keys else None) if t is not None)
-        total += sum(s.numel() * s.element_size() for s in self.states if s is not None)
+        total += sum(s.numel() * s.element_size() for s in self.states + self.block_states if s is not None)
         return total
 
     def check(self) -> None:

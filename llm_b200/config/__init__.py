@@ -1,4 +1,5 @@
 from .base import ConfigReader, read_config_json
+from .duvozen import DuvozenConfig
 from .guberax import GuberaxConfig
 from .llama import LlamaConfig
 from .mefolorn import MefolornConfig
@@ -12,6 +13,8 @@ register_architecture(GuberaxConfig.architecture, GuberaxConfig)
 register_architecture(MefolornConfig.architecture, MefolornConfig)
 register_architecture(ZogapelConfig.architecture, ZogapelConfig)
 register_architecture(ZemozenConfig.architecture, ZemozenConfig)
+register_architecture(DuvozenConfig.architecture, DuvozenConfig)
 
-__all__ = ["ConfigReader", "read_config_json", "LlamaConfig", "GuberaxConfig", "MefolornConfig", "ZogapelConfig", "ZemozenConfig", "config_class_for",
+__all__ = ["ConfigReader", "read_config_json", "LlamaConfig", "GuberaxConfig", "MefolornConfig", "ZogapelConfig", "ZemozenConfig",
+           "DuvozenConfig", "config_class_for",
            "config_from_dict", "known_architectures", "load_config", "register_architecture"]

@@ -22,7 +22,7 @@ using namespace llmb;
 
 LLMB_DEFINE_LAST_ERROR(llmb_attention_generic)
 
-constexpr int GENERIC_MAX_HEAD_DIM = 512;              // head sizes above LLMB_MAX_HEAD_DIM run the wider instantiation
+constexpr int GENERIC_MAX_HEAD_DIM = 1024;             // head sizes above LLMB_MAX_HEAD_DIM run the wider instantiations
 constexpr int WARPS = 4;
 
 // AHEAD: keys a warp fetches together. Four hide the loads' latency where a step has few blocks
@@ -32,7 +32,8 @@ constexpr int WARPS = 4;
 // Three optional extras, all applied in 32-bit when the four partial results are merged: `sinks` [heads]
 // (e^sink is one more term of the head's softmax denominator: it has no key and no value and is not
 // scaled), `gate` [T, heads] (the head's result is multiplied by sigmoid(gate)), `out_scale`. When the
-// value cache IS the key cache (a mixer whose cached rows serve as both), a row is loaded once.
+// value cache IS the key cache (a mixer whose cached rows serve as both), a row is loaded once; values narrower
+// than keys are then a row's first elements.
 // `softcap` > 0 bounds a score before the softmax: s <- softcap * tanh(s / softcap), after the scale.
 // Values may be wider or narrower than keys (`value_dim`; the value cache then has rows of that size and
 // the result rows hold n_heads * value_dim elements).
@@ -153,7 +154,7 @@ LLMB_EXPORT int llmb_attention_generic(const void* q, int q_stride, const void* 
     if (value_dim <= 0) value_dim = head_dim;
     LLMB_REQUIRE(head_dim > 0 && head_dim <= GENERIC_MAX_HEAD_DIM && value_dim <= GENERIC_MAX_HEAD_DIM,
                  "attention_generic: head_dim %d or value_dim %d exceeds %d", head_dim, value_dim, GENERIC_MAX_HEAD_DIM);
-    LLMB_REQUIRE(k_cache != v_cache || value_dim == head_dim, "attention_generic: values that are the keys have their size");
+    LLMB_REQUIRE(k_cache != v_cache || value_dim <= head_dim, "attention_generic: values that are the keys are not longer than they are");
     LLMB_REQUIRE(n_heads > 0 && n_kv_heads > 0 && n_heads % n_kv_heads == 0,
                  "attention_generic: %d heads are no multiple of %d kv heads", n_heads, n_kv_heads);
     LLMB_REQUIRE(n_heads <= 65535 && ring_pages > 0 && window >= 0, "attention_generic: bad sizes");
@@ -167,7 +168,8 @@ LLMB_EXPORT int llmb_attention_generic(const void* q, int q_stride, const void* 
         sinks, (const T*)gate, gate_stride, out_scale, softcap, value_dim)
 #define LLMB_GENERIC(T, AHEAD)                                                                          \
     do {                                                                                                \
-        if (wide) LLMB_GENERIC_AS(T, 1, GENERIC_MAX_HEAD_DIM / 32);                                      \
+        if (head_dim > 512 || value_dim > 512) LLMB_GENERIC_AS(T, 1, GENERIC_MAX_HEAD_DIM / 32);         \
+        else if (wide) LLMB_GENERIC_AS(T, 1, 512 / 32);                                                  \
         else LLMB_GENERIC_AS(T, AHEAD, LLMB_MAX_HEAD_DIM / 32);                                          \
     } while (0)
     if (dtype == LLMB_DTYPE_F32) {

@@ -580,10 +580,16 @@ LLMB_EXPORT int llmb_add_rows(float* x, const float* y, int n_rows, int hidden, 
 // ----------------------------------------------------------------------------- gated activation
 // act[t, f] = silu(gu[t, f]) * gu[t, F + f], silu(z) = z / (1 + exp(-z))
 // (apps/engine/kernels/gpu.cu:409-418, apps/engine/src/ops.rs:33-35). The gate
-// and up projections are one matrix product whose row holds [gate | up].
+// and up projections are one matrix product whose row holds [gate | up]. With `gelu` the activation is the
+// tanh form of gelu: 0.5 z (1 + tanh(w)) = z sigmoid(2 w), w = sqrt(2 / pi) (z + 0.044715 z^3).
+__device__ __forceinline__ float gated(float gate, float up, float linear, float cubic) {
+    float t = gate * fmaf(cubic * gate, gate, linear);          // silu: linear 1, cubic 0
+    return gate / (1.0f + expf(-t)) * up;
+}
+
 template <typename T>
 __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ act, long long total,
-                              int width) {
+                              int width, float linear, float cubic) {
     long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     long long stride = (long long)gridDim.x * blockDim.x;
     for (; i < total; i += stride) {
@@ -591,13 +597,13 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ act, lon
         int f = (int)(i - t * width);
         float g = to_float(gu[t * 2 * width + f]);
         float u = to_float(gu[t * 2 * width + width + f]);
-        act[i] = from_float<T>(g / (1.0f + expf(-g)) * u);
+        act[i] = from_float<T>(gated(g, u, linear, cubic));
     }
 }
 
 // bfloat16 rows whose width is a multiple of 8: 16 bytes of gate and of up per thread and step
 __global__ void swiglu_vec_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ act,
-                                  long long total_vectors, int vectors_per_row) {
+                                  long long total_vectors, int vectors_per_row, float linear, float cubic) {
     long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     long long stride = (long long)gridDim.x * blockDim.x;
     for (; i < total_vectors; i += stride) {
@@ -611,16 +617,16 @@ __global__ void swiglu_vec_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfl
         __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(&packed);
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
-            float gate = __bfloat162float(g[j]);
-            o[j] = __float2bfloat16_rn(gate / (1.0f + expf(-gate)) * __bfloat162float(u[j]));
+            o[j] = __float2bfloat16_rn(gated(__bfloat162float(g[j]), __bfloat162float(u[j]), linear, cubic));
         }
         reinterpret_cast<uint4*>(act)[i] = packed;
     }
 }
 
-LLMB_EXPORT int llmb_swiglu(const void* gu, void* act, int dtype, int n_tokens, int width,
+LLMB_EXPORT int llmb_swiglu(const void* gu, void* act, int dtype, int n_tokens, int width, int gelu,
                             cudaStream_t stream) {
     if (n_tokens == 0) return LLMB_OK;
+    float linear = gelu ? 1.5957691216057308f : 1.0f, cubic = gelu ? 0.0713548162726009f : 0.0f;
     LLMB_REQUIRE(n_tokens > 0 && width > 0, "swiglu: bad sizes");
     long long total = (long long)n_tokens * width;
     if (dtype == LLMB_DTYPE_BF16 && width % 8 == 0 &&
@@ -628,14 +634,14 @@ LLMB_EXPORT int llmb_swiglu(const void* gu, void* act, int dtype, int n_tokens, 
         long long vectors = total / 8;
         int blocks = (int)((vectors + 255) / 256 < 148 * 16 ? (vectors + 255) / 256 : 148 * 16);
         swiglu_vec_kernel<<<blocks, 256, 0, stream>>>((const __nv_bfloat16*)gu, (__nv_bfloat16*)act,
-                                                      vectors, width / 8);
+                                                      vectors, width / 8, linear, cubic);
         return check_launch("swiglu");
     }
     int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
     if (dtype == LLMB_DTYPE_F32)
-        swiglu_kernel<float><<<blocks, 256, 0, stream>>>((const float*)gu, (float*)act, total, width);
+        swiglu_kernel<float><<<blocks, 256, 0, stream>>>((const float*)gu, (float*)act, total, width, linear, cubic);
     else if (dtype == LLMB_DTYPE_BF16)
-        swiglu_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>((const __nv_bfloat16*)gu, (__nv_bfloat16*)act, total, width);
+        swiglu_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>((const __nv_bfloat16*)gu, (__nv_bfloat16*)act, total, width, linear, cubic);
     else
         return fail(LLMB_ERR_ARGUMENT, "swiglu: unknown dtype %d", dtype);
     return check_launch("swiglu");

@@ -64,8 +64,9 @@ struct Epilogue {
     int ldo;
     int tokens, outs;        // valid tokens and output columns (rows of the weight matrix)
     int glu;                 // gated activation: the weight rows alternate 16 gate rows, 16 up rows;
-                             // out is bfloat16 [tokens, ldo] with outs / 2 columns silu(gate) * up
+                             // out is bfloat16 [tokens, ldo] with outs / 2 columns act(gate) * up
     llmb_gemm_fusion f;      // what else the epilogue does (fusion.h); all zero: nothing
+    float act_linear, act_cubic;      // which act (see gated)
 };
 
 // 1 / sqrt(mean of squares + eps) of an input row from the partial sums its producer left. A whole warp
@@ -129,7 +130,12 @@ __device__ __forceinline__ void tile_rstd(const Epilogue& ep, float* rstd, int q
 
 static_assert(LLMB_GLU_BLOCK == 16, "the gated epilogue reads 16 gate and 16 up columns of tensor memory per pair");
 
-__device__ __forceinline__ float silu_mul(float gate, float up) { return gate / (1.0f + expf(-gate)) * up; }
+// act(gate) * up. Both activations are z sigmoid(t): silu has t = z, and the tanh form of gelu, 0.5 z (1 + tanh(u)) with
+// u = sqrt(2 / pi) (z + 0.044715 z^3), is z sigmoid(2 u); t = z (act_linear + act_cubic z^2) gives either.
+__device__ __forceinline__ float gated(const Epilogue& ep, float gate, float up) {
+    float t = gate * fmaf(ep.act_cubic * gate, gate, ep.act_linear);
+    return gate / (1.0f + expf(-t)) * up;
+}
 
 // One work unit: output tile (tile_a, tile_b) and one slice of its k-blocks.
 struct Unit {
@@ -172,7 +178,7 @@ __device__ __forceinline__ void store_columns(const Epilogue& ep, int swap, int 
             float up = __shfl_xor_sync(0xffffffffu, v[j], 16);
             int token = tile_b * BN + c + j;
             if (lane < 16 && a_row < ep.outs && token < ep.tokens)
-                o[(size_t)token * ep.ldo + feature] = __float2bfloat16_rn(silu_mul(v[j], up));
+                o[(size_t)token * ep.ldo + feature] = __float2bfloat16_rn(gated(ep, v[j], up));
         }
         return;
     }
@@ -587,8 +593,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
 #pragma unroll
                         for (int j = 0; j < 8; ++j)
                             h[j] = __floats2bfloat162_rn(
-                                silu_mul(__uint_as_float(g[2 * j]) * r, __uint_as_float(u[2 * j]) * r),
-                                silu_mul(__uint_as_float(g[2 * j + 1]) * r, __uint_as_float(u[2 * j + 1]) * r));
+                                gated(ep, __uint_as_float(g[2 * j]) * r, __uint_as_float(u[2 * j]) * r),
+                                gated(ep, __uint_as_float(g[2 * j + 1]) * r, __uint_as_float(u[2 * j + 1]) * r));
                         __nv_bfloat16* dst = o + (size_t)a_row * ep.ldo + n0 / 2;
                         if ((ep.ldo & 7) == 0) {
                             reinterpret_cast<uint4*>(dst)[0] = packed[0];
@@ -779,7 +785,7 @@ splitk_sum_kernel(const float* __restrict__ partials, Epilogue ep, int tiles_a, 
             int gate_row = (feature / LLMB_GLU_BLOCK) * 2 * LLMB_GLU_BLOCK + feature % LLMB_GLU_BLOCK;
             float gate = split_sum(partials, tiles_a, splits, bn, token, gate_row) * scale;
             float up = split_sum(partials, tiles_a, splits, bn, token, gate_row + LLMB_GLU_BLOCK) * scale;
-            reinterpret_cast<__nv_bfloat16*>(ep.out)[(size_t)token * ep.ldo + feature] = __float2bfloat16_rn(silu_mul(gate, up));
+            reinterpret_cast<__nv_bfloat16*>(ep.out)[(size_t)token * ep.ldo + feature] = __float2bfloat16_rn(gated(ep, gate, up));
         } else {
             float v = split_sum(partials, tiles_a, splits, bn, token, feature) * scale + (ep.bias ? ep.bias[feature] : 0.f);
             size_t at = (size_t)token * ep.ldo + feature;
@@ -870,8 +876,8 @@ splitk_sum4_kernel(const float* __restrict__ partials, Epilogue ep, int tiles_a,
             float4 g = split_sum4(partials, tiles_a, splits, bn, token, gate_row);
             float4 u = split_sum4(partials, tiles_a, splits, bn, token, gate_row + LLMB_GLU_BLOCK);
             *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(ep.out) + (size_t)token * ep.ldo + feature) =
-                pack4(silu_mul(g.x * scale, u.x * scale), silu_mul(g.y * scale, u.y * scale),
-                      silu_mul(g.z * scale, u.z * scale), silu_mul(g.w * scale, u.w * scale));
+                pack4(gated(ep, g.x * scale, u.x * scale), gated(ep, g.y * scale, u.y * scale),
+                      gated(ep, g.z * scale, u.z * scale), gated(ep, g.w * scale, u.w * scale));
         } else {
             float4 v = split_sum4(partials, tiles_a, splits, bn, token, feature);
             float4 b = ep.bias ? *reinterpret_cast<const float4*>(ep.bias + feature) : make_float4(0.f, 0.f, 0.f, 0.f);
@@ -1299,8 +1305,8 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
 #pragma unroll
                         for (int j = 0; j < 8; ++j)
                             h[j] = __floats2bfloat162_rn(
-                                silu_mul(__uint_as_float(g[2 * j]) * r, __uint_as_float(uu[2 * j]) * r),
-                                silu_mul(__uint_as_float(g[2 * j + 1]) * r, __uint_as_float(uu[2 * j + 1]) * r));
+                                gated(ep, __uint_as_float(g[2 * j]) * r, __uint_as_float(uu[2 * j]) * r),
+                                gated(ep, __uint_as_float(g[2 * j + 1]) * r, __uint_as_float(uu[2 * j + 1]) * r));
                         __nv_bfloat16* dst = o + (size_t)a_row * ep.ldo + n0 / 2;
                         if ((ep.ldo & 7) == 0) {
                             reinterpret_cast<uint4*>(dst)[0] = packed[0];
@@ -1593,7 +1599,7 @@ LLMB_EXPORT int llmb_gemm_tc_fuses_rope(int M, int N, int K, int n_heads, int n_
 // out[M, N] = x[M, K] . w[N, K]^T (+ bias[N]); or residual[M, N] += the same.
 // allow_pair != 0: products with more than 128 rows run 256 x 256 tiles on pairs of SMs.
 // glu != 0: w holds gate and up rows alternating in blocks of 16 (N = 2 F rows, N % 32 == 0) and
-// out is bfloat16 [M, ldo] with F columns silu(gate) * up; no bias, no residual.
+// out is bfloat16 [M, ldo] with F columns act(gate) * up (1: silu, 2: the tanh form of gelu); no bias, no residual.
 // fusion (optional): see fusion.h. *applied (optional) tells which parts ran inside the kernels:
 // a folded norm always does; the rows and sums for the next norm and the rotation with the cache
 // write only where the shape's kernels have them, else the caller runs them as kernels of their own.
@@ -1612,6 +1618,7 @@ LLMB_EXPORT int llmb_gemm_tc_ex(const void* x, int ldx, const void* w, const flo
     LLMB_REQUIRE((out != nullptr) != (residual != nullptr), "gemm_tc: give out or residual");
     LLMB_REQUIRE(residual || out_dtype == LLMB_DTYPE_BF16 || out_dtype == LLMB_DTYPE_F32,
                  "gemm_tc: unknown output dtype %d", out_dtype);
+    LLMB_REQUIRE(glu >= 0 && glu <= 2, "gemm_tc: unknown gated activation %d", glu);
     if (glu) {
         LLMB_REQUIRE(N % 32 == 0 && !bias && !residual && out_dtype == LLMB_DTYPE_BF16 && ldo >= N / 2,
                      "gemm_tc: the gated epilogue needs N %% 32 == 0, a bfloat16 output and no bias");
@@ -1624,7 +1631,8 @@ LLMB_EXPORT int llmb_gemm_tc_ex(const void* x, int ldx, const void* w, const flo
         LLMB_REQUIRE(partials && counters && partial_floats >= llmb_gemm_tc_scratch_floats(M, N, K) &&
                      n_counters >= p.tiles_a * p.tiles_b, "gemm_tc: scratch is missing or too small");
     }
-    Epilogue ep{bias, out, residual, out_dtype == LLMB_DTYPE_BF16, ldo, M, N, glu != 0, {}};
+    Epilogue ep{bias, out, residual, out_dtype == LLMB_DTYPE_BF16, ldo, M, N, glu != 0, {},
+                glu == 2 ? 1.5957691216057308f : 1.0f, glu == 2 ? 0.0713548162726009f : 0.0f};
     int did = 0;
     if (fusion) {
         llmb_gemm_fusion f = *fusion;

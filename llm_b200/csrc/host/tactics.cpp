@@ -25,6 +25,9 @@ struct Shape {
     int decode = 0, n_heads = 1, n_kv_heads = 1, head_dim = 0, window = 0, packed = 0;
     // differential attention: head_dim is the size of one map, value_dim the size of a value
     int value_dim = 0, keep_first = 0;
+    // latent attention with a shared rotated key part: head_dim is a head's unrotated part, fresh says that every
+    // sequence of the pass starts at its first token
+    int kv_rank = 0, rot_dim = 0, fresh = 0;
     // both
     int bf16 = 0;          // operands (and caches) are bfloat16
     int aligned = 1;       // operands start on 16-byte boundaries
@@ -156,6 +159,23 @@ std::string sigmoid_decode_guard(const Shape& s) {
     return sigmoid_tiles_guard(s);
 }
 
+std::string latent_generic_guard(const Shape& s) {
+    if (s.kv_rank + s.rot_dim > 1024)
+        return "a cached row of " + std::to_string(s.kv_rank) + " + " + std::to_string(s.rot_dim) + " elements exceeds 1024";
+    return "";
+}
+
+std::string latent_tiles_guard(const Shape& s) {
+    if (!s.bf16) return "bfloat16 caches only";
+    if (s.kv_rank % 8 || s.rot_dim % 8)
+        return "a latent of " + std::to_string(s.kv_rank) + " or a rotated part of " + std::to_string(s.rot_dim) +
+               " elements is no multiple of 8 (16-byte copies)";
+    if (s.kv_rank > 512 || s.kv_rank + s.rot_dim > 640)
+        return "a cached row of " + std::to_string(s.kv_rank) + " + " + std::to_string(s.rot_dim) +
+               " elements (served: up to 512, and 640 in all)";
+    return "";
+}
+
 const std::vector<Row>& table(int family) {
     static const std::vector<Row> linear = {
         {"gemm_tc", 30, tc_guard,
@@ -219,7 +239,17 @@ const std::vector<Row>& table(int family) {
          "32-bit arithmetic, any sizes up to 256, up to 128 heads, any group and window; the only variant of the "
          "32-bit path"},
     };
-    return family == 0 ? linear : family == 1 ? attention : family == 2 ? diff_attention : sigmoid_attention;
+    static const std::vector<Row> latent_attention = {
+        {"latent_tiles", 10, latent_tiles_guard,
+         "softmax attention of (token, head) pairs over the cached latent rows: all heads share a row, so a page goes "
+         "into shared memory once for up to 64 pairs; mma.sync tiles, scores by (row, key) parts over eight warps, value "
+         "columns over eight warps; slices of a long sequence in decode steps, merged by a second kernel"},
+        {"latent_generic", 0, latent_generic_guard,
+         "attention_generic with one key head whose first elements are the values: one block per (token, head), 32-bit "
+         "arithmetic, rows up to 1024; the only variant of the 32-bit path"},
+    };
+    return family == 0 ? linear : family == 1 ? attention : family == 2 ? diff_attention
+         : family == 3 ? sigmoid_attention : latent_attention;
 }
 
 std::set<std::string>& switched_off() {
@@ -249,17 +279,19 @@ void copy_out(const std::string& text, char* out, int capacity) {
 
 }  // namespace
 
-// family: 0 products, 1 attention, 2 differential attention, 3 sigmoid attention. shape: 12 ints {m, n, k, lda, decode,
-// n_heads, n_kv_heads, head_dim, window, packed, bf16, aligned}, for families 2 and 3 two more {value_dim, keep_first}. name and
-// reasons are filled up to their capacities.
+// family: 0 products, 1 attention, 2 differential attention, 3 sigmoid attention, 4 latent attention. shape: 12 ints {m, n, k, lda, decode,
+// n_heads, n_kv_heads, head_dim, window, packed, bf16, aligned}, from family 2 on two more {value_dim, keep_first}, for family 4
+// (latent attention with a shared rotated key part) three more {kv_rank, rot_dim, fresh}. name and reasons are filled up to
+// their capacities.
 LLMH_EXPORT int llmh_tactics_choose(int family, const int* shape, char* name, int name_capacity, char* reasons,
                                     int reasons_capacity) {
     return guarded([&] {
-        if (family < 0 || family > 3) throw Failure{LLMH_FORMAT, "unknown kernel family"};
+        if (family < 0 || family > 4) throw Failure{LLMH_FORMAT, "unknown kernel family"};
         Shape s;
         s.m = shape[0]; s.n = shape[1]; s.k = shape[2]; s.lda = shape[3];
         s.decode = shape[4]; s.n_heads = std::max(shape[5], 1); s.n_kv_heads = std::max(shape[6], 1);
         s.head_dim = shape[7]; s.window = shape[8]; s.packed = shape[9]; s.bf16 = shape[10]; s.aligned = shape[11];
+        if (family == 4) { s.kv_rank = shape[14]; s.rot_dim = shape[15]; s.fresh = shape[16]; }
         if (family >= 2) { s.value_dim = shape[12]; s.keep_first = shape[13]; }
         std::string why;
         copy_out(choose(family, s, &why), name, name_capacity);
@@ -275,10 +307,10 @@ LLMH_EXPORT void llmh_tactics_set_disabled(const char* name, int disabled) {
 }
 LLMH_EXPORT int llmh_tactics_is_disabled(const char* name) { return switched_off().count(name) ? 1 : 0; }
 
-LLMH_EXPORT int llmh_tactics_rows(int family) { return (family >= 0 && family <= 3) ? (int)table(family).size() : 0; }
+LLMH_EXPORT int llmh_tactics_rows(int family) { return (family >= 0 && family <= 4) ? (int)table(family).size() : 0; }
 LLMH_EXPORT int llmh_tactics_row(int family, int index, const char** name, int* rank, const char** evidence) {
     return guarded([&] {
-        if (family < 0 || family > 3 || index < 0 || index >= (int)table(family).size())
+        if (family < 0 || family > 4 || index < 0 || index >= (int)table(family).size())
             throw Failure{LLMH_INVARIANT, "no such row"};
         const Row& row = table(family)[index];
         *name = row.name;

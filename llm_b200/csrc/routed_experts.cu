@@ -11,6 +11,7 @@
 //          router may have more outputs than there are experts: the last ones are pass-through experts without
 //          matrices whose result is the token's own row h (times the weight); a small kernel writes those rows,
 //          the plan and the products see only the assignments of experts that have matrices.
+//          `scoring` 2: scores s = sigmoid(z), the `top` largest chosen, weights s as they are.
 //          `weight_scale` multiplies every weight (a constant in front of the whole feed-forward).
 // plan     counts the assignments of every expert, lists them grouped by expert (inside an expert in rising
 //          order, so the plan is a function of the routing alone) and cuts every expert's list into tiles of 32
@@ -21,6 +22,8 @@
 //          (h_t gathered through the list), one weight matrix [2 F, K] per expert (gate rows, then up).
 // down     for every tile: y[t * top + k, :] = weight[t, k] * (W_down,e act[s, :]), 32-bit, written at the
 //          assignment's own index; the sum over k is taken by the kernel behind (fixed order).
+// With the weight on the expert's input instead of its result, up applies it to its 32-bit sums (W (w h) = w W h) in
+// front of the activation, and down's rows are not weighted.
 // Every output element is one sum over K in rising order, whatever else is in its tile: results do
 // not depend on the batch.
 //
@@ -40,7 +43,7 @@ using namespace llmb;
 
 LLMB_DEFINE_LAST_ERROR(llmb_routed_experts)
 
-constexpr int MAX_TOP = 16;
+constexpr int MAX_TOP = 64;
 constexpr int TILE_M = 32;
 
 __device__ __forceinline__ void load4(const float* p, float (&x)[4]) {
@@ -142,6 +145,10 @@ router_kernel(const T* __restrict__ h, int ld, const float* __restrict__ w, cons
         ids[t * top + k] = best;
         mine[best] = -INFINITY;
     }
+    if (scoring == 2) {                    // (the sigmoid rises with the logit: the largest logits are the largest scores)
+        for (int k = 0; k < top; ++k) weights[t * top + k] = 1.0f / (1.0f + expf(-chosen[k])) * weight_scale;
+        return;
+    }
     float total = 0.f, largest = chosen[0];
     for (int k = 0; k < top; ++k) { chosen[k] = expf(chosen[k] - largest); total += chosen[k]; }
     for (int k = 0; k < top; ++k) weights[t * top + k] = chosen[k] / total * weight_scale;
@@ -241,7 +248,8 @@ plan_kernel(const int* __restrict__ ids, int n_assign, int E, int* __restrict__ 
 constexpr int BN = 64, BK = 16;
 
 // GLU: W is [2 N, K] per expert (gate rows, then up rows), the result silu(gate) * up in T.
-// else: the result weight[row] * sum in 32-bit at row `sorted[s]` of y.
+// else: the result weight[row] * sum in 32-bit at row `sorted[s]` of y. `weights` may be null (1) in either; with
+// GLU both sums are multiplied by the row's weight first (a weight on the expert's input).
 template <typename T, bool GLU>
 __global__ void __launch_bounds__(256)
 expert_product_kernel(const T* __restrict__ A, int lda, int a_div, const T* __restrict__ W, long long w_stride, int N,
@@ -298,18 +306,18 @@ expert_product_kernel(const T* __restrict__ A, int lda, int a_div, const T* __re
         int r = ty * 2 + i;
         if (r >= rows) continue;
         int s = first + r;
+        int assignment = sorted[s];
+        float wgt = weights ? weights[assignment] : 1.f;
         if (GLU) {
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 int col = n0 + tx * 4 + j;
                 if (col < N) {
-                    float g = acc[0][i][j];
-                    act[(long long)s * N + col] = from_float<T>(g / (1.0f + expf(-g)) * acc[GLU ? 1 : 0][i][j]);
+                    float g = wgt * acc[0][i][j];
+                    act[(long long)s * N + col] = from_float<T>(g / (1.0f + expf(-g)) * (wgt * acc[GLU ? 1 : 0][i][j]));
                 }
             }
         } else {
-            int assignment = sorted[s];
-            float wgt = weights[assignment];
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 int col = n0 + tx * 4 + j;
@@ -415,8 +423,9 @@ expert_product_tc_kernel(const __nv_bfloat16* __restrict__ A, int lda, int a_div
                         int c = warp * 32 + nj * 8 + (lane & 3) * 2 + (f & 1);
                         int feature = n0 + c;
                         if (r < rows && feature < N) {
-                            float g = acc[mi][nj][f];
-                            act[(long long)(first + r) * N + feature] = __float2bfloat16_rn(g / (1.0f + expf(-g)) * up[r][c]);
+                            float wgt = weights ? weights[sorted[first + r]] : 1.f;
+                            float g = wgt * acc[mi][nj][f];
+                            act[(long long)(first + r) * N + feature] = __float2bfloat16_rn(g / (1.0f + expf(-g)) * (wgt * up[r][c]));
                         }
                     }
     } else {
@@ -427,7 +436,7 @@ expert_product_tc_kernel(const __nv_bfloat16* __restrict__ A, int lda, int a_div
                 int r = mi * 16 + (lane >> 2) + f2 * 8;
                 if (r >= rows) continue;
                 int assignment = sorted[first + r];
-                float wgt = weights[assignment];
+                float wgt = weights ? weights[assignment] : 1.f;
 #pragma unroll
                 for (int nj = 0; nj < 4; ++nj)
 #pragma unroll
@@ -572,6 +581,7 @@ expert_product_wide_kernel(const __grid_constant__ CUtensorMap map_a, const __gr
             uint32_t taddr = tmem_base + ((uint32_t)(quarter * 32) << 16);
             bool live = row < rows;
             if (GLU) {
+                float wgt = (live && weights) ? weights[sorted[first + row]] : 1.f;
                 __nv_bfloat16* out = act + (long long)(first + row) * N + n0;
                 bool vector = N % 8 == 0;
 #pragma unroll 1
@@ -583,8 +593,8 @@ expert_product_wide_kernel(const __grid_constant__ CUtensorMap map_a, const __gr
                     float v[16];
 #pragma unroll
                     for (int j = 0; j < 16; ++j) {
-                        float gate = __uint_as_float(g[j]);
-                        v[j] = gate / (1.0f + expf(-gate)) * __uint_as_float(u[j]);
+                        float gate = wgt * __uint_as_float(g[j]);
+                        v[j] = gate / (1.0f + expf(-gate)) * (wgt * __uint_as_float(u[j]));
                     }
                     if (vector && n0 + c + 16 <= N) {
                         uint32_t packed[8];
@@ -604,7 +614,7 @@ expert_product_wide_kernel(const __grid_constant__ CUtensorMap map_a, const __gr
                 }
             } else {
                 int assignment = live ? sorted[first + row] : 0;
-                float wgt = live ? weights[assignment] : 0.f;
+                float wgt = live ? (weights ? weights[assignment] : 1.f) : 0.f;
                 float* out = y + (long long)assignment * N + n0;
                 bool vector = N % 4 == 0;
 #pragma unroll 1
@@ -665,11 +675,15 @@ LLMB_EXPORT int llmb_routed_experts(const void* h, int ld, int dtype, const floa
                                     const void* w_up, const void* w_down, int* ids, float* weights, int* sorted,
                                     int* plan, void* act, float* y, void* gathered, int n_tokens, int hidden, int F,
                                     int E, int top, int tensor_cores, int scoring, const float* correction,
-                                    int pass_through, float weight_scale, cudaStream_t stream) {
+                                    int pass_through, float weight_scale, int weight_on_input, cudaStream_t stream) {
     if (n_tokens == 0) return LLMB_OK;
     LLMB_REQUIRE(hidden > 0 && F > 0 && E > 0 && top > 0 && pass_through >= 0 && top <= E + pass_through && top <= MAX_TOP,
                  "routed_experts: %d of %d experts (at most %d are chosen)", top, E + pass_through, MAX_TOP);
-    LLMB_REQUIRE(scoring == 0 || scoring == 1, "routed_experts: scoring %d (0: softmax over the chosen, 1: over all)", scoring);
+    LLMB_REQUIRE(scoring >= 0 && scoring <= 2, "routed_experts: scoring %d (0: softmax over the chosen, 1: over all, 2: sigmoid)", scoring);
+    LLMB_REQUIRE(!weight_on_input || pass_through == 0, "routed_experts: rows handed through have no input to weight");
+    // where the routing weights enter: the gate and up sums, or the rows of the down product
+    const float* up_weights = weight_on_input ? weights : nullptr;
+    const float* down_weights = weight_on_input ? nullptr : weights;
     int R = E + pass_through;                                  // outputs of the router
     LLMB_REQUIRE(E <= 2048, "routed_experts: %d experts (up to 2048 are built)", E);
     int n_assign = n_tokens * top;
@@ -740,33 +754,33 @@ LLMB_EXPORT int llmb_routed_experts(const void* h, int ld, int dtype, const floa
         auto down = wide256 ? expert_product_wide_kernel<false, 256> : expert_product_wide_kernel<false, 128>;
         LLMB_CUDA(llmb::launch(up, dim3((F + GN / 2 - 1) / (GN / 2), tiles), dim3(G_THREADS), smem, stream, true, map_x, map_up,
                                (const int*)plan, E, max_tiles, 2 * F, F, (hidden + GK - 1) / GK, (B*)act, (float*)nullptr,
-                               (const int*)sorted, (const float*)nullptr, status_dev));
+                               (const int*)sorted, up_weights, status_dev));
         LLMB_CUDA(llmb::launch(down, dim3((hidden + GN - 1) / GN, tiles), dim3(G_THREADS), smem, stream, true, map_act, map_down,
                                (const int*)plan, E, max_tiles, hidden, hidden, (F + GK - 1) / GK, (B*)nullptr, y,
-                               (const int*)sorted, (const float*)weights, status_dev));
+                               (const int*)sorted, down_weights, status_dev));
     } else if (tc) {
         typedef __nv_bfloat16 B;
         LLMB_CUDA(llmb::launch(expert_product_tc_kernel<true>, dim3((F + 63) / 64, max_tiles), dim3(128), 0, stream, true,
                                (const B*)h, ld, top, (const B*)w_up, up_stride, F, hidden, (const int*)sorted,
-                               (const int*)plan, E, max_tiles, (B*)act, (float*)nullptr, (const float*)nullptr));
+                               (const int*)plan, E, max_tiles, (B*)act, (float*)nullptr, up_weights));
         LLMB_CUDA(llmb::launch(expert_product_tc_kernel<false>, dim3((hidden + 127) / 128, max_tiles), dim3(128), 0, stream,
                                true, (const B*)act, F, 1, (const B*)w_down, down_stride, hidden, F, (const int*)sorted,
-                               (const int*)plan, E, max_tiles, (B*)nullptr, y, (const float*)weights));
+                               (const int*)plan, E, max_tiles, (B*)nullptr, y, down_weights));
     } else if (dtype == LLMB_DTYPE_F32) {
         LLMB_CUDA(llmb::launch(expert_product_kernel<float, true>, grid_up, dim3(256), 0, stream, true, (const float*)h, ld,
                                top, (const float*)w_up, up_stride, F, hidden, (const int*)sorted, (const int*)plan, E,
-                               max_tiles, (float*)act, (float*)nullptr, (const float*)nullptr));
+                               max_tiles, (float*)act, (float*)nullptr, up_weights));
         LLMB_CUDA(llmb::launch(expert_product_kernel<float, false>, grid_down, dim3(256), 0, stream, true,
                                (const float*)act, F, 1, (const float*)w_down, down_stride, hidden, F, (const int*)sorted,
-                               (const int*)plan, E, max_tiles, (float*)nullptr, y, (const float*)weights));
+                               (const int*)plan, E, max_tiles, (float*)nullptr, y, down_weights));
     } else {
         typedef __nv_bfloat16 B;
         LLMB_CUDA(llmb::launch(expert_product_kernel<B, true>, grid_up, dim3(256), 0, stream, true, (const B*)h, ld, top,
                                (const B*)w_up, up_stride, F, hidden, (const int*)sorted, (const int*)plan, E, max_tiles,
-                               (B*)act, (float*)nullptr, (const float*)nullptr));
+                               (B*)act, (float*)nullptr, up_weights));
         LLMB_CUDA(llmb::launch(expert_product_kernel<B, false>, grid_down, dim3(256), 0, stream, true, (const B*)act, F, 1,
                                (const B*)w_down, down_stride, hidden, F, (const int*)sorted, (const int*)plan, E,
-                               max_tiles, (B*)nullptr, y, (const float*)weights));
+                               max_tiles, (B*)nullptr, y, down_weights));
     }
     return check_launch("routed_experts");
 }

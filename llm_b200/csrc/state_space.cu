@@ -22,7 +22,7 @@
 //             tokens meet in one butterfly. A block holds 32 neighbouring columns, the grid is
 //             (column tiles, heads, sequences).
 // finish      y silu(z), the grouped norm, the weight and a scale, rounded to the run's dtype.
-#include "common.cuh"
+#include "scan.cuh"
 
 using namespace llmb;
 
@@ -83,33 +83,6 @@ __global__ void ssm_conv_state_kernel(const T* __restrict__ proj, int ld, int n_
         held[r] = src >= 0 ? to_float(in[(size_t)(first + src) * ld + c]) : st[(size_t)(r + n) * C + c];
     }
     for (int r = 0; r < n_taps - 1; ++r) st[(size_t)r * C + c] = held[r];
-}
-
-__device__ __forceinline__ void copy4(float* smem, const float* global) {
-    unsigned s = (unsigned)__cvta_generic_to_shared(smem);
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(s), "l"(global));
-}
-__device__ __forceinline__ void copy16(float* smem, const float* global) {
-    unsigned s = (unsigned)__cvta_generic_to_shared(smem);
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(s), "l"(global));
-}
-__device__ __forceinline__ void copies_commit() { asm volatile("cp.async.commit_group;\n" ::); }
-template <int LEFT> __device__ __forceinline__ void copies_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(LEFT)); }
-
-// One level of a butterfly over COUNT values a lane: lanes whose bit OFFSET is set keep the upper half of the
-// values and hand over the lower half, the others the reverse; what stays is own + partner's. After the
-// levels 16, 8, 4, 2, 1 on 32 values lane l holds the sum over all lanes of value l. Every value's sum runs through
-// the same tree of lane pairs (l, l ^ 16), then (l, l ^ 8), ..., whatever its index: a sum does not depend on the
-// place of its token in a group.
-template <int COUNT, int OFFSET>
-__device__ __forceinline__ void fold(float (&v)[32], int lane) {
-    bool up = (lane & OFFSET) != 0;
-#pragma unroll
-    for (int k = 0; k < COUNT; ++k) {
-        float send = up ? v[k] : v[COUNT + k];
-        float keep = up ? v[COUNT + k] : v[k];
-        v[k] = keep + __shfl_xor_sync(0xffffffffu, send, OFFSET);
-    }
 }
 
 // PER: state rows a lane holds of each column (N <= 32 * PER). A block: WARPS warps of COLS columns each, the

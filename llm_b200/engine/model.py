@@ -163,6 +163,10 @@ class DecoderModel:
             states.append(mixer.state_request())
         return kv, states
 
+    def block_state_requests(self) -> list:
+        """Per schedule entry, the StateRequest of the block's arrangement (or None)."""
+        return [self.blocks[item.layer].state_request() for item in self.spec.schedule]
+
     # ------------------------------------------------------------------ forward
 
     def forward(self, tokens, ctx, logit_rows):
@@ -178,7 +182,11 @@ class DecoderModel:
             if position >= len(schedule):
                 return None
             block = self.blocks[schedule[position].layer]
-            return block.input_emit(ctx, n, self.device) if getattr(block, "chains_norms", False) else None
+            if not getattr(block, "chains_norms", False):
+                return None
+            if getattr(block, "emit_has_state", False):      # what it asks for touches its own run's state
+                return block.input_emit(ctx, n, self.device, position)
+            return block.input_emit(ctx, n, self.device)
 
         def added_before(position):
             return position < len(schedule) and getattr(schedule[position], "add_embedding", False)

@@ -113,7 +113,8 @@ class Engine:
         model.prepare(self.max_seq_len)
         kv, states = model.cache_requests()
         self.cache = PagedCache(kv, states, max_tokens, self.max_seq_len, self.max_slots,
-                                self.dtype, self.device, self.step_tokens)
+                                self.dtype, self.device, self.step_tokens,
+                                block_states=model.block_state_requests())
         self.vocab = model.spec.vocab
         self.steps_run = 0
         self.workspace = Workspace(self.device, model.scratch_requests)

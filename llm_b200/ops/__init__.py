@@ -504,6 +504,81 @@ def norm_add_(x, y, gain_post, eps_post, terms: int = 1, gain_next=None, eps_nex
     return out
 
 
+#: the norms ops.output_norm_add_ knows, by the kind of their spec (LLMB: 0, 1)
+OUTPUT_NORMS = ("rmsnorm", "layernorm")
+
+
+def layernorm(x, gain, eps, out_dtype, rows=None, out=None):
+    """out[r, :] = (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps) * gain with v = x[rows[r] or r, :]; x and gain float32."""
+    _require_cuda(x, gain, rows)
+    hidden = x.shape[-1]
+    n = rows.numel() if rows is not None else x.shape[0]
+    if x.dtype != torch.float32 or gain.dtype != torch.float32 or not x.is_contiguous() or gain.numel() != hidden:
+        raise KernelError("layernorm: x and gain must be float32, x contiguous, the gain of x's width")
+    _check_out(out, (n, hidden), out_dtype, "layernorm")
+    if out is None:
+        out = torch.empty((n, hidden), dtype=out_dtype, device=x.device)
+    _call("output_norm", "llmb_layernorm", _ptr(x), _ptr(gain), _ptr(rows), _ptr(out), _c_int(_code(out_dtype)), _c_int(n),
+          _c_int(hidden), _c_float(eps), _stream())
+    return out
+
+
+def _check_conv(x, taps, state, out, what: str):
+    n, width = x.shape
+    k = taps.shape[0] if taps is not None else 0
+    _require_cuda(taps, state, out)
+    if taps is not None and (taps.dtype != torch.float32 or tuple(taps.shape) != (k, width) or not taps.is_contiguous()):
+        raise KernelError(f"{what}: the taps must be contiguous float32 [taps, {width}]")
+    if k > 1 and (state is None or state.dtype != torch.float32 or tuple(state.shape[1:]) != (k - 1, width)
+                  or state.stride(2) != 1 or state.stride(1) != width):
+        raise KernelError(f"{what}: the state must be float32 [slots, {k - 1}, {width}] with contiguous rows")
+    if tuple(out.shape) != (n, width) or not out.is_contiguous():
+        raise KernelError(f"{what}: the result must be contiguous [{n}, {width}]")
+    return k
+
+
+def input_conv(x, taps, state, cu_seqlens, slot_ids, out, max_new: int):
+    """out[t, c] = x[t, c] + sum_j taps[j, c] x[t - (K - 1) + j, c] over the tokens of each sequence (x float32 [T, width];
+    `taps` float32 [K, width], the last row the current token's, or None: out = x). The K - 1 rows before a sequence's first
+    token of the step come from `state` float32 [slots, K - 1, width] (a range of a wider row a slot is fine) and are
+    replaced by its last K - 1 rows. `max_new`: the most tokens a sequence brings. `out` in the run's dtype."""
+    _require_cuda(x, cu_seqlens, slot_ids)
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise KernelError("input_conv: x must be contiguous float32")
+    k = _check_conv(x, taps, state, out, "input_conv")
+    _call("output_norm", "llmb_input_conv", _ptr(x), _ptr(taps), _c_int(k), _ptr(state if k > 1 else None),
+          ctypes.c_longlong(state.stride(0) if k > 1 else 0), _ptr(cu_seqlens), _ptr(slot_ids), _ptr(out), _c_int(_code(out.dtype)),
+          _c_int(x.shape[0]), _c_int(cu_seqlens.numel() - 1), _c_int(max_new), _c_int(x.shape[1]), _stream())
+    return out
+
+
+def output_norm_add_(x, y, gain, eps, kind: str, terms: int = 1, extra=None, conv=None):
+    """x[t] += norm(s) * gain with s = sum_k y[t * terms + k] (+ extra[t]); x float32 [T, width], y float32 [T * terms, width],
+    extra float32 [T, width] or None; `kind` one of OUTPUT_NORMS. `conv` = (taps, state, slot_ids, out), in steps of one token
+    a sequence (token b is sequence b's): also what input_conv does with the new x."""
+    _require_cuda(x, y, gain, extra)
+    n, width = x.shape
+    if kind not in OUTPUT_NORMS:
+        raise KernelError(f"output_norm_add_: unknown norm '{kind}'")
+    for t, rows, what in ((x, n, "x"), (y, n * terms, "y"), (extra, n, "extra")):
+        if t is not None and (t.dtype != torch.float32 or tuple(t.shape) != (rows, width) or not t.is_contiguous()):
+            raise KernelError(f"output_norm_add_: {what} must be contiguous float32 [{rows}, {width}]")
+    if gain.dtype != torch.float32 or gain.numel() != width:
+        raise KernelError(f"output_norm_add_: the gain must be float32 [{width}]")
+    taps = state = slot_ids = out = None
+    k = 0
+    if conv is not None:
+        taps, state, slot_ids, out = conv
+        k = _check_conv(x, taps, state, out, "output_norm_add_")
+        if k > 1 and slot_ids.numel() != n:
+            raise KernelError("output_norm_add_: the convolution rides along in steps of one token a sequence only")
+    _call("output_norm", "llmb_output_norm_add", _ptr(y), _c_int(terms), _ptr(extra), _ptr(gain), _c_float(eps),
+          _c_int(OUTPUT_NORMS.index(kind)), _ptr(x), _c_int(n), _c_int(width), _c_int(1 if conv is not None else 0), _ptr(taps),
+          _c_int(k), _ptr(state if k > 1 else None), ctypes.c_longlong(state.stride(0) if k > 1 else 0), _ptr(slot_ids), _ptr(out),
+          _c_int(_code(out.dtype) if out is not None else 0), _stream())
+    return x
+
+
 def gelu_(a):
     """a = 0.5 a (1 + tanh(sqrt(2 / pi) (a + 0.044715 a^3))) in place (contiguous; 32-bit arithmetic)."""
     _require_cuda(a)
@@ -639,7 +714,52 @@ def state_space(proj, taps, conv_bias, state, tok_seq, cu_seqlens, slot_ids, rat
     return mixed
 
 
+# ----------------------------------------------------------------------------- forget-gated recurrence
+
+def forget_recurrence_work_width(n_heads: int, dim: int, vdim: int) -> int:
+    """Floats of a token's 32-bit work row: f, q and v."""
+    return (2 * n_heads * dim + n_heads * vdim + 3) // 4 * 4
+
+
+def forget_recurrence(proj, f_bias, lower, state, cu_seqlens, slot_ids, norm_weight, eps, work, o, mixed, n_heads, dim, vdim,
+                      single_tokens=False):
+    """Linear attention whose forget gate decides what is written, behind its projection. `proj` [T, >= 2 H D + H V] (run
+    dtype, rows contiguous) holds per token [q (H D) | f (H D) | v (H V)]; q <- silu(q), f <- l + (1 - l) sigmoid(f + bias)
+    (`f_bias`, `lower` float32 [H D]); per head S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T, o_t = S_t^T q_t; then
+    o / sqrt(mean(o^2) + eps) * norm_weight (float32 [V]) per head into `mixed` [T, H V] (run dtype). `state` float32
+    [slots, H V D]: S as [H, V, D], read and updated for the slots of the step. `work` float32
+    [T, forget_recurrence_work_width], `o` float32 [T, H V]: scratch. `single_tokens`: every sequence brings exactly one
+    token (token b is sequence b's)."""
+    _require_cuda(proj, f_bias, lower, state, cu_seqlens, slot_ids, norm_weight, work, o, mixed)
+    n, H, D, V = proj.shape[0], n_heads, dim, vdim
+    if proj.dim() != 2 or proj.shape[1] < 2 * H * D + H * V or proj.stride(1) != 1:
+        raise KernelError(f"forget_recurrence: the projection {tuple(proj.shape)} does not hold {2 * H * D + H * V} columns")
+    _check_rows(mixed, n, H * V, proj.dtype, "forget_recurrence: mixed")
+    for t, shape, what in ((f_bias, (H * D,), "the gate's bias"), (lower, (H * D,), "the lower bound"),
+                           (norm_weight, (V,), "norm weight"), (o, (n, H * V), "o")):
+        if t.dtype != torch.float32 or tuple(t.shape) != shape or not t.is_contiguous():
+            raise KernelError(f"forget_recurrence: {what} must be contiguous float32 {shape}")
+    width = forget_recurrence_work_width(H, D, V)
+    if work.dtype != torch.float32 or work.dim() != 2 or work.shape[0] < n or work.shape[1] < width or not work.is_contiguous():
+        raise KernelError(f"forget_recurrence: work must be contiguous float32 [T, >= {width}]")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.shape[1] < H * D * V or state.stride(1) != 1:
+        raise KernelError(f"forget_recurrence: the state must be float32 [slots, >= {H * D * V}]")
+    n_seqs = cu_seqlens.numel() - 1
+    warps = (V + 7) // 8
+    one = single_tokens and n == n_seqs and warps <= 32 and D <= 256 and not (D > 128 and warps > 16)
+    _call("forget_recurrence", "llmb_forget_recurrence", _ptr(proj), _c_int(proj.stride(0)), _c_int(_code(proj.dtype)),
+          _ptr(f_bias), _ptr(lower), _ptr(state), ctypes.c_longlong(state.stride(0)), _ptr(cu_seqlens), _ptr(slot_ids),
+          _ptr(norm_weight), _c_float(eps), _ptr(work), _c_int(work.shape[1]), _ptr(o), _ptr(mixed), _c_int(mixed.stride(0)),
+          _c_int(n), _c_int(n_seqs), _c_int(H), _c_int(D), _c_int(V), _c_int(1 if single_tokens else 0), _stream(),
+          kernels=1 if one else 3)
+    return mixed
+
+
 # ----------------------------------------------------------------------------- routed experts
+
+#: how a router scores and weights its outputs (RoutedExpertsSpec.scoring), by the number the kernel takes
+ROUTER_SCORING = ("chosen", "all", "sigmoid")
+
 
 def routed_experts_plan_ints(n_tokens: int, top: int, n_experts: int) -> int:
     sizer = load_library("routed_experts").llmb_routed_experts_plan_ints
@@ -661,7 +781,8 @@ def routed_experts_wide(n_tokens: int, top: int, n_experts: int, hidden: int, in
 
 
 def routed_experts(h, router, router_bias, w_up, w_down, top: int, ids, weights, order, plan, act, y, gathered=None,
-                   scoring: int = 0, correction=None, pass_through: int = 0, weight_scale: float = 1.0):
+                   scoring: int = 0, correction=None, pass_through: int = 0, weight_scale: float = 1.0,
+                   weight_on_input: bool = False):
     """A feed-forward of routed experts on the rows of h [T, hidden] (run dtype). Router logits
     z = router h + router_bias in 32-bit (`router` float32 [E, hidden]); the `top` largest are chosen and
     weighted by the softmax over them. Expert e: W_down,e (silu(W_gate,e h) * (W_up,e h)) with `w_up`
@@ -674,7 +795,8 @@ def routed_experts(h, router, router_bias, w_up, w_down, top: int, ids, weights,
     `scoring` 1: scores s = softmax(z) over all router outputs, the `top` largest of s + `correction` (float32, one
     per output; it takes part in the choice only) are chosen, weights s / (sum of the chosen s + 1e-20).
     `pass_through` > 0: the router has E + pass_through outputs, and the last ones are experts without matrices
-    whose result is h itself. `weight_scale` multiplies every weight."""
+    whose result is h itself. `weight_scale` multiplies every weight. `scoring` 2: scores s = sigmoid(z), the `top`
+    largest chosen, weights s as they are. `weight_on_input`: y[t * top + k] = expert(weight[t, k] h[t]) instead."""
     _require_cuda(h, router, router_bias, w_up, w_down, ids, weights, order, plan, act, y, gathered, correction)
     n, hidden = h.shape
     E, two_f, _ = w_up.shape
@@ -702,13 +824,14 @@ def routed_experts(h, router, router_bias, w_up, w_down, top: int, ids, weights,
     _call("routed_experts", "llmb_routed_experts", _ptr(h), _c_int(h.stride(0)), _c_int(_code(h.dtype)), _ptr(router),
           _ptr(router_bias), _ptr(w_up), _ptr(w_down), _ptr(ids), _ptr(weights), _ptr(order), _ptr(plan), _ptr(act),
           _ptr(y), _ptr(gathered if wide else None), _c_int(n), _c_int(hidden), _c_int(F), _c_int(E), _c_int(top),
-          _c_int(level), _c_int(scoring), _ptr(correction), _c_int(pass_through), _c_float(weight_scale), _stream(),
+          _c_int(level), _c_int(scoring), _ptr(correction), _c_int(pass_through), _c_float(weight_scale),
+          _c_int(1 if weight_on_input else 0), _stream(),
           kernels=(5 if wide else 4) + (1 if pass_through else 0))
     return y
 
 
-def swiglu(gate_up, out=None):
-    """act[t, f] = silu(gate_up[t, f]) * gate_up[t, F + f]."""
+def swiglu(gate_up, out=None, gelu: bool = False):
+    """act[t, f] = act(gate_up[t, f]) * gate_up[t, F + f]; act is silu, or with `gelu` the tanh form of gelu."""
     _require_cuda(gate_up)
     n, two_f = gate_up.shape
     width = two_f // 2
@@ -718,7 +841,7 @@ def swiglu(gate_up, out=None):
     if out is None:
         out = torch.empty((n, width), dtype=gate_up.dtype, device=gate_up.device)
     _call("elementwise", "llmb_swiglu", _ptr(gate_up), _ptr(out), _c_int(_code(gate_up.dtype)),
-          _c_int(n), _c_int(width), _stream())
+          _c_int(n), _c_int(width), _c_int(1 if gelu else 0), _stream())
     return out
 
 
@@ -851,7 +974,7 @@ def check_device_status() -> None:
     """Raise if a kernel of a loaded library reported a wait that ran out. Cheap (it
     reads a word of host memory); meaningful after the stream was synchronised."""
     from .build import _loaded
-    for name in ("gemm_tc", "attention_prefill_tc", "routed_experts"):
+    for name in ("gemm_tc", "attention_prefill_tc", "routed_experts", "latent_prefill_tc"):
         if name in _loaded:
             code = getattr(_loaded[name], f"llmb_{name}_status")()
             if code != 0:
@@ -907,7 +1030,7 @@ def linear(a, w, bias=None, out_dtype=None, residual=None, out=None, glu=False, 
     [M, N]) the product is added to it in place and it is returned; otherwise a
     new [M, N] tensor of `out_dtype` (default: a's dtype). With `glu`, w holds
     gate and up rows alternating in blocks of 16 and the result is
-    silu(gate) * up as [M, N / 2] in a's dtype, computed in the product's epilogue.
+    silu(gate) * up (or, with glu="gelu", the tanh form of gelu in silu's place) as [M, N / 2] in a's dtype, computed in the product's epilogue.
 
     What can ride along (bfloat16; where the shape's kernel does not have it, a kernel of its
     own runs behind the product, with the same result):
@@ -937,7 +1060,7 @@ def linear(a, w, bias=None, out_dtype=None, residual=None, out=None, glu=False, 
         _call("gemm_tc", "llmb_gemm_tc_ex", _ptr(a), _c_int(a.stride(0)), _ptr(w), None, _ptr(result),
               _c_int(_code(a.dtype)), None, _ptr(partials), ctypes.c_longlong(partials.numel()),
               _ptr(counters), _c_int(counters.numel()), _c_int(m), _c_int(n), _c_int(k),
-              _c_int(n // 2), _c_int(1), _c_int(0 if tactics.is_disabled("gemm_tc_pair") else 1),
+              _c_int(n // 2), _c_int(2 if glu == "gelu" else 1), _c_int(0 if tactics.is_disabled("gemm_tc_pair") else 1),
               ctypes.byref(_fusion_struct(norm, None, None)) if norm is not None else None, None,
               _stream(), kernels=_tc_kernels(m, n, k))
         return result
@@ -1176,6 +1299,123 @@ def attention_replay_key(step, n_heads: int, n_kv_heads: int, window: int = 0):
     return (False, max(step.new_counts))
 
 
+# ----------------------------------------------------------------------------- latent attention, shared rotated keys
+
+def latent_write(u, n_heads, dim, rot, rank, gain, eps, rope_table, interleaved, tok_pos, tok_seq, block_table, ring_pages,
+                 cache, queries=None, dense=None, write_cache=True):
+    """Behind the projection of a latent attention: `u` [T, >= H (D + R) + C + R] holds per token H query heads of
+    [D | R] elements, the latent c (C) and a rotated key part r (R) that all heads share. c / sqrt(mean(c^2) + eps) * gain
+    and the rotated r go as one row [C | R] into `cache` [pages, 1, 64, C + R] (unless `write_cache` is False) and, where given, into
+    `dense` [T, C + R]. The query heads' last R elements rotate: into the last R columns of `queries` [T, H (C + R)], or,
+    without it, where they are. `rope_table` float32 [positions, n_rot], n_rot <= R, or None. Norm and angles are 32-bit."""
+    _require_cuda(u, gain, rope_table, tok_pos, tok_seq, block_table, cache, queries, dense)
+    n, width = u.shape[0], rank + rot
+    if u.dim() != 2 or u.stride(1) != 1 or u.shape[1] < n_heads * (dim + rot) + width:
+        raise KernelError(f"latent_write: u {tuple(u.shape)} does not hold {n_heads} heads of {dim} + {rot} and {rank} + {rot}")
+    if gain.dtype != torch.float32 or gain.numel() != rank:
+        raise KernelError(f"latent_write: the gain must be float32 [{rank}]")
+    if tuple(cache.shape[1:]) != (1, PAGE, width) or cache.dtype != u.dtype or not cache.is_contiguous():
+        raise KernelError(f"latent_write: the cache {tuple(cache.shape)} does not hold rows of {width}")
+    for t, shape, what in ((queries, (n, n_heads * width), "queries"), (dense, (n, width), "dense")):
+        if t is not None and (tuple(t.shape) != shape or t.dtype != u.dtype or not t.is_contiguous()):
+            raise KernelError(f"latent_write: {what} must be contiguous {u.dtype} {shape}")
+    if rope_table is not None and (rope_table.dtype != torch.float32 or not rope_table.is_contiguous()
+                                   or rope_table.shape[1] > rot or rope_table.shape[1] % 2):
+        raise KernelError(f"latent_write: the table of angles must be contiguous float32 [positions, n_rot <= {rot}]")
+    _call("latent_attention", "llmb_latent_write", _ptr(u), _c_int(u.stride(0)), _c_int(_code(u.dtype)), _c_int(n_heads),
+          _c_int(dim), _c_int(rot), _c_int(rank), _ptr(gain), _c_float(eps), _ptr(rope_table),
+          _c_int(rope_table.shape[1] if rope_table is not None else 0), _c_int(1 if interleaved else 0), _ptr(tok_pos),
+          _ptr(tok_seq), _ptr(block_table), _c_int(block_table.shape[1]), _c_int(ring_pages), _ptr(cache),
+          _c_int(1 if write_cache else 0), _ptr(queries), _ptr(dense), _c_int(n), _stream())
+
+
+def head_products(x, x_head: int, w, out, out_head: int):
+    """out[t, h * out_head + n] = sum_k x[t, h * x_head + k] w[h, n, k]: a matrix per head (w [H, N, K] in x's dtype), heads
+    x_head columns of x and out_head columns of `out` apart. Columns of `out` between the heads' results are left alone."""
+    _require_cuda(x, w, out)
+    H, N, K = w.shape
+    if (x.dim() != 2 or out.dim() != 2 or out.shape[0] != x.shape[0] or x.stride(1) != 1 or out.stride(1) != 1
+            or x.shape[1] < (H - 1) * x_head + K or out.shape[1] < (H - 1) * out_head + N or x_head < K or out_head < N
+            or w.dtype != x.dtype or out.dtype != x.dtype or not w.is_contiguous()):
+        raise KernelError(f"head_products: {tuple(x.shape)} and {tuple(out.shape)} do not fit {H} matrices of {N} x {K}")
+    _call("latent_attention", "llmb_head_products", _ptr(x), _c_int(x.stride(0)), _c_int(x_head), _ptr(w), _c_int(H), _c_int(N),
+          _c_int(K), _ptr(out), _c_int(out.stride(0)), _c_int(out_head), _c_int(_code(x.dtype)), _c_int(x.shape[0]),
+          _c_int(0 if tactics.is_disabled("head_products_mma") else 1), _stream())
+    return out
+
+
+def latent_decode_splits(n_seqs: int, n_heads: int, max_len: int, pairs_fit: bool = False) -> int:
+    """Slices of the latent attention in a decode step: `decode_splits` for its blocks a sequence (64 heads each)."""
+    tile = 16 if n_heads <= 16 else 32 if n_heads <= 32 else 64
+    return decode_splits(n_seqs, (n_heads + tile - 1) // tile, max_len, wave=296 if pairs_fit else 148)
+
+
+@functools.lru_cache(maxsize=256)
+def _latent_pairs_fit(rank: int, rot: int, rows: int) -> bool:
+    return bool(load_library("latent_attention").llmb_latent_tile_pairs(_c_int(rank), _c_int(rot), _c_int(rows)))
+
+
+def latent_attention_replay_key(step, n_heads: int):
+    """What the launches of latent_attention depend on beyond the token and sequence counts (Part.replay_key)."""
+    if step.decode:          # (the slices follow from the sequences and the power-of-two bucket of the longest one's pages)
+        return (True, step.n_seqs, ((step.max_len + PAGE - 1) // PAGE - 1).bit_length())
+    return (False, max(step.new_counts))
+
+
+def latent_attention(queries, cache, block_table, ring_pages, tok_pos, tok_seq, n_heads, rank, rot, scale, out, decode=False,
+                     seq_lens=None, max_len=0, cu_seqlens=None, max_new=0, seq_order=None):
+    """Causal softmax attention of the new tokens' latent queries [T, H (C + R)] over the cached rows [pages, 1, 64, C + R],
+    whose first C elements are the values: out[t, h * C :] = sum_j softmax_j(scale q_h . row_j) row_j[:C]."""
+    _require_cuda(queries, cache, block_table, tok_pos, tok_seq, out)
+    n, width = queries.shape[0], rank + rot
+    if tuple(queries.shape) != (n, n_heads * width) or not queries.is_contiguous():
+        raise KernelError(f"latent_attention: queries {tuple(queries.shape)} are not contiguous [T, {n_heads} * {width}]")
+    if tuple(cache.shape[1:]) != (1, PAGE, width) or cache.dtype != queries.dtype or not cache.is_contiguous():
+        raise KernelError(f"latent_attention: the cache {tuple(cache.shape)} does not hold rows of {width}")
+    _check_out(out, (n, n_heads * rank), queries.dtype, "latent_attention")
+    variant = tactics.choose_latent_attention(decode, queries.dtype, n_heads, 0, 0, rank, rot)
+    if variant == "latent_generic" or cu_seqlens is None or seq_lens is None:
+        _call("attention_generic", "llmb_attention_generic", _ptr(queries), _c_int(queries.stride(0)), _ptr(cache), _ptr(cache),
+              _ptr(block_table), _c_int(block_table.shape[1]), _c_int(ring_pages), _ptr(tok_pos), _ptr(tok_seq), _ptr(out),
+              _c_int(out.stride(0)), _c_int(_code(queries.dtype)), _c_int(n), _c_int(n_heads), _c_int(1), _c_int(width),
+              _c_float(scale), _c_int(0), None, None, _c_int(0), _c_float(1.0), _c_float(0.0), _c_int(rank), _stream())
+        return out
+    splits, scratch = 1, None
+    if decode:
+        splits = latent_decode_splits(n, n_heads, max_len, _latent_pairs_fit(rank, rot, n_heads))
+        need = n * n_heads * splits * (rank + 2) if splits > 1 else 0
+        scratch = _attention_scratch.get(queries.device)
+        if scratch is None or scratch.numel() < need:
+            if scratch is not None:
+                global _scratch_generation
+                _retired.append(scratch)
+                _scratch_generation += 1
+            scratch = torch.empty(max(need, 1 << 23), dtype=torch.float32, device=queries.device)
+            _attention_scratch[queries.device] = scratch
+    _call("latent_attention", "llmb_latent_attention", _ptr(queries), _ptr(cache), _ptr(block_table), _c_int(block_table.shape[1]),
+          _c_int(ring_pages), _ptr(cu_seqlens), _ptr(seq_lens), _ptr(seq_order), _ptr(out), _ptr(scratch),
+          ctypes.c_longlong(scratch.numel() if scratch is not None else 0), _c_int(n), _c_int(cu_seqlens.numel() - 1),
+          _c_int(1 if decode else max_new), _c_int(n_heads), _c_int(rank), _c_int(rot), _c_float(scale), _c_int(splits), _stream(),
+          kernels=2 if splits > 1 else 1)
+    return out
+
+
+def latent_prefill(proj, kv, dense, n_heads, dim, rot, vdim, rank, scale, out, cu_seqlens, max_new, seq_order=None):
+    """Causal softmax attention of packed prompts that all start at their first token, with the keys and values of every
+    head formed: head h's queries are columns h (D + R).. of `proj` (rotated), its keys [D columns h (D + V).. of `kv` | the
+    last R columns of `dense` [T, C + R]], its values the V columns behind them in `kv`. Result [T, H V] into `out`."""
+    _require_cuda(proj, kv, dense, out, cu_seqlens)
+    n = proj.shape[0]
+    if tuple(kv.shape) != (n, n_heads * (dim + vdim)) or tuple(dense.shape) != (n, rank + rot) or not kv.is_contiguous() \
+            or not dense.is_contiguous() or proj.stride(1) != 1 or proj.shape[1] < n_heads * (dim + rot):
+        raise KernelError("latent_prefill: the operands do not fit the sizes")
+    _check_rows(out, n, n_heads * vdim, proj.dtype, "latent_prefill: out")
+    _call("latent_prefill_tc", "llmb_latent_prefill_tc", _ptr(proj), _c_int(proj.stride(0)), _ptr(kv), _ptr(dense), _c_int(n),
+          _ptr(cu_seqlens), _ptr(seq_order), _ptr(out), _c_int(out.stride(0)), _c_int(cu_seqlens.numel() - 1), _c_int(max_new),
+          _c_int(n_heads), _c_int(dim), _c_int(rot), _c_int(vdim), _c_int(rank), _c_float(scale), _stream())
+    return out
+
+
 def sigmoid_decode_splits(n_seqs: int, max_len: int, window: int, mixed_width: int = 1024) -> int:
     """Slices of the decode kernel of the sigmoid attention (a block serves all heads of a sequence):
     `decode_splits` for the keys a query sees at most. Two blocks share an SM where the mixed queries are
@@ -1400,6 +1640,7 @@ def required_libraries() -> list:
 
 __all__ = ["PAGE", "GLU_BLOCK", "glu_fusable", "embed", "scale_", "random_normal_", "begin_recording", "end_recording", "RecordedPass", "scratch_generation", "Emit", "FoldedNorm", "RopeWrite", "cast_sumsq", "SUMSQ_LD", "rmsnorm", "swiglu", "rope_cache_write", "linear", "attention",
            "softcap_", "add_rows_", "conv_rope_cache_write", "diff_attention", "tanh_norm", "norm_rope_cache_write",
-           "sigmoid_attention", "gated_recurrence", "state_space", "attention_replay_key", "attention_decode_splits", "sigmoid_attention_replay_key", "sigmoid_decode_splits",
+           "sigmoid_attention", "gated_recurrence", "state_space", "attention_replay_key", "layernorm", "input_conv", "output_norm_add_", "forget_recurrence",
+           "latent_write", "head_products", "latent_attention", "latent_prefill", "attention_decode_splits", "sigmoid_attention_replay_key", "sigmoid_decode_splits",
            "argmax_rows", "sample_rows", "launch_count", "count_launches", "tensor_core_status", "check_device_status", "ensure_built", "load_library", "all_sources",
            "required_libraries", "tactics"]

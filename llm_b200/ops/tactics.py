@@ -21,7 +21,7 @@ import torch
 
 from .. import native
 
-_FAMILY = {"linear": 0, "attention": 1, "diff_attention": 2, "sigmoid_attention": 3}
+_FAMILY = {"linear": 0, "attention": 1, "diff_attention": 2, "sigmoid_attention": 3, "latent_attention": 4}
 
 
 @dataclass(frozen=True)
@@ -70,11 +70,11 @@ def is_disabled(name: str) -> bool:
 
 def _choose(family: str, m=0, n=0, k=0, lda=0, decode=False, n_heads=1, n_kv_heads=1, head_dim=0,
             window=0, packed=False, aligned=True, in_dtype=None, out_dtype=None, dtype=None, value_dim=0,
-            keep_first=0):
+            keep_first=0, kv_rank=0, rot_dim=0, fresh=False):
     bf16 = (in_dtype if in_dtype is not None else dtype) == torch.bfloat16
-    shape = (c_int * 14)(int(m), int(n), int(k), int(lda), int(bool(decode)), int(n_heads), int(n_kv_heads),
+    shape = (c_int * 17)(int(m), int(n), int(k), int(lda), int(bool(decode)), int(n_heads), int(n_kv_heads),
                          int(head_dim), int(window), int(bool(packed)), int(bf16), int(bool(aligned)),
-                         int(value_dim), int(keep_first))
+                         int(value_dim), int(keep_first), int(kv_rank), int(rot_dim), int(bool(fresh)))
     name, reasons = ctypes.create_string_buffer(64), ctypes.create_string_buffer(2048)
     native.check(native.lib().llmh_tactics_choose(_FAMILY[family], shape, name, 64, reasons, 2048))
     return name.value.decode(), reasons.value.decode()
@@ -123,6 +123,17 @@ def choose_sigmoid_attention(decode, dtype, n_heads, n_kv_heads, head_dim, value
         name = _chosen[key] = _choose("sigmoid_attention", decode=decode, dtype=dtype, n_heads=n_heads,
                                       n_kv_heads=n_kv_heads, head_dim=head_dim, value_dim=value_dim, window=window,
                                       packed=packed, aligned=aligned)[0]
+    return name
+
+
+def choose_latent_attention(decode, dtype, n_heads, head_dim, value_dim, kv_rank, rot_dim, fresh=False) -> str:
+    """The variant for an attention over cached latent rows of kv_rank + rot_dim elements; `fresh`: every sequence of
+    the pass starts at its first token."""
+    key = ("latent_attention", decode, dtype, n_heads, head_dim, value_dim, kv_rank, rot_dim, fresh)
+    name = _chosen.get(key)
+    if name is None:
+        name = _chosen[key] = _choose("latent_attention", decode=decode, dtype=dtype, n_heads=n_heads, head_dim=head_dim,
+                                      value_dim=value_dim, kv_rank=kv_rank, rot_dim=rot_dim, fresh=fresh)[0]
     return name
 
 

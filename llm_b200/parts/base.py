@@ -71,6 +71,8 @@ class Part:
     overwrites: bool = False
     #: rows of the result a token has when `fresh` (the block adds them in index order)
     result_terms: int = 1
+    #: 1 if, behind those rows, `fresh` leaves one more row a token [T, hidden] (a shared expert's), else 0
+    result_extra: int = 0
 
     def parameters(self) -> dict:
         """tensor name -> ParamSpec of everything this part binds."""
@@ -155,6 +157,11 @@ class PositionEncoding(Part):
 
 
 class Block(Part):
+    def state_request(self):
+        """A cache.StateRequest if the arrangement itself keeps fixed-size state per sequence (beside its
+        mixer's; read with `ctx.cache.block_state_view(entry)`), else None."""
+        return None
+
     def forward(self, x, ctx: StepContext, entry: int, cache_entry: int) -> None:
         """Run one layer on the residual stream x (float32 [T, hidden]) in place."""
         raise NotImplementedError

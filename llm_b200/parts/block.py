@@ -7,7 +7,7 @@ import torch
 
 from .. import ops
 from ..errors import Unsupported
-from .base import (Block, Part, build_feed_forward, build_mixer, build_norm, register_block)
+from .base import (Block, Part, build_feed_forward, build_mixer, build_norm, register_block, to_float32)
 
 # LLMB_NO_FUSION=1: every norm stays a kernel of its own (for comparisons)
 FOLD_NORMS = os.environ.get("LLMB_NO_FUSION", "0") in ("", "0")
@@ -347,6 +347,8 @@ class SandwichBlock(Block):
         for norm in (self.mixer_norm, self.mixer_post_norm, self.ffn_norm, self.ffn_post_norm):
             if norm is not None and not getattr(norm, "foldable", False):
                 raise Unsupported("a sandwich block needs RMS norms (a gain and an eps) on both sides of its parts")
+        if self.feed_forward is not None and self.feed_forward.result_extra:
+            raise Unsupported("a sandwich block adds a token's result rows in one run: no row of its own behind them")
 
     @property
     def parts(self):
@@ -485,3 +487,203 @@ class SandwichBlock(Block):
 
 
 register_block("sandwich", SandwichBlock)
+
+
+class OutputNormBlock(Block):
+    """x += norm(mixer(c1(x))); x += norm'(feed_forward(c2(x))): norms on the parts' results only, and in front of a
+    part, instead of a norm, a short causal convolution over time of the stream itself, c(x) = x + conv(x) (or x
+    as it is, without taps). A part's result is a stream of its own (32-bit, `y`; possibly several rows a token) that
+    is normed before it joins x. The norm is a layer norm or an RMS norm.
+
+    The convolution reads the 32-bit stream; its last taps - 1 inputs are state of the block, kept per run and slot
+    for both parts ([2, taps - 1, size], 32-bit: ctx.cache.block_state_view). Launches beside the parts': in a step of one
+    token a sequence ONE kernel behind each part norms the result, adds it to x, convolves the new x for the part that runs
+    next and shifts that part's inputs (behind the last part: for the block that runs next, which asks for it through
+    `input_emit`); in other steps the norm with the sum (ops.output_norm_add_) and the convolution (ops.input_conv)
+    are a launch each, because a token's convolution reads rows that other blocks of the first kernel write."""
+
+    chains_norms = True
+    emit_has_state = True
+
+    def __init__(self, spec):
+        self.spec = spec
+        self.mixer = build_mixer(spec.mixer)
+        self.mixer_norm = build_norm(spec.mixer_norm)
+        self.feed_forward = build_feed_forward(spec.feed_forward) if spec.feed_forward is not None else None
+        self.ffn_norm = build_norm(spec.ffn_norm) if self.feed_forward is not None else None
+        for norm in (self.mixer_norm, self.ffn_norm):
+            if norm is not None and norm.spec.kind not in ops.OUTPUT_NORMS:
+                raise Unsupported(f"an output norm of kind '{norm.spec.kind}' (built: {', '.join(ops.OUTPUT_NORMS)})")
+        if spec.conv_taps < 0:
+            raise Unsupported("a convolution of the stream with a negative number of taps")
+        self.conv = [None, None]           # taps of the two parts as [taps, size]
+
+    @property
+    def size(self):
+        return self.spec.mixer_norm.size
+
+    @property
+    def parts(self):
+        return tuple(p for p in (self.mixer, self.mixer_norm, self.feed_forward, self.ffn_norm) if p is not None)
+
+    @property
+    def graph_safe(self):
+        return all(p.graph_safe for p in self.parts)
+
+    @property
+    def libraries(self):
+        return ("output_norm", "post_norm") + tuple(lib for p in self.parts for lib in p.libraries)
+
+    def _conv_names(self):
+        s = self.spec
+        return [s.mixer_conv, s.ffn_conv if self.feed_forward is not None else None] if s.conv_taps else [None, None]
+
+    def parameters(self):
+        from ..weights.loader import ParamSpec
+        out = {}
+        for p in self.parts:
+            out.update(p.parameters())
+        for name in self._conv_names():
+            if name is not None:
+                out[name] = ParamSpec((self.size, self.spec.conv_taps), "taps")
+        return out
+
+    def bind(self, tensors, dtype, device):
+        for p in self.parts:
+            p.bind(tensors, dtype, device)
+        self.conv = [to_float32(tensors[name], device).t().contiguous() if name is not None else None
+                     for name in self._conv_names()]
+
+    def state_request(self):
+        from ..cache import StateRequest
+        if self.spec.conv_taps > 1:
+            return StateRequest((2, self.spec.conv_taps - 1, self.size), torch.float32)
+        return None
+
+    def replay_key(self, step):
+        keys = [p.replay_key(step) for p in self.parts]
+        return None if any(k is None for k in keys) else (bool(step.decode), max(step.new_counts), tuple(keys))
+
+    def prepare(self, max_positions, device):
+        for p in self.parts:
+            p.prepare(max_positions, device)
+
+    def weights(self):
+        return [w for p in self.parts for w in p.weights()] + [c for c in self.conv if c is not None]
+
+    def kernel_shapes(self, dtype, token_counts):
+        return [shape for p in self.parts for shape in p.kernel_shapes(dtype, token_counts)]
+
+    def _state(self, ctx, entry, which):
+        """The last taps - 1 inputs of part `which`'s convolution, [slots, taps - 1, size]."""
+        return ctx.cache.block_state_view(entry)[:, which] if self.spec.conv_taps > 1 else None
+
+    class _Input:
+        """Where the kernel that last updates x leaves a part's input: rows (run dtype), the convolution's taps
+        and its state (this run's), filled or not."""
+        __slots__ = ("rows", "taps", "state", "filled")
+
+        def __init__(self, rows, taps, state):
+            self.rows, self.taps, self.state, self.filled = rows, taps, state, False
+
+    @staticmethod
+    def accepts_emit(emit) -> bool:
+        return isinstance(emit, OutputNormBlock._Input)
+
+    def input_emit(self, ctx, n_tokens: int, device, entry: int):
+        """Steps of one token a sequence: the block before leaves this block's first input (and shifts its state)."""
+        return self._input(ctx, 0, n_tokens, entry) if ctx.decode else None
+
+    def _input(self, ctx, which, n, entry):
+        name = ("h_first", "h_ffn")[which]
+        rows = ctx.scratch(name, (n, self.size), ctx.dtype)
+        if rows is None:
+            rows = torch.empty((n, self.size), dtype=ctx.dtype, device=ctx.device)
+        return OutputNormBlock._Input(rows, self.conv[which], self._state(ctx, entry, which))
+
+    @staticmethod
+    def _rows(part) -> int:
+        return int(part.result_terms) + int(part.result_extra)
+
+    def scratch_requests(self, n_tokens, dtype):
+        """h_first lives through the whole layer (in decode steps this layer's last kernel writes the next layer's
+        into it; the mixer has read it by then); y takes a part's result rows."""
+        from ..engine.workspace import BufferRequest
+        mixer = self.mixer.scratch_requests(n_tokens, dtype)
+        ffn = self.feed_forward.scratch_requests(n_tokens, dtype) if self.feed_forward is not None else []
+        mixer_end = 1 + max([r.last_use for r in mixer] + [0])
+        ffn_start = mixer_end + 2
+        ffn_end = ffn_start + max([r.last_use for r in ffn] + [0])
+        rows = max(self._rows(self.mixer), self._rows(self.feed_forward) if self.feed_forward is not None else 1)
+        out = [BufferRequest("h_first", (n_tokens, self.size), dtype, 0, ffn_end + 2),
+               BufferRequest("y_part", (n_tokens * rows, self.size), torch.float32, 0, ffn_end + 1)]
+        out += [r.shifted(1, "mixer.") for r in mixer]
+        if self.feed_forward is not None:
+            out.append(BufferRequest("h_ffn", (n_tokens, self.size), dtype, mixer_end + 1, ffn_end))
+            out += [r.shifted(ffn_start, "ffn.") for r in ffn]
+        return out
+
+    def _result(self, ctx, part, n, device):
+        """(buffer, fresh): where the part's result goes; zeroed where the part adds instead of writing."""
+        rows = self._rows(part) if part.overwrites else 1
+        y = ctx.scratch("y_part", (n * rows, self.size), torch.float32)
+        if y is None:
+            y = torch.empty((n * rows, self.size), dtype=torch.float32, device=device)
+        if not part.overwrites:
+            ops.fill_(y, 0.0)
+        return y, bool(part.overwrites)
+
+    def _filled(self, ctx, x, target):
+        """The part's input by a launch of its own."""
+        ops.input_conv(x, target.taps, target.state, ctx.cu_seqlens, ctx.slot_ids, target.rows, max(ctx.new_counts))
+        target.filled = True
+        return target.rows
+
+    def _join(self, ctx, x, y, part, norm, following):
+        """x += norm(result); where `following` is given, also the next part's input."""
+        terms, extra = (int(part.result_terms), int(part.result_extra)) if part.overwrites else (1, 0)
+        n = x.shape[0]
+        ops.output_norm_add_(x, y[:n * terms], norm.gain, norm.spec.eps, norm.spec.kind, terms,
+                             extra=y[n * terms:n * (terms + 1)] if extra else None,
+                             conv=None if following is None else (following.taps, following.state, ctx.slot_ids, following.rows))
+        if following is not None:
+            following.filled = True
+
+    def forward(self, x, ctx, entry, cache_entry, normed=None, emit_next=None):
+        """`normed`: this block's first input as the block before left it (a filled _Input), or None.
+        `emit_next`: where this block's last kernel leaves the next block's (an _Input, or None)."""
+        views = ctx.workspace
+        n = x.shape[0]
+
+        def prefixed(prefix):
+            if views is not None:
+                views.prefix = prefix
+
+        if isinstance(normed, OutputNormBlock._Input) and normed.filled:
+            h = normed.rows
+        else:
+            h = self._filled(ctx, x, self._input(ctx, 0, n, entry))
+        y, fresh = self._result(ctx, self.mixer, n, x.device)
+        prefixed("mixer.")
+        if fresh:
+            self.mixer.forward(h, ctx, entry, cache_entry, y, fresh=True)
+        else:
+            self.mixer.forward(h, ctx, entry, cache_entry, y)
+        prefixed("")
+        if self.feed_forward is None:
+            self._join(ctx, x, y, self.mixer, self.mixer_norm, emit_next)
+            return
+        target = self._input(ctx, 1, n, entry)
+        self._join(ctx, x, y, self.mixer, self.mixer_norm, target if ctx.decode else None)
+        h = target.rows if target.filled else self._filled(ctx, x, target)
+        y, fresh = self._result(ctx, self.feed_forward, n, x.device)
+        prefixed("ffn.")
+        if fresh:
+            self.feed_forward.forward(h, ctx, y, fresh=True)
+        else:
+            self.feed_forward.forward(h, ctx, y)
+        prefixed("")
+        self._join(ctx, x, y, self.feed_forward, self.ffn_norm, emit_next)
+
+
+register_block("output_norm", OutputNormBlock)

@@ -10,17 +10,19 @@ from .base import FeedForward, register_feed_forward, to_run_dtype
 
 
 class GatedMlp(FeedForward):
-    """down(silu(gate h) * (up h)) added to the residual stream, gate and up as
-    one matrix product (apps/engine/src/model.rs:1180-1216 of MythEclipse/llm)."""
+    """down(act(gate h) * (up h)) added to the residual stream, gate and up as
+    one matrix product (apps/engine/src/model.rs:1180-1216 of MythEclipse/llm); act is silu or the
+    tanh form of gelu, in either case in the product's epilogue where that takes it."""
     graph_safe = True
     emits = True
     overwrites = True
     libraries = ("elementwise", "gemm_simt", "gemm_skinny", "gemm_tc")
 
     def __init__(self, spec):
-        if spec.activation != "silu":
-            raise Unsupported(f"activation '{spec.activation}' in a gated feed-forward")
+        if spec.activation not in ("silu", "gelu_tanh"):
+            raise Unsupported(f"activation '{spec.activation}' in a gated feed-forward (built: 'silu', 'gelu_tanh')")
         self.spec = spec
+        self.gelu = spec.activation == "gelu_tanh"
         self.w_gate_up = self.w_down = None
         self.fused = False
 
@@ -80,10 +82,11 @@ class GatedMlp(FeedForward):
             h = norm.rows
         n, width = h.shape[0], self.spec.intermediate
         if self.fused:
-            act = ops.linear(h, self.w_gate_up, glu=True, out=ctx.scratch("act", (n, width), h.dtype), norm=norm)
+            act = ops.linear(h, self.w_gate_up, glu="gelu" if self.gelu else True,
+                             out=ctx.scratch("act", (n, width), h.dtype), norm=norm)
         else:
             gate_up = ops.linear(h, self.w_gate_up, out=ctx.scratch("gate_up", (n, 2 * width), h.dtype), norm=norm)
-            act = ops.swiglu(gate_up, out=ctx.scratch("act", (n, width), h.dtype))
+            act = ops.swiglu(gate_up, out=ctx.scratch("act", (n, width), h.dtype), gelu=self.gelu)
         if fresh:
             ops.linear(act, self.w_down, out_dtype=torch.float32, out=residual)
         else:

@@ -26,7 +26,7 @@ class GatedAttentionMixer(ProjectedMixer):
     The spec's switches (all off by default) ride in the same launches: `head_norm` in the launch that rotates
     (per-head RMS norms of queries and keys with weights the heads share), `value_mix` there too (the values are
     blended with those the first layer of the same name cached for the same token, before they are cached),
-    `head_gate` (one gate per head), `softcap`, `unit_sink` and `out_scale` inside the attention kernels. Values
+    `head_gate` (one gate per head), `softcap`, `unit_sink`, `sink` and `out_scale` inside the attention kernels. Values
     may be wider or narrower than keys (the cache keeps a tensor for each; the kernel for any sizes runs)."""
     libraries = ("elementwise", "gemm_simt", "gemm_skinny", "gemm_tc", "projection_norm", "post_norm",
                  "attention_generic", "attention_decode", "attention_decode_window", "attention_prefill",
@@ -42,6 +42,8 @@ class GatedAttentionMixer(ProjectedMixer):
             raise FormatError("a gated attention has a gate per element or a gate per head, not both")
         if s.value_mix is not None and s.values_are_keys:
             raise FormatError("values that are the keys cannot be blended with another layer's")
+        if s.sink and s.unit_sink:
+            raise FormatError("a softmax has a learned sink per head or a one in its denominator, not both")
         self.spec = spec
         self.position = build_position(spec.position)
         self.q_gain = self.k_gain = self.sinks = None
@@ -88,6 +90,8 @@ class GatedAttentionMixer(ProjectedMixer):
         if s.head_norm:
             out[t["q_norm"]] = ParamSpec((s.head_dim,), "gain")
             out[t["k_norm"]] = ParamSpec((s.head_dim,), "gain")
+        if s.sink:
+            out[t["sink"]] = ParamSpec((s.n_heads,), "vector")
         if s.value_mix is not None:
             out[t["value_mix"]] = ParamSpec((), "gate_scalar")         # (stored, but unused, in the first such layer too)
         return out
@@ -105,6 +109,8 @@ class GatedAttentionMixer(ProjectedMixer):
             self.k_gain = to_float32(tensors[t["k_norm"]], device)
         if s.value_mix is not None:
             self.mix_weight = float(tensors[t["value_mix"]].float())
+        if s.sink:
+            self.sinks = to_float32(tensors[t["sink"]], device)
         if s.unit_sink:
             self.sinks = torch.zeros(s.n_heads, dtype=torch.float32, device=device)
 

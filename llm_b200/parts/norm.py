@@ -1,4 +1,4 @@
-"""Norms: RMSNorm, and the element-wise tanh norm."""
+"""Norms: RMSNorm, layer norm, and the element-wise tanh norm."""
 from __future__ import annotations
 
 import torch
@@ -38,6 +38,32 @@ class RmsNorm(Norm):
 
 
 register_norm("rmsnorm", RmsNorm)
+
+
+class LayerNorm(Norm):
+    """(x - mean) / sqrt(mean squared deviation + eps) * weight, without a bias. The weight is held in 32-bit."""
+    graph_safe = True
+    libraries = ("output_norm",)
+    foldable = False
+
+    def __init__(self, spec):
+        self.spec = spec
+        self.gain = None
+
+    def parameters(self):
+        return {self.spec.weight: ParamSpec((self.spec.size,), "gain")}
+
+    def bind(self, tensors, dtype, device):
+        self.gain = to_float32(tensors[self.spec.weight], device)
+
+    def replay_key(self, step):
+        return ()
+
+    def forward(self, x, out_dtype, rows=None, out=None):
+        return ops.layernorm(x, self.gain, self.spec.eps, out_dtype, rows, out=out)
+
+
+register_norm("layernorm", LayerNorm)
 
 
 class TanhNorm(Norm):

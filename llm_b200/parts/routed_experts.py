@@ -6,7 +6,7 @@ import torch
 from .. import ops
 from ..errors import FormatError, Unsupported
 from ..weights.loader import ParamSpec
-from .base import FeedForward, register_feed_forward, to_float32, to_run_dtype
+from .base import FeedForward, build_feed_forward, register_feed_forward, to_float32, to_run_dtype
 
 
 class RoutedExperts(FeedForward):
@@ -26,10 +26,14 @@ class RoutedExperts(FeedForward):
     plus a stored correction, and the weights are the chosen scores over their sum; with `pass_through` the
     router's last outputs stand for experts without matrices that hand their input through; `out_scale`
     multiplies the weights. All of it is the router kernel's work (and one small launch for the rows handed
-    through): the plan and the grouped products see the assignments of experts with matrices only."""
+    through): the plan and the grouped products see the assignments of experts with matrices only.
+
+    `scoring` 'sigmoid' weights the chosen experts by their scores sigmoid(z) as they are; `weight_on_input` puts
+    the weight on the expert's input, where the epilogue of the gate and up product applies it to its 32-bit sums
+    (W (w h) = w W h) and the down product leaves its rows unweighted. `shared`: a feed-forward of its own for every
+    token, one more row a token behind the experts' (`result_extra`) or added into the residual."""
     graph_safe = True
     overwrites = True
-    libraries = ("routed_experts", "post_norm")
 
     def __init__(self, spec):
         s = spec
@@ -37,16 +41,27 @@ class RoutedExperts(FeedForward):
             raise Unsupported(f"activation '{s.activation}' in routed experts")
         if min(s.hidden, s.intermediate, s.n_experts, s.top) < 1 or s.pass_through < 0 or s.top > s.n_experts + s.pass_through:
             raise FormatError(f"{s.top} of {s.n_experts + max(s.pass_through, 0)} experts cannot be chosen")
-        if s.scoring not in ("chosen", "all"):
-            raise Unsupported(f"scoring '{s.scoring}' in routed experts (built: 'chosen', 'all')")
+        if s.scoring not in ops.ROUTER_SCORING:
+            raise Unsupported(f"scoring '{s.scoring}' in routed experts (built: {', '.join(ops.ROUTER_SCORING)})")
         if s.correction and s.scoring != "all":
             raise Unsupported("a correction of the choice needs scores over all experts")
+        if s.weight_on_input and s.pass_through:
+            raise Unsupported("experts that hand their input through with the weight on the input")
         self.spec = spec
+        self.shared = build_feed_forward(s.shared) if s.shared is not None else None
         self.router = self.router_bias = self.correction = self.w_up = self.w_down = None
+
+    @property
+    def libraries(self):
+        return ("routed_experts", "post_norm") + (tuple(self.shared.libraries) if self.shared is not None else ())
 
     @property
     def result_terms(self):
         return self.spec.top
+
+    @property
+    def result_extra(self):
+        return 1 if self.shared is not None else 0
 
     def parameters(self):
         s, t = self.spec, self.spec.tensor
@@ -61,6 +76,8 @@ class RoutedExperts(FeedForward):
             out[names["gate"]] = ParamSpec((s.intermediate, s.hidden))
             out[names["up"]] = ParamSpec((s.intermediate, s.hidden))
             out[names["down"]] = ParamSpec((s.hidden, s.intermediate))
+        if self.shared is not None:
+            out.update(self.shared.parameters())
         return out
 
     def bind(self, tensors, dtype, device):
@@ -76,10 +93,15 @@ class RoutedExperts(FeedForward):
             downs.append(to_run_dtype(tensors[names["down"]], dtype, device))
         self.w_up = torch.stack(ups).contiguous()                      # [E, 2 F, hidden]
         self.w_down = torch.stack(downs).contiguous()                  # [E, hidden, F]
+        if self.shared is not None:
+            self.shared.bind(tensors, dtype, device)
 
     def weights(self):
         """A decode step reads the router and, per token, `top` experts (counted as if all differed)."""
-        return [self.router]
+        return [self.router] + (self.shared.weights() if self.shared is not None else [])
+
+    def kernel_shapes(self, dtype, token_counts):
+        return self.shared.kernel_shapes(dtype, token_counts) if self.shared is not None else []
 
     def replay_key(self, step):
         return ()
@@ -95,6 +117,8 @@ class RoutedExperts(FeedForward):
                BufferRequest("expert_rows", (a, s.hidden), torch.float32, 0, 0)]
         if ops.routed_experts_wide(n_tokens, s.top, s.n_experts, s.hidden, s.intermediate, dtype):
             out.append(BufferRequest("expert_in", (a, s.hidden), dtype, 0, 0))       # the rows of h in the plan's order
+        if self.shared is not None:                                                      # runs behind the experts
+            out += [r.shifted(1, "shared.") for r in self.shared.scratch_requests(n_tokens, dtype)]
         return out
 
     def forward(self, h, ctx, residual, fresh=False):
@@ -113,10 +137,21 @@ class RoutedExperts(FeedForward):
         wide = ops.routed_experts_wide(n, s.top, s.n_experts, s.hidden, s.intermediate, h.dtype)
         gathered = buffer("expert_in", (a, s.hidden), h.dtype) if wide else None
         ops.routed_experts(h, self.router, self.router_bias, self.w_up, self.w_down, s.top, ids, weights, order, plan,
-                           act, rows, gathered, scoring=1 if s.scoring == "all" else 0, correction=self.correction,
-                           pass_through=s.pass_through, weight_scale=s.out_scale)
+                           act, rows, gathered, scoring=ops.ROUTER_SCORING.index(s.scoring), correction=self.correction,
+                           pass_through=s.pass_through, weight_scale=s.out_scale, weight_on_input=s.weight_on_input)
         if not fresh:
             ops.add_terms_(residual, rows, s.top)
+        if self.shared is None:
+            return
+        views, prefix = ctx.workspace, None
+        if views is not None:
+            prefix, views.prefix = views.prefix, views.prefix + "shared."
+        if fresh:
+            self.shared.forward(h, ctx, residual[a:], fresh=True)
+        else:
+            self.shared.forward(h, ctx, residual)
+        if views is not None:
+            views.prefix = prefix
 
 
 register_feed_forward("routed_experts", RoutedExperts)

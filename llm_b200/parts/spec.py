@@ -36,6 +36,15 @@ class TanhNormSpec:
 
 
 @dataclass(frozen=True)
+class LayerNormSpec:
+    """(x - mean) / sqrt(mean squared deviation + eps) * weight; no bias."""
+    size: int
+    eps: float
+    weight: str                      # tensor name
+    kind: str = "layernorm"
+
+
+@dataclass(frozen=True)
 class PositionSpec:
     """Rotary encoding: angle = position * inv_freq[pair]."""
     head_dim: int
@@ -122,6 +131,29 @@ class LatentAttentionSpec:
 
 
 @dataclass(frozen=True)
+class RotaryLatentSpec:
+    """Attention over one cached latent row per position with a rotated key part that all heads share. A query head
+    is [head_dim unrotated | rot_dim rotated] elements of W_q h; W_dkv h is [kv_rank | rot_dim]: the first part,
+    RMS-normed (eps), is the latent c, the second the shared rotated key part. Head a's key is [W_uk,a c | shared part],
+    its value W_uv,a c. Only c and the rotated part are cached."""
+    hidden: int
+    n_heads: int
+    head_dim: int                    # unrotated query / key elements of a head
+    rot_dim: int                     # rotated ones
+    value_dim: int
+    kv_rank: int                     # size of the latent
+    scale: float                     # multiplies q.k
+    eps: float                       # of the latent's norm
+    position: Optional[PositionSpec] # of the rotated part (head_dim == rot_dim there)
+    names: tuple                     # sorted (role, tensor name): q, dkv, dkv_norm, uk, uv, o
+    kind: str = "rotary_latent_attention"
+
+    @property
+    def tensor(self):
+        return dict(self.names)
+
+
+@dataclass(frozen=True)
 class SigmoidAttentionSpec:
     """Grouped-query attention without a softmax: the weight of a visible key is
     sigmoid(score + bias[head]), not normalised over the keys. Before that, optionally, the heads'
@@ -181,7 +213,8 @@ class GatedAttentionSpec:
     own root mean square over head_dim (eps `norm_eps`) and multiplied by a weight of head_dim elements that the
     heads share, before the rotation); `head_gate` (one gate number per head, sigmoid(W_g h)[head] with W_g
     [n_heads, hidden], instead of one per element); `softcap` (c > 0: score <- c tanh(score / c) behind the
-    scale); `unit_sink` (the softmax's denominator holds one more term e^0 that has no value);
+    scale); `unit_sink` (the softmax's denominator holds one more term e^0 that has no value); `sink` (one more term
+    e^sink[head] with a learned number per head, role `sink`, that has neither key nor value and is not scaled);
     `value_mix` (a name shared by the layers whose values are blended: in every such layer but the one with
     `value_mix_first`, v <- (1 - w) v + w v_first with w one stored number (role `value_mix`) and v_first the
     values that the first such layer computed for the same token; the blended values are what is cached);
@@ -206,6 +239,7 @@ class GatedAttentionSpec:
     value_mix: Optional[str] = None
     value_mix_first: bool = False
     out_scale: float = 1.0
+    sink: bool = False
 
     @property
     def tensor(self):
@@ -231,6 +265,26 @@ class DeltaRuleSpec:
     names: tuple                     # sorted (role, tensor name): q, k, v, q_conv, k_conv, v_conv, beta, decay, a_log, dt_bias, gate, norm, o
     unit_eps: float = 1e-6
     kind: str = "delta_rule"
+
+    @property
+    def tensor(self):
+        return dict(self.names)
+
+
+@dataclass(frozen=True)
+class ForgetRecurrenceSpec:
+    """Linear attention whose forget gate also decides what is written (Qin et al., "HGRN2: Gated Linear RNNs with
+    State Expansion"): q = silu(W_q h) (n_heads heads of head_dim), v = W_v h (n_heads heads of value_dim),
+    f = l + (1 - l) sigmoid(W_f h + b_f) per head and channel with a stored lower bound l; per head
+    S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T, o_t = S_t^T q_t; every head's o is divided by its root mean square (eps)
+    and multiplied by a weight of value_dim elements that the heads share, then W_o."""
+    hidden: int
+    n_heads: int
+    head_dim: int
+    value_dim: int
+    eps: float
+    names: tuple                     # sorted (role, tensor name): q, f, f_bias, lower, v, norm, o
+    kind: str = "forget_recurrence"
 
     @property
     def tensor(self):
@@ -274,7 +328,7 @@ class SideBySideSpec:
 class GatedMlpSpec:
     hidden: int
     intermediate: int
-    activation: str                  # 'silu'
+    activation: str                  # 'silu' or 'gelu_tanh' (the tanh form of gelu)
     names: tuple                     # sorted (role, tensor name): gate, up, down
     kind: str = "gated_mlp"
 
@@ -308,7 +362,11 @@ class RoutedExpertsSpec:
     (`correction`: a stored vector that takes part in the choice only) are chosen, and the weights are the
     chosen scores divided by their sum (+ 1e-20). `pass_through` > 0: the router has n_experts + pass_through
     outputs; the last ones are experts without tensors whose result is their input. `out_scale` multiplies
-    the result."""
+    the result.
+
+    `scoring` 'sigmoid': scores s = sigmoid(z), the `top` largest are chosen, and the weights are the chosen scores
+    as they are. `weight_on_input`: the weight multiplies the expert's input instead of its result, expert(w h).
+    `shared` (a GatedMlpSpec): one more feed-forward that every token passes, added to the result."""
     hidden: int
     intermediate: int
     n_experts: int
@@ -318,10 +376,12 @@ class RoutedExpertsSpec:
     expert_names: tuple              # sorted (role, pattern): gate, up, down
     activation: str = "silu"
     kind: str = "routed_experts"
-    scoring: str = "chosen"          # 'chosen': softmax over the chosen logits; 'all': see above
+    scoring: str = "chosen"          # 'chosen': softmax over the chosen logits; 'all', 'sigmoid': see above
     correction: bool = False
     pass_through: int = 0
     out_scale: float = 1.0
+    weight_on_input: bool = False
+    shared: Optional[GatedMlpSpec] = None
 
     @property
     def tensor(self):
@@ -342,6 +402,22 @@ class SandwichBlockSpec:
     feed_forward: object
     ffn_post_norm: object
     kind: str = "sandwich"
+
+
+@dataclass(frozen=True)
+class OutputNormBlockSpec:
+    """x += mixer_norm(mixer(c1(x))); x += ffn_norm(feed_forward(c2(x))): norms on the parts' results only. With
+    `conv_taps` > 0 a part reads c(x) = x + conv(x), a causal convolution over time on every channel of the stream
+    (`mixer_conv`, `ffn_conv`: tensors [size, conv_taps], the last column the current token's); without, x itself.
+    `feed_forward` (with its norm and convolution) may be None."""
+    mixer: object
+    mixer_norm: object
+    feed_forward: object
+    ffn_norm: object
+    conv_taps: int = 0
+    mixer_conv: Optional[str] = None
+    ffn_conv: Optional[str] = None
+    kind: str = "output_norm"
 
 
 @dataclass(frozen=True)

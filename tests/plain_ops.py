@@ -42,11 +42,17 @@ def rmsnorm(x, gain, eps, out_dtype, rows=None, out=None):
     return (x * scale * gain.to(torch.float32)).to(out_dtype)
 
 
-def swiglu(gate_up, out=None):
+def _activated(g, gelu):
+    if gelu:
+        return 0.5 * g * (1.0 + torch.tanh(0.7978845608028654 * (g + 0.044715 * g * g * g)))
+    return g / (1.0 + torch.exp(-g))
+
+
+def swiglu(gate_up, out=None, gelu=False):
     width = gate_up.shape[1] // 2
     g = gate_up[:, :width].to(torch.float32)
     u = gate_up[:, width:].to(torch.float32)
-    return (g / (1.0 + torch.exp(-g)) * u).to(gate_up.dtype)
+    return (_activated(g, gelu) * u).to(gate_up.dtype)
 
 
 def linear(a, w, bias=None, out_dtype=None, residual=None, out=None, glu=False, norm=None, emit=None,
@@ -69,7 +75,7 @@ def linear(a, w, bias=None, out_dtype=None, residual=None, out=None, glu=False, 
         m = product.shape[0]
         blocks = product.view(m, -1, 2, 16)
         g, u = blocks[:, :, 0, :].reshape(m, -1), blocks[:, :, 1, :].reshape(m, -1)
-        return (g / (1.0 + torch.exp(-g)) * u).to(a.dtype)
+        return (_activated(g, glu == "gelu") * u).to(a.dtype)
     if bias is not None:
         product = product + bias.to(torch.float32)
     if residual is not None:
@@ -379,11 +385,12 @@ def routed_experts_wide(n_tokens, top, n_experts, hidden, intermediate, dtype):
 
 
 def routed_experts(h, router, router_bias, w_up, w_down, top, ids, weights, order, plan, act, y, gathered=None,
-                   scoring=0, correction=None, pass_through=0, weight_scale=1.0):
+                   scoring=0, correction=None, pass_through=0, weight_scale=1.0, weight_on_input=False):
     """Token by token: 32-bit router logits, the `top` largest, the softmax over them, and one row
     weight * expert(h) per choice, in the order of choice (largest logit first). scoring 1: the scores are the
     softmax over all outputs, the choice is by score + correction, the weights are the chosen scores over
-    their sum (+ 1e-20). The router's last `pass_through` outputs are experts whose result is h."""
+    their sum (+ 1e-20). The router's last `pass_through` outputs are experts whose result is h. scoring 2: the weights are the
+    sigmoids of the chosen logits. weight_on_input: expert(weight h) in place of weight * expert(h)."""
     n, hidden = h.shape
     F = w_up.shape[1] // 2
     x = h.to(torch.float32)
@@ -397,6 +404,9 @@ def routed_experts(h, router, router_bias, w_up, w_down, top, ids, weights, orde
             choice = scores + correction if correction is not None else scores
             chosen = torch.sort(choice, descending=True, stable=True).indices[:top]
             share = scores[chosen] / (scores[chosen].sum() + 1e-20) * weight_scale
+        elif scoring == 2:
+            chosen = torch.sort(logits[t], descending=True, stable=True).indices[:top]
+            share = torch.sigmoid(logits[t, chosen]) * weight_scale
         else:
             chosen = torch.topk(logits[t], top).indices
             share = torch.softmax(logits[t, chosen], 0) * weight_scale
@@ -408,9 +418,11 @@ def routed_experts(h, router, router_bias, w_up, w_down, top, ids, weights, orde
                 y[t * top + k] = share[k] * x[t]
                 continue
             gate_up = x[t] @ w_up[e].to(torch.float32).T
+            if weight_on_input:
+                gate_up = gate_up * share[k]
             g, u = gate_up[:F], gate_up[F:]
             a = (g / (1.0 + torch.exp(-g)) * u).to(h.dtype).to(torch.float32)
-            y[t * top + k] = share[k] * (a @ w_down[e].to(torch.float32).T)
+            y[t * top + k] = (1.0 if weight_on_input else share[k]) * (a @ w_down[e].to(torch.float32).T)
     return y
 
 
@@ -461,6 +473,141 @@ def state_space(proj, taps, conv_bias, state, tok_seq, cu_seqlens, slot_ids, rat
         state[slot, (K - 1) * C:(K - 1) * C + H * N * V] = S.transpose(1, 2).reshape(-1)
     mixed.copy_(result.to(mixed.dtype))
     return mixed
+
+
+def layernorm(x, gain, eps, out_dtype, rows=None, out=None):
+    if rows is not None:
+        x = x[rows.long()]
+    d = x.to(torch.float32) - x.to(torch.float32).mean(dim=-1, keepdim=True)
+    result = (d / torch.sqrt((d * d).mean(dim=-1, keepdim=True) + eps) * gain).to(out_dtype)
+    if out is not None:
+        out.copy_(result)
+        return out
+    return result
+
+
+def input_conv(x, taps, state, cu_seqlens, slot_ids, out, max_new):
+    """Token by token: x plus the convolution over the sequence's last rows; the state moves on."""
+    K = taps.shape[0] if taps is not None else 0
+    for b in range(cu_seqlens.numel() - 1):
+        first, end = int(cu_seqlens[b]), int(cu_seqlens[b + 1])
+        past = [state[int(slot_ids[b]), r].clone() for r in range(K - 1)] if K > 1 else []
+        for t in range(first, end):
+            rows = past + [x[t]]
+            y = x[t].clone()
+            for j in range(K):
+                y = y + taps[j] * rows[j]
+            out[t] = y.to(out.dtype)
+            past = rows[1:] if K > 1 else []
+        for r in range(K - 1):
+            state[int(slot_ids[b]), r] = past[r]
+    return out
+
+
+def output_norm_add_(x, y, gain, eps, kind, terms=1, extra=None, conv=None):
+    n, width = x.shape
+    s = y.view(n, terms, width)[:, 0].clone()
+    for k in range(1, terms):                       # the terms in index order
+        s = s + y.view(n, terms, width)[:, k]
+    if extra is not None:
+        s = s + extra
+    if kind == "layernorm":
+        s = s - s.mean(dim=-1, keepdim=True)
+    x += s / torch.sqrt((s * s).mean(dim=-1, keepdim=True) + eps) * gain
+    if conv is not None:
+        taps, state, slot_ids, out = conv
+        input_conv(x, taps, state, torch.arange(n + 1), slot_ids, out, 1)
+    return x
+
+
+def forget_recurrence_work_width(n_heads, dim, vdim):
+    return (2 * n_heads * dim + n_heads * vdim + 3) // 4 * 4
+
+
+def forget_recurrence(proj, f_bias, lower, state, cu_seqlens, slot_ids, norm_weight, eps, work, o, mixed, n_heads, dim, vdim,
+                      single_tokens=False):
+    """Token by token and head by head; S lies in the state as [H, V, D]."""
+    H, D, V = n_heads, dim, vdim
+    u = proj.to(torch.float32)
+    n = u.shape[0]
+    q = u[:, :H * D]
+    q = (q / (1.0 + torch.exp(-q))).view(n, H, D)
+    f = (lower + (1.0 - lower) * torch.sigmoid(u[:, H * D:2 * H * D] + f_bias)).view(n, H, D)
+    v = u[:, 2 * H * D:2 * H * D + H * V].view(n, H, V)
+    for b in range(cu_seqlens.numel() - 1):
+        slot = int(slot_ids[b])
+        S = state[slot, :H * D * V].view(H, V, D).clone()
+        for t in range(int(cu_seqlens[b]), int(cu_seqlens[b + 1])):
+            S = f[t][:, None, :] * S + v[t][:, :, None] * (1.0 - f[t])[:, None, :]
+            r = (S * q[t][:, None, :]).sum(-1)
+            r = r / torch.sqrt((r * r).mean(-1, keepdim=True) + eps) * norm_weight
+            mixed[t] = r.reshape(-1).to(mixed.dtype)
+        state[slot, :H * D * V] = S.reshape(-1)
+    return mixed
+
+
+def latent_write(u, n_heads, dim, rot, rank, gain, eps, rope_table, interleaved, tok_pos, tok_seq, block_table, ring_pages,
+                 cache, queries=None, dense=None, write_cache=True):
+    n, qw = u.shape[0], n_heads * (dim + rot)
+    for t in range(n):
+        pos, b = int(tok_pos[t]), int(tok_seq[t])
+        row = u[t, qw:qw + rank + rot].to(torch.float32).clone()
+        c = row[:rank]
+        row[:rank] = c / torch.sqrt((c * c).mean() + eps) * gain
+        q = u[t, :qw].to(torch.float32).view(n_heads, dim + rot).clone()
+        if rope_table is not None:
+            n_rot = rope_table.shape[1]
+            cos, sin = rope_table[pos:pos + 1, :n_rot // 2], rope_table[pos:pos + 1, n_rot // 2:]
+            row[rank:rank + n_rot] = _rotate(row[None, None, rank:rank + n_rot], cos, sin, interleaved)[0, 0]
+            q[:, dim:dim + n_rot] = _rotate(q[None, :, dim:dim + n_rot], cos, sin, interleaved)[0]
+        if write_cache:
+            cache[int(block_table[b, (pos // PAGE) % ring_pages]), 0, pos % PAGE] = row.to(cache.dtype)
+        if dense is not None:
+            dense[t] = row.to(dense.dtype)
+        if queries is not None:
+            queries.view(n, n_heads, rank + rot)[t, :, rank:] = q[:, dim:].to(queries.dtype)
+        else:
+            u[t, :qw] = q.reshape(-1).to(u.dtype)
+
+
+def head_products(x, x_head, w, out, out_head):
+    H, N, K = w.shape
+    for h in range(H):
+        out[:, h * out_head:h * out_head + N] = (x[:, h * x_head:h * x_head + K].to(torch.float32)
+                                                 @ w[h].to(torch.float32).T).to(out.dtype)
+    return out
+
+
+def latent_attention_replay_key(step, n_heads):
+    return ()
+
+
+def latent_attention(queries, cache, block_table, ring_pages, tok_pos, tok_seq, n_heads, rank, rot, scale, out, decode=False,
+                     seq_lens=None, max_len=0, cu_seqlens=None, max_new=0, seq_order=None):
+    n, width = queries.shape[0], rank + rot
+    for t in range(n):
+        pos, b = int(tok_pos[t]), int(tok_seq[t])
+        js = torch.arange(pos + 1, device=queries.device)
+        rows = cache[block_table.long()[b, (js // PAGE) % ring_pages], 0, js % PAGE].to(torch.float32)
+        q = queries[t].to(torch.float32).view(n_heads, width)
+        p = torch.softmax((q @ rows.T) * scale, dim=-1)
+        out[t] = (p @ rows[:, :rank]).reshape(-1).to(out.dtype)
+    return out
+
+
+def latent_prefill(proj, kv, dense, n_heads, dim, rot, vdim, rank, scale, out, cu_seqlens, max_new, seq_order=None):
+    """Causal attention of packed prompts that start at their first token, keys and values of every head formed."""
+    for b in range(cu_seqlens.numel() - 1):
+        lo, hi = int(cu_seqlens[b]), int(cu_seqlens[b + 1])
+        q = proj[lo:hi, :n_heads * (dim + rot)].to(torch.float32).view(hi - lo, n_heads, dim + rot)
+        heads = kv[lo:hi].to(torch.float32).view(hi - lo, n_heads, dim + vdim)
+        shared = dense[lo:hi, rank:].to(torch.float32)
+        mask = torch.ones((hi - lo, hi - lo), dtype=torch.bool, device=proj.device).tril()
+        for h in range(n_heads):
+            s = (q[:, h, :dim] @ heads[:, h, :dim].T + q[:, h, dim:] @ shared.T) * scale
+            p = torch.softmax(s.masked_fill(~mask, float("-inf")), dim=-1)
+            out[lo:hi, h * vdim:(h + 1) * vdim] = (p @ heads[:, h, dim:]).to(out.dtype)
+    return out
 
 
 def softcap_(x, cap):
@@ -672,7 +819,11 @@ OPS = {"embed": embed, "scale_": scale_, "cast_sumsq": cast_sumsq, "rmsnorm": rm
        "add_terms_": add_terms_, "fill_": fill_, "delta_rule": delta_rule, "delta_rule_work_width": delta_rule_work_width,
        "routed_experts": routed_experts, "routed_experts_plan_ints": routed_experts_plan_ints,
        "routed_experts_wide": routed_experts_wide, "state_space": state_space,
-       "state_space_work_width": state_space_work_width}
+       "state_space_work_width": state_space_work_width, "layernorm": layernorm, "input_conv": input_conv,
+       "output_norm_add_": output_norm_add_, "forget_recurrence": forget_recurrence,
+       "forget_recurrence_work_width": forget_recurrence_work_width, "latent_write": latent_write,
+       "head_products": head_products, "latent_attention": latent_attention, "latent_prefill": latent_prefill,
+       "latent_attention_replay_key": latent_attention_replay_key}
 
 
 def install(monkeypatch):
