@@ -49,6 +49,7 @@
 //
 // The key block's keys beyond a query's own position are masked by value (-inf), so the
 // diagonal needs no special path; blocks wholly above the tile's diagonal are never loaded.
+// A sink (e^sink in a head's denominator, without a key) joins in the epilogue.
 // All waits are bounded by a clock limit and report through the status word of this library.
 #include "tc.cuh"
 
@@ -117,7 +118,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             int table_stride, int ring_pages, const int* __restrict__ cu_seqlens,
                             const int* __restrict__ seq_lens, const int* __restrict__ seq_order,
                             __nv_bfloat16* __restrict__ out, int out_stride,
-                            int n_heads, int n_kv_heads, float scale_log2, int* status) {
+                            int n_heads, int n_kv_heads, float scale_log2, const float* __restrict__ sinks, int* status) {
     constexpr int PIECES = HD / 64;
     constexpr int Q_BYTES = PIECES * Q_PIECE;         // the block's queries
     constexpr int KV_BYTES = PIECES * KV_PIECE;       // the K or the V of one key block
@@ -366,7 +367,14 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         if (ok) {
             __syncwarp();
             tcgen05_fence_after();
-            float inv = 1.0f / run_sum;
+            float inv;
+            if (sinks) {                                     // e^sink joins the denominator; the larger of both is the reference
+                float m = run_max * scale_log2, sink2 = sinks[head] * 1.4426950408889634f, r = fmaxf(m, sink2);
+                float w = fast_exp2(m - r);
+                inv = w / (run_sum * w + fast_exp2(sink2 - r));
+            } else {
+                inv = 1.0f / run_sum;
+            }
             __nv_bfloat16* o = out + (size_t)(first_token + q_index) * out_stride + (size_t)head * HD;
 #pragma unroll 1
             for (int c = 0; c < HD; c += 32) {
@@ -429,7 +437,7 @@ template <int HD>
 int launch(const CUtensorMap& map_q, const CUtensorMap& map_k, const CUtensorMap& map_v,
            const int* block_table, int table_stride, int ring_pages, const int* cu_seqlens,
            const int* seq_lens, const int* seq_order, void* out, int out_stride, int n_seqs, int max_new, int n_heads,
-           int n_kv_heads, float scale, cudaStream_t stream) {
+           int n_kv_heads, float scale, const float* sinks, cudaStream_t stream) {
     constexpr int Q_BYTES = (HD / 64) * Q_PIECE, KV_BYTES = (HD / 64) * KV_PIECE;
     // never less than 80 KB, so that no third block lands on an SM and waits for tensor memory
     size_t smem = 1024 + (size_t)Q_BYTES + 4 * KV_BYTES + 16 * 8 + 16;
@@ -445,20 +453,20 @@ int launch(const CUtensorMap& map_q, const CUtensorMap& map_k, const CUtensorMap
     dim3 grid(n_heads, (max_new + BQ - 1) / BQ, n_seqs);
     llmb::launch(attention_prefill_tc_kernel<HD>, grid, THREADS, smem, stream, true,
                  map_q, map_k, map_v, block_table, table_stride, ring_pages, cu_seqlens, seq_lens, seq_order,
-                 (__nv_bfloat16*)out, out_stride, n_heads, n_kv_heads, scale * 1.4426950408889634f, status_dev);
+                 (__nv_bfloat16*)out, out_stride, n_heads, n_kv_heads, scale * 1.4426950408889634f, sinks, status_dev);
     return check_launch("attention_prefill_tc");
 }
 }  // namespace
 
 // q: the fused projection of the new tokens [n_tokens, q_stride] (queries in its first columns);
 // k_cache, v_cache: one layer of the paged cache [n_pages, n_kv_heads, 64, head_dim]; the rest as in
-// llmb_attention_prefill. out must be 16-byte aligned with a row stride that is a multiple of 8.
+// llmb_attention_prefill; sinks float32 [n_heads] or null: e^sink is one more term of a head's softmax denominator. out must be 16-byte aligned with a row stride that is a multiple of 8.
 LLMB_EXPORT int llmb_attention_prefill_tc(const void* q, int q_stride, int n_tokens, const void* k_cache,
                                           const void* v_cache, int n_pages, const int* block_table,
                                           int table_stride, int ring_pages, const int* cu_seqlens,
                                           const int* seq_lens, const int* seq_order, void* out, int out_stride, int n_seqs,
                                           int max_new, int n_heads, int n_kv_heads, int head_dim,
-                                          float scale, int window, cudaStream_t stream) {
+                                          float scale, int window, const float* sinks, cudaStream_t stream) {
     if (n_seqs == 0 || max_new == 0) return LLMB_OK;
     int code = llmb_attention_prefill_tc_supports(n_heads, n_kv_heads, head_dim, window);
     if (code) return code;
@@ -474,9 +482,9 @@ LLMB_EXPORT int llmb_attention_prefill_tc(const void* q, int q_stride, int n_tok
     if ((code = make_map_2d(&map_v, v_cache, cache_rows, head_dim, head_dim, 64, LLMB_PAGE))) return code;
     if (head_dim == 64)
         return launch<64>(map_q, map_k, map_v, block_table, table_stride, ring_pages, cu_seqlens, seq_lens, seq_order, out,
-                          out_stride, n_seqs, max_new, n_heads, n_kv_heads, scale, stream);
+                          out_stride, n_seqs, max_new, n_heads, n_kv_heads, scale, sinks, stream);
     return launch<128>(map_q, map_k, map_v, block_table, table_stride, ring_pages, cu_seqlens, seq_lens, seq_order, out,
-                       out_stride, n_seqs, max_new, n_heads, n_kv_heads, scale, stream);
+                       out_stride, n_seqs, max_new, n_heads, n_kv_heads, scale, sinks, stream);
 }
 
 // the packed doors of the launching entry points (common.cuh)

@@ -176,6 +176,17 @@ std::string latent_tiles_guard(const Shape& s) {
     return "";
 }
 
+std::string latent_prefill_guard(const Shape& s) {
+    if (s.decode || !s.fresh) return "serves steps whose sequences all start at their first token";
+    if (!s.bf16) return "bfloat16 operands only";
+    if ((s.head_dim != 64 && s.head_dim != 128) || (s.value_dim != 64 && s.value_dim != 128))
+        return "unrotated part " + std::to_string(s.head_dim) + " with value size " + std::to_string(s.value_dim) + " (served: 64, 128)";
+    if (s.rot_dim > 64 || s.rot_dim % 8 || s.kv_rank % 8)
+        return "a rotated part of " + std::to_string(s.rot_dim) + " over a latent of " + std::to_string(s.kv_rank) +
+               " elements (served: up to 64; multiples of 8: TMA strides of 16 bytes)";
+    return "";
+}
+
 const std::vector<Row>& table(int family) {
     static const std::vector<Row> linear = {
         {"gemm_tc", 30, tc_guard,
@@ -240,6 +251,10 @@ const std::vector<Row>& table(int family) {
          "32-bit path"},
     };
     static const std::vector<Row> latent_attention = {
+        {"latent_prefill_tc", 20, latent_prefill_guard,
+         "prompts from their first token with the keys and values of every head formed by one product: flash attention "
+         "with both products on tcgen05, two tiles of 128 queries a block over shared key and value blocks by TMA, one "
+         "thread per query row"},
         {"latent_tiles", 10, latent_tiles_guard,
          "softmax attention of (token, head) pairs over the cached latent rows: all heads share a row, so a page goes "
          "into shared memory once for up to 64 pairs; mma.sync tiles, scores by (row, key) parts over eight warps, value "

@@ -25,7 +25,7 @@ from .build import all_sources, ensure_built, load_library
 
 PAGE = native.plan_constant("page")              # positions per cache page (csrc/plan.h)
 BFLOAT16_ONLY = ("gemm_tc", "gemm_skinny", "attention_decode", "attention_decode_window", "attention_prefill",
-                 "attention_prefill_tc")     # (diff_attention holds the 32-bit kernel too)
+                 "attention_prefill_tc", "latent_prefill_tc")     # (diff_attention holds the 32-bit kernel too)
 
 _DTYPE_CODE = {torch.float32: 0, torch.bfloat16: 1}
 _c_int, _c_float, _c_void = ctypes.c_int, ctypes.c_float, ctypes.c_void_p
@@ -1220,7 +1220,10 @@ def attention(qkv, k_cache, v_cache, block_table, ring_pages, tok_pos, tok_seq, 
     variant = tactics.choose_attention(decode, qkv.dtype, n_heads, n_kv_heads, head_dim, window,
                                        cu_seqlens is not None and seq_lens is not None,
                                        qkv.stride(0) % 8 == 0 and qkv.data_ptr() % 16 == 0)
-    if extras and variant not in _ATTENTION_WITH_EXTRAS:
+    # the tcgen05 prefill takes a sink, none of the others
+    sink_only = (sinks is not None and gate is None and out_scale == 1.0 and softcap <= 0.0 and value_dim == head_dim
+                 and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0)
+    if extras and variant not in _ATTENTION_WITH_EXTRAS and not (variant == "attention_prefill_tc" and sink_only):
         # the next choice that takes a sink, a gate, a scale and rows inside a wider buffer
         variant = "attention_generic"
         if not tactics.is_disabled("attention_prefill") and qkv.dtype == torch.bfloat16 and head_dim in (32, 64, 96, 128) \
@@ -1237,7 +1240,7 @@ def attention(qkv, k_cache, v_cache, block_table, ring_pages, tok_pos, tok_seq, 
               _c_int(block_table.shape[1]), _c_int(ring_pages), _ptr(cu_seqlens), _ptr(seq_lens),
               _ptr(seq_order), _ptr(out), _c_int(out.stride(0)), _c_int(cu_seqlens.numel() - 1),
               _c_int(max_new), _c_int(n_heads), _c_int(n_kv_heads), _c_int(head_dim), _c_float(scale),
-              _c_int(window), _stream())
+              _c_int(window), _ptr(sinks), _stream())
     elif variant == "attention_prefill":
         _call("attention_prefill", "llmb_attention_prefill", _ptr(qkv), _c_int(qkv.stride(0)),
               _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _c_int(block_table.shape[1]),

@@ -29,7 +29,8 @@ class RotaryLatentMixer(ProjectedMixer):
 
     Launches: the product [q; dkv], ops.latent_write (norm, rotations, cache write), then the form's own, then
     the output product."""
-    libraries = ("elementwise", "gemm_simt", "gemm_skinny", "gemm_tc", "latent_attention", "attention_generic")
+    libraries = ("elementwise", "gemm_simt", "gemm_skinny", "gemm_tc", "latent_attention", "latent_prefill_tc",
+                 "attention_generic")
 
     def __init__(self, spec):
         s = spec

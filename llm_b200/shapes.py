@@ -115,6 +115,33 @@ SHAPES["zemozen-8b"] = _zemozen(4096, 32, 8, 128, 14336, 128256, 32, 2048, 32, 2
 SHAPES["zemozen-1b"] = _zemozen(2048, 32, 8, 64, 8192, 128256, 16, 2048, 32, 2, 8)
 
 
+def _duvozen(width, heads, kv_heads, dim, ff, vocab, layers, latent, experts, top):
+    """A Duvozen configuration whose layers match a Llama shape in size (width, heads, head size, feed-forward,
+    vocabulary): a pattern of four layers, latent attention twice (the Llama shape's heads as the unrotated part; `latent` =
+    rotated part and cached latent), attention with sinks and gates, the forget-gated recurrence (states of head size x
+    head size), with dense and routed feed-forwards in turn; a routed layer's `top` chosen experts together are as wide
+    as the dense feed-forward, and a shared expert has an expert's width. Four taps."""
+    rot_dim, kv_rank = latent
+    base = {"heads": heads, "dim": dim, "vdim": dim}
+    latent_mixer = {**base, "rot_dim": rot_dim, "kv_rank": kv_rank, "scale": (dim + rot_dim) ** -0.5,
+                    "rot": {"base": 10000.0, "dims": rot_dim,
+                            "scaling": {"factor": 16.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    attention = {**base, "kv_heads": kv_heads, "scale": dim ** -0.5, "rot": {"base": 500000.0, "dims": dim}}
+    dense = {"kind": "dense", "ff": ff}
+    routed = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff // top}, "shared": {"ff": ff // top}}
+    kinds = [{"type": "latent_attention", "mixer": latent_mixer, "mlp": dense},
+             {"type": "latent_attention", "mixer": latent_mixer, "mlp": routed},
+             {"type": "attention", "mixer": attention, "mlp": dense},
+             {"type": "hgrn2", "mixer": base, "mlp": routed}]
+    return {"architecture": "Duvozen", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+            "logit_scale": 0.5, "canon": {"taps": 4}, "layers": [kinds[i % 4] for i in range(layers)]}
+
+
+# the layer sizes of llama-3.1-8b and llama-3.2-1b; 8 of 32 experts; cached rows of 512 + 64 and 256 + 32
+SHAPES["duvozen-8b"] = _duvozen(4096, 32, 8, 128, 14336, 128256, 32, (64, 512), 32, 8)
+SHAPES["duvozen-1b"] = _duvozen(2048, 32, 8, 64, 8192, 128256, 16, (32, 256), 32, 8)
+
+
 def shape(name: str, layers: int | None = None, window: int | None = None) -> dict:
     """A copy of the named shape's config.json, optionally with fewer layers (and, for a shape
     with windowed attention, another window)."""
