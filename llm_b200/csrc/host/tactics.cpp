@@ -176,6 +176,16 @@ std::string latent_tiles_guard(const Shape& s) {
     return "";
 }
 
+std::string latent_decode_guard(const Shape& s) {
+    if (!s.decode) return "serves steps in which every sequence brings one token";
+    if (!s.bf16) return "bfloat16 caches only";
+    if (s.kv_rank != 64 && s.kv_rank != 128 && s.kv_rank != 256 && s.kv_rank != 512)
+        return "a latent of " + std::to_string(s.kv_rank) + " elements (served: 64, 128, 256, 512)";
+    if (s.rot_dim > 64 || s.rot_dim % 8)
+        return "a rotated part of " + std::to_string(s.rot_dim) + " elements (served: multiples of 8 up to 64)";
+    return "";
+}
+
 std::string latent_prefill_guard(const Shape& s) {
     if (s.decode || !s.fresh) return "serves steps whose sequences all start at their first token";
     if (!s.bf16) return "bfloat16 operands only";
@@ -255,6 +265,10 @@ const std::vector<Row>& table(int family) {
          "prompts from their first token with the keys and values of every head formed by one product: flash attention "
          "with both products on tcgen05, two tiles of 128 queries a block over shared key and value blocks by TMA, one "
          "thread per query row"},
+        {"latent_decode_tc", 15, latent_decode_guard,
+         "one token a sequence on tcgen05: the cached rows by TMA through a ring of stages of 32, each read once for up to 32 "
+         "heads; scores with the heads as rows, values turned (O^T = V^T P^T) so that the accumulators fit in tensor memory; "
+         "slices of a long sequence merged by a second kernel"},
         {"latent_tiles", 10, latent_tiles_guard,
          "softmax attention of (token, head) pairs over the cached latent rows: all heads share a row, so a page goes "
          "into shared memory once for up to 64 pairs; mma.sync tiles, scores by (row, key) parts over eight warps, value "

@@ -12,11 +12,13 @@
 //                 the rows' maxima, and forms P V with every warp on a range of value columns for all rows. Long
 //                 sequences of a decode step are cut into slices of pages whose partial results a second kernel merges.
 //                 Shared memory rows are swizzled by 16-byte pieces (piece ^ row % 8).
+// latent_decode_tc (bfloat16)  the same for a step of one token a sequence on tcgen05, with the rows by TMA: see there.
 //
 // Norm, rotation, scores, weights and sums are 32-bit (weights are rounded as the operand of P V, whose sum is 32-bit).
 // A query at position p sees the keys j <= p.
 #include "common.cuh"
 #include "mma.cuh"
+#include "tc.cuh"
 
 using namespace llmb;
 
@@ -523,6 +525,350 @@ latent_tiles_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
         }
 }
 
+// One token a sequence on the fifth-generation tensor cores: block (slice, chunk of NH heads, sequence). The cached rows
+// stream through a ring of pages (boxes of 64 columns and 64 rows a piece, 128-byte swizzle; the last piece is the rotated
+// part, zeros beyond it), each read once for all heads of the block, by both products:
+//
+// * scores: S[head, key] = Q K^T, the heads as rows of the 128-row side, with the queries in tensor memory (written there
+//   once: a product that reads its 128 rows from shared memory takes twice as long, whatever its width; rows beyond NH
+//   hold what tensor memory held before: their results are not looked at).
+// * values: O^T[value element, head] += V^T P^T, 128 value elements a product, the rows' own bytes as an MN-major operand, P
+//   from shared memory (bfloat16 [head, key]); ceil(C / 128) accumulators of NH columns. Turned this way nothing is padded:
+//   with the heads on the 128-row side O alone would fill tensor memory.
+//
+// Warp 0: softmax, a lane a head (its 64 scores read once, and their buffer given back at once; running maximum and sum in
+// 32-bit). Warp 1, one lane: TMA. Warp 2, one lane: the products, whichever is ready first. Warps 4-7: rescale O where a
+// head's maximum outgrew its reference by 2^8 (a column is a head; rare), and the result. Pages of older rows than the
+// step's are requested before the kernel in front has ended. Waits are bounded.
+namespace decode {
+
+using namespace llmb::tc;
+
+constexpr int KEYS = LLMB_PAGE, PIECE = KEYS * 128, MAX_STAGES = 8;
+
+// whether the phase is complete, without waiting for it
+__device__ __forceinline__ bool mbar_test(uint32_t bar, uint32_t parity) {
+    uint32_t done;
+    asm volatile(
+        "{\n\t.reg .pred p;\n\t"
+        "mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
+        "selp.u32 %0, 1, 0, p;\n\t}"
+        : "=r"(done) : "r"(bar), "r"(parity) : "memory");
+    return done != 0;
+}
+
+struct Shape { int stages; size_t smem; };
+
+inline Shape shape_of(int C, int nh) {
+    Shape s;
+    size_t fixed = 1024 + 2 * (size_t)nh * 128 + 1024, stage = (size_t)(C / 64 + 1) * PIECE;
+    s.stages = (int)((227 * 1024 - fixed) / stage);
+    if (s.stages > MAX_STAGES) s.stages = MAX_STAGES;
+    s.smem = fixed + s.stages * stage;
+    if (s.smem < 120 * 1024) s.smem = 120 * 1024;           // one block an SM: it takes all of tensor memory
+    return s;
+}
+
+// NH: heads of a block; C: the latent
+template <int NH, int C>
+__global__ void __launch_bounds__(256, 1)
+latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __nv_bfloat16* __restrict__ q,
+                        const int* __restrict__ block_table, int table_stride, int ring_pages, const int* __restrict__ seq_lens,
+                        const int* __restrict__ seq_order, __nv_bfloat16* __restrict__ out, float* __restrict__ part_acc,
+                        float* __restrict__ part_stats, int H, int R, int stages, float scale_log2, int* status) {
+    constexpr int pieces = C / 64 + 1, values = (C + 127) / 128;         // of a row; accumulators
+    // tensor memory: the queries (two elements a column), the scores, the accumulators
+    constexpr uint32_t Q_COL = 0, S_COL = pieces * 32, O_COL = S_COL + KEYS, COLS = 512;
+    static_assert(O_COL + values * NH <= COLS, "tensor memory");
+    extern __shared__ __align__(1024) unsigned char smem_raw[];
+    unsigned char* base = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
+    unsigned char* ring = base;                                          // [stages][pieces][64][64]
+    unsigned char* p_tile = ring + (size_t)stages * pieces * PIECE;      // [2][NH][64]
+    uint64_t* full = reinterpret_cast<uint64_t*>(p_tile + 2 * NH * 128); // [8]
+    uint64_t* empty = full + 8;                                          // [8]
+    uint64_t* s_full = full + 16;                                        // the scores are complete
+    uint64_t* s_free = full + 17;                                        // they have been read
+    uint64_t* p_full = full + 18;                                        // [2] a buffer's weights are written (and O rescaled)
+    uint64_t* o_full = full + 20;                                        // [2] its values have been added
+    uint64_t* q_full = full + 22;
+    uint64_t* go = full + 23;                                            // warps 4-7: rescale, or the end
+    uint64_t* went = full + 24;                                          // they have rescaled
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(full + 25);
+    volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+    float* alphas = reinterpret_cast<float*>(full + 26);                 // [NH] factors, at the end the sums
+    float* maxima = alphas + NH;                                         // [NH]
+    volatile int* at_end = reinterpret_cast<volatile int*>(maxima + NH);
+
+    griddep_launch();
+    int split = blockIdx.x, n_splits = gridDim.x;
+    int seq = seq_order ? seq_order[blockIdx.z] : (int)blockIdx.z, head0 = blockIdx.y * NH;
+    int len = seq_lens[seq];
+    int n_pages = (len + KEYS - 1) / KEYS, per_split = (n_pages + n_splits - 1) / n_splits;
+    int page_begin = min(split * per_split, n_pages);
+    int n = min(page_begin + per_split, n_pages) - page_begin;           // pages of this slice
+    const int* pages = block_table + (size_t)seq * table_stride;
+    int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < 25; ++i) mbar_init(smem_u32(&full[i]), i == 24 ? 128 : (i == 17 || i == 18 || i == 19 || i == 22) ? 32 : 1);
+        *abort_flag = 0;
+        *at_end = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (warp == 2) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;"
+                     ::"r"(smem_u32(tmem_slot)), "r"(COLS) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    tcgen05_fence_before();
+    __syncthreads();
+    tcgen05_fence_after();
+    uint32_t tmem_base = *tmem_slot;
+
+    if (warp == 1) {
+        if (lane == 0) {
+            auto request = [&](int j) {
+                int s = j % stages;
+                uint32_t bar = smem_u32(&full[s]);
+                mbar_expect_tx(bar, pieces * PIECE);
+                int row = pages[(page_begin + j) % ring_pages] * KEYS;
+                for (int c = 0; c < pieces; ++c)
+                    tma_load_2d(smem_u32(ring + ((size_t)s * pieces + c) * PIECE), &map_rows, bar, c * 64, row);
+            };
+            int j = 0;
+            // pages of older positions are final: requested before the kernel in front has ended
+            while (j < n && j < stages && (page_begin + j + 1) * KEYS <= len - 1) request(j++);
+            griddep_wait();
+            for (; j < n; ++j) {
+                if (j >= stages && !mbar_wait(smem_u32(&empty[j % stages]), (j / stages - 1) & 1, abort_flag, status, 41)) break;
+                request(j);
+            }
+        } else {
+            griddep_wait();
+        }
+    } else if (warp == 2) {
+        griddep_wait();
+        if (lane == 0 && n > 0) {
+            // D 32-bit, A and B bfloat16, M = 128. Scores: N = 64 keys, K-major. Values: N = NH heads, A MN-major.
+            constexpr uint32_t idesc_s = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(KEYS >> 3) << 17) | (8u << 24);
+            constexpr uint32_t idesc_o = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 15) | ((uint32_t)(NH >> 3) << 17) | (8u << 24);
+            const uint64_t k_desc0 = smem_desc(smem_u32(ring)), v_desc0 = smem_desc_mn(smem_u32(ring), PIECE);
+            const uint64_t p_desc0 = smem_desc(smem_u32(p_tile));
+            int next_s = 0, next_o = 0, s_stage = 0, o_stage = 0;
+            uint32_t s_phase = 0;
+            long long since = 0;
+            bool ok = mbar_wait(smem_u32(q_full), 0, abort_flag, status, 42);
+            tcgen05_fence_after();
+            while (ok && next_o < n) {
+                bool moved = false;
+                if (next_s < n && mbar_test(smem_u32(&full[s_stage]), s_phase) &&
+                    (next_s == 0 || mbar_test(smem_u32(s_free), (next_s - 1) & 1))) {
+                    tcgen05_fence_after();
+                    uint64_t k_desc = k_desc0 + (uint64_t)((s_stage * pieces * PIECE) >> 4);
+                    // (all steps spelled out: the one lane that issues them sets their pace)
+#pragma unroll
+                    for (int k = 0; k < pieces * 4; ++k)
+                        tcgen05_mma_ts(tmem_base + S_COL, tmem_base + Q_COL + k * 8,
+                                       k_desc + (uint64_t)(((k >> 2) * PIECE + (k & 3) * 32) >> 4), idesc_s, k > 0 ? 1u : 0u);
+                    tcgen05_commit(smem_u32(s_full));
+                    ++next_s;
+                    if (++s_stage == stages) { s_stage = 0; s_phase ^= 1; }
+                    moved = true;
+                }
+                if (next_o < next_s && mbar_test(smem_u32(&p_full[next_o & 1]), (next_o >> 1) & 1)) {
+                    tcgen05_fence_after();
+                    uint64_t v_desc = v_desc0 + (uint64_t)((o_stage * pieces * PIECE) >> 4);
+                    uint64_t p_desc = p_desc0 + (uint64_t)(((next_o & 1) * NH * 128) >> 4);
+#pragma unroll
+                    for (int m = 0; m < values; ++m)
+#pragma unroll
+                        for (int k = 0; k < KEYS / 16; ++k)           // 16 keys: 2,048 bytes of rows, 32 bytes of P
+                            tcgen05_mma(tmem_base + O_COL + m * NH, v_desc + (uint64_t)((2 * m * PIECE + k * 2048) >> 4),
+                                        p_desc + 2 * k, idesc_o, (next_o > 0 || k > 0) ? 1u : 0u);
+                    tcgen05_commit(smem_u32(&o_full[next_o & 1]));
+                    tcgen05_commit(smem_u32(&empty[o_stage]));
+                    ++next_o;
+                    if (++o_stage == stages) o_stage = 0;
+                    moved = true;
+                }
+                if (moved) {
+                    since = 0;
+                } else {
+                    if (*abort_flag) break;
+                    long long now = clock64();
+                    if (since == 0) since = now;
+                    else if (now - since > WAIT_CYCLES) {
+                        *abort_flag = 1;
+                        if (status) atomicCAS(status, 0, 43);
+                        break;
+                    }
+                }
+            }
+        }
+    } else if (warp == 0) {
+        griddep_wait();
+        // the queries, a lane a head, into tensor memory (zeros beyond the head count and beyond the row)
+        const bool live = lane < NH && head0 + lane < H;
+        const __nv_bfloat16* row_q = q + ((size_t)seq * H + head0 + (live ? lane : 0)) * (C + R);
+#pragma unroll 1
+        for (int c = 0; c < pieces; ++c) {
+            uint32_t r[32];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                uint4 v = make_uint4(0u, 0u, 0u, 0u);
+                if (live && c * 64 + i * 8 < C + R) v = *reinterpret_cast<const uint4*>(row_q + c * 64 + i * 8);
+                r[4 * i] = v.x; r[4 * i + 1] = v.y; r[4 * i + 2] = v.z; r[4 * i + 3] = v.w;
+            }
+            uint32_t lo[16], hi[16];
+#pragma unroll
+            for (int i = 0; i < 16; ++i) { lo[i] = r[i]; hi[i] = r[16 + i]; }
+            tmem_st16(tmem_base + Q_COL + c * 32, lo);
+            tmem_st16(tmem_base + Q_COL + c * 32 + 16, hi);
+        }
+        tmem_st_wait();
+        tcgen05_fence_before();
+        mbar_arrive(smem_u32(q_full));
+        float run_max = -INFINITY, run_sum = 0.f;
+        bool ok = true;
+        int rescales = 0;
+        for (int j = 0; j < n && ok; ++j) {
+            int b = j & 1, phase = (j >> 1) & 1;
+            ok = mbar_wait(smem_u32(s_full), j & 1, abort_flag, status, 44);
+            if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
+            tcgen05_fence_after();
+            uint32_t ra[32], rb[32];
+            tmem_ld32_start(tmem_base + S_COL, ra);
+            tmem_ld32_start(tmem_base + S_COL + 32, rb);
+            tmem_ld32_wait(ra);
+            tmem_ld32_wait(rb);
+            tcgen05_fence_before();
+            mbar_arrive(smem_u32(s_free));
+            int left = len - (page_begin + j) * KEYS;                // keys of this page that exist
+            if (left < KEYS) {
+#pragma unroll
+                for (int i = 0; i < 32; ++i) {
+                    if (i >= left) ra[i] = 0xff800000u;              // -inf
+                    if (32 + i >= left) rb[i] = 0xff800000u;
+                }
+            }
+            float block_max = -INFINITY;
+#pragma unroll
+            for (int i = 0; i < 32; ++i) block_max = max3(block_max, __uint_as_float(ra[i]), __uint_as_float(rb[i]));
+            bool move = j == 0 || (block_max - run_max) * scale_log2 > 8.f;
+            float new_max = move ? block_max : run_max;
+            float alpha = (move && j > 0) ? fast_exp2((run_max - new_max) * scale_log2) : 1.f;
+            float shift = new_max * scale_log2, add = 0.f;
+            run_max = new_max;
+            if (j >= 2) ok = mbar_wait(smem_u32(&o_full[b]), phase ^ 1, abort_flag, status, 45);          // P's buffer has been read
+            if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
+            unsigned char* row = p_tile + (b * NH + (lane < NH ? lane : 0)) * 128;
+            auto weights = [&](const uint32_t (&r)[32], int half) {
+#pragma unroll
+                for (int c = 0; c < 4; ++c) {                        // 8 keys: 16 bytes
+                    uint32_t packed[4];
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        float p0 = fast_exp2(fmaf(__uint_as_float(r[8 * c + 2 * i]), scale_log2, -shift));
+                        float p1 = fast_exp2(fmaf(__uint_as_float(r[8 * c + 2 * i + 1]), scale_log2, -shift));
+                        add += p0 + p1;
+                        packed[i] = pack_bf16(p0, p1);
+                    }
+                    if (lane < NH)
+                        *reinterpret_cast<uint4*>(row + (((half * 4 + c) ^ (lane & 7)) << 4)) =
+                            make_uint4(packed[0], packed[1], packed[2], packed[3]);
+                }
+            };
+            weights(ra, 0);
+            weights(rb, 1);
+            run_sum = run_sum * alpha + add;
+            if (!live) alpha = 1.f;                                  // (no head: whatever its scores are)
+            if (j > 0 && __any_sync(0xffffffffu, alpha != 1.f)) {
+                ok = mbar_wait(smem_u32(&o_full[b ^ 1]), ((j - 1) >> 1) & 1, abort_flag, status, 46);     // the page before has been added
+                if (lane < NH) alphas[lane] = alpha;
+                __syncwarp();
+                if (lane == 0) mbar_arrive(smem_u32(go));
+                ok = ok && mbar_wait(smem_u32(went), rescales & 1, abort_flag, status, 47);
+                ++rescales;
+            }
+            if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
+            fence_async_shared();
+            tcgen05_fence_before();
+            mbar_arrive(smem_u32(&p_full[b]));
+        }
+        // what the result needs, then the signal
+        if (lane < NH) { alphas[lane] = run_sum; maxima[lane] = run_max; }
+        if (lane == 0) *at_end = 1;
+        __threadfence_block();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(smem_u32(go));
+    } else if (warp >= 4) {
+        griddep_wait();
+        int quarter = warp & 3;
+        uint32_t lane_addr = tmem_base + O_COL + ((uint32_t)(quarter * 32) << 16);
+        bool ok = true;
+        for (int turn = 0;; ++turn) {
+            ok = mbar_wait(smem_u32(go), turn & 1, abort_flag, status, 48);
+            if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
+            if (*at_end) break;
+            tcgen05_fence_after();
+#pragma unroll 1
+            for (int c = 0; c < values * NH; c += 16) {
+                uint32_t r[16];
+                tmem_ld16(lane_addr + c, r);
+#pragma unroll
+                for (int i = 0; i < 16; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * alphas[(c % NH) + i]);
+                tmem_st16(lane_addr + c, r);
+            }
+            tmem_st_wait();
+            tcgen05_fence_before();
+            mbar_arrive(smem_u32(went));
+        }
+        if (ok && n > 0) ok = mbar_wait(smem_u32(&o_full[(n - 1) & 1]), ((n - 1) >> 1) & 1, abort_flag, status, 49);
+        if (__all_sync(0xffffffffu, ok)) {
+            tcgen05_fence_after();
+            int heads = min(NH, H - head0);
+            size_t row0 = (size_t)seq * H + head0;
+            if (n_splits > 1 && warp == 4 && lane < heads) {
+                float* to = part_stats + ((row0 + lane) * n_splits + split) * 2;
+                to[0] = n > 0 ? maxima[lane] * scale_log2 : -INFINITY;
+                to[1] = n > 0 ? alphas[lane] : 0.f;
+            }
+#pragma unroll 1
+            for (int m = 0; m < values; ++m) {
+                int d = m * 128 + quarter * 32 + lane;
+#pragma unroll
+                for (int c = 0; c < NH; c += 16) {
+                    uint32_t r[16];
+                    if (n > 0) tmem_ld16(lane_addr + m * NH + c, r);
+                    if (d >= C) continue;
+#pragma unroll
+                    for (int i = 0; i < 16; ++i) {
+                        if (c + i >= heads) break;
+                        float v = n > 0 ? __uint_as_float(r[i]) : 0.f;
+                        if (n_splits == 1) out[(row0 + c + i) * C + d] = __float2bfloat16_rn(v / alphas[c + i]);
+                        else part_acc[((row0 + c + i) * n_splits + split) * C + d] = v;
+                    }
+                }
+            }
+        }
+    } else {
+        griddep_wait();
+    }
+
+    tcgen05_fence_before();
+    __syncthreads();
+    if (*abort_flag) {
+        for (int i = 0; i < 100; ++i) __nanosleep(10000);          // copies in flight land before shared memory is given up
+        __syncthreads();
+    }
+    if (warp == 2) {
+        tcgen05_fence_after();
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"(COLS) : "memory");
+    }
+}
+
+}  // namespace decode
+
 // block (row): the slices' weighted values, maxima (base-2 units) and sums merged in slice order
 __global__ void __launch_bounds__(128)
 latent_combine_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_stats, __nv_bfloat16* __restrict__ out,
@@ -630,3 +976,67 @@ LLMB_EXPORT int llmb_latent_attention(const void* q, const void* cache, const in
     return check_launch("latent_attention_combine");
 }
 LLMB_PACKED(llmb_latent_attention)
+
+LLMB_EXPORT int llmb_latent_attention_status() {
+    int* s = llmb::tc::status_word();
+    if (!s) return -1;
+    int v = *s;
+    *s = 0;
+    return v;
+}
+
+// A step of one token a sequence: q [n_seqs, H, C + R] (contiguous), cache [n_pages, 1, 64, C + R], out [n_seqs, H, C]; all
+// bfloat16. scratch as in llmb_latent_attention.
+LLMB_EXPORT int llmb_latent_decode_tc(const void* q, const void* cache, int n_pages, const int* block_table, int table_stride,
+                                      int ring_pages, const int* seq_lens, const int* seq_order, void* out, float* scratch,
+                                      long long scratch_floats, int n_seqs, int H, int C, int R, float scale, int n_splits,
+                                      cudaStream_t stream) {
+    if (n_seqs == 0) return LLMB_OK;
+    LLMB_REQUIRE(H > 0 && (C == 64 || C == 128 || C == 256 || C == 512) && R > 0 && R <= 64 && R % 8 == 0,
+                 "latent_decode_tc: rows of %d + %d (64, 128, 256 or 512, a multiple of 8 up to 64)", C, R);
+    LLMB_REQUIRE(n_seqs <= 65535 && n_pages > 0 && ring_pages > 0 && n_splits >= 1 && scale > 0.f, "latent_decode_tc: bad sizes");
+    LLMB_REQUIRE(((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(out)) & 15) == 0,
+                 "latent_decode_tc: operands must be 16-byte aligned");
+    LLMB_REQUIRE(n_splits == 1 || (scratch && scratch_floats >= llmb_latent_scratch_floats(n_seqs, H, C, n_splits)),
+                 "latent_decode_tc: scratch too small");
+    int nh = H <= 16 ? 16 : 32;
+    decode::Shape s = decode::shape_of(C, nh);
+    LLMB_REQUIRE(s.stages >= 2 && s.smem <= 227 * 1024, "latent_decode_tc: %zu bytes of shared memory", s.smem);
+    CUtensorMap map_rows;
+    int code;
+    if ((code = llmb::tc::make_map_2d(&map_rows, cache, (long long)n_pages * LLMB_PAGE, C + R, C + R, 64, decode::KEYS))) return code;
+    float* part_acc = scratch;
+    float* part_stats = scratch ? scratch + (long long)n_seqs * H * n_splits * C : nullptr;
+    int* status_dev = nullptr;
+    int* status_host = llmb::tc::status_word();
+    if (status_host) LLMB_CUDA(cudaHostGetDevicePointer((void**)&status_dev, status_host, 0));
+#define LLMB_DECODE_AS(NH, CC)                                                                                            \
+    do {                                                                                                                  \
+        static bool configured = false;                                                                                   \
+        if (!configured) {                                                                                                \
+            LLMB_CUDA(cudaFuncSetAttribute(decode::latent_decode_tc_kernel<NH, CC>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                           (int)s.smem));                                                                 \
+            configured = true;                                                                                            \
+        }                                                                                                                 \
+        LLMB_CUDA(llmb::launch(decode::latent_decode_tc_kernel<NH, CC>, dim3(n_splits, ceil_div(H, NH), n_seqs), dim3(256), s.smem, \
+                               stream, true, map_rows, (const __nv_bfloat16*)q, block_table, table_stride, ring_pages, seq_lens, seq_order, \
+                               (__nv_bfloat16*)out, part_acc, part_stats, H, R, s.stages, scale * 1.4426950408889634f, status_dev)); \
+    } while (0)
+#define LLMB_DECODE(NH)                               \
+    do {                                              \
+        if (C == 64) LLMB_DECODE_AS(NH, 64);          \
+        else if (C == 128) LLMB_DECODE_AS(NH, 128);   \
+        else if (C == 256) LLMB_DECODE_AS(NH, 256);   \
+        else LLMB_DECODE_AS(NH, 512);                 \
+    } while (0)
+    if (nh == 16) LLMB_DECODE(16);
+    else LLMB_DECODE(32);
+#undef LLMB_DECODE
+#undef LLMB_DECODE_AS
+    code = check_launch("latent_decode_tc");
+    if (code || n_splits == 1) return code;
+    LLMB_CUDA(llmb::launch(latent_combine_kernel, dim3(n_seqs * H), dim3(128), 0, stream, true, (const float*)part_acc,
+                           (const float*)part_stats, (__nv_bfloat16*)out, C, n_splits));
+    return check_launch("latent_attention_combine");
+}
+LLMB_PACKED(llmb_latent_decode_tc)

@@ -974,7 +974,7 @@ def check_device_status() -> None:
     """Raise if a kernel of a loaded library reported a wait that ran out. Cheap (it
     reads a word of host memory); meaningful after the stream was synchronised."""
     from .build import _loaded
-    for name in ("gemm_tc", "attention_prefill_tc", "routed_experts", "latent_prefill_tc"):
+    for name in ("gemm_tc", "attention_prefill_tc", "routed_experts", "latent_prefill_tc", "latent_attention"):
         if name in _loaded:
             code = getattr(_loaded[name], f"llmb_{name}_status")()
             if code != 0:
@@ -1347,15 +1347,17 @@ def head_products(x, x_head: int, w, out, out_head: int):
     return out
 
 
-def latent_decode_splits(n_seqs: int, n_heads: int, max_len: int, pairs_fit: bool = False) -> int:
-    """Slices of the latent attention in a decode step: `decode_splits` for its blocks a sequence (64 heads each)."""
-    tile = 16 if n_heads <= 16 else 32 if n_heads <= 32 else 64
-    return decode_splits(n_seqs, (n_heads + tile - 1) // tile, max_len, wave=296 if pairs_fit else 148)
-
-
-@functools.lru_cache(maxsize=256)
-def _latent_pairs_fit(rank: int, rot: int, rows: int) -> bool:
-    return bool(load_library("latent_attention").llmb_latent_tile_pairs(_c_int(rank), _c_int(rot), _c_int(rows)))
+@functools.lru_cache(maxsize=1024)
+def latent_decode_splits(n_seqs: int, n_heads: int, rank: int, rot: int, max_len: int, tensor: bool) -> int:
+    """Slices of the latent attention in a decode step: `decode_splits` for its blocks a sequence and the blocks that
+    fit on an SM together (one or two)."""
+    lib = load_library("latent_attention")
+    if tensor:
+        tile, pairs = (16 if n_heads <= 16 else 32), 0
+    else:
+        tile = lib.llmb_latent_tile_rows(_c_int(rank), _c_int(rot), _c_int(n_heads))
+        pairs = lib.llmb_latent_tile_pairs(_c_int(rank), _c_int(rot), _c_int(n_heads))
+    return decode_splits(n_seqs, (n_heads + tile - 1) // tile, max_len, wave=296 if pairs else 148)
 
 
 def latent_attention_replay_key(step, n_heads: int):
@@ -1385,7 +1387,8 @@ def latent_attention(queries, cache, block_table, ring_pages, tok_pos, tok_seq, 
         return out
     splits, scratch = 1, None
     if decode:
-        splits = latent_decode_splits(n, n_heads, max_len, _latent_pairs_fit(rank, rot, n_heads))
+        tensor = variant == "latent_decode_tc"
+        splits = latent_decode_splits(n, n_heads, rank, rot, max_len, tensor)
         need = n * n_heads * splits * (rank + 2) if splits > 1 else 0
         scratch = _attention_scratch.get(queries.device)
         if scratch is None or scratch.numel() < need:
@@ -1395,6 +1398,12 @@ def latent_attention(queries, cache, block_table, ring_pages, tok_pos, tok_seq, 
                 _scratch_generation += 1
             scratch = torch.empty(max(need, 1 << 23), dtype=torch.float32, device=queries.device)
             _attention_scratch[queries.device] = scratch
+        if tensor:
+            _call("latent_attention", "llmb_latent_decode_tc", _ptr(queries), _ptr(cache), _c_int(cache.shape[0]),
+                  _ptr(block_table), _c_int(block_table.shape[1]), _c_int(ring_pages), _ptr(seq_lens), _ptr(seq_order), _ptr(out),
+                  _ptr(scratch), ctypes.c_longlong(scratch.numel()), _c_int(n), _c_int(n_heads), _c_int(rank), _c_int(rot),
+                  _c_float(scale), _c_int(splits), _stream(), kernels=2 if splits > 1 else 1)
+            return out
     _call("latent_attention", "llmb_latent_attention", _ptr(queries), _ptr(cache), _ptr(block_table), _c_int(block_table.shape[1]),
           _c_int(ring_pages), _ptr(cu_seqlens), _ptr(seq_lens), _ptr(seq_order), _ptr(out), _ptr(scratch),
           ctypes.c_longlong(scratch.numel() if scratch is not None else 0), _c_int(n), _c_int(cu_seqlens.numel() - 1),

@@ -154,7 +154,8 @@ def phase_sums(fn, label: str) -> int:
 
 def main(argv=None) -> int:
     p = argparse.ArgumentParser(description=__doc__.split("\n")[0])
-    p.add_argument("op", choices=["delta_rule", "gated_recurrence", "state_space", "routed_experts", "norm_add",
+    p.add_argument("op", choices=["forget_recurrence", "latent_attention", "latent_prefill", "head_products", "latent_write",
+                                  "output_norm", "input_conv", "delta_rule", "gated_recurrence", "state_space", "routed_experts", "norm_add",
                                   "linear", "attention_decode", "attention_prefill", "rmsnorm",
                                   "swiglu", "rope", "sample"])
     p.add_argument("--m", type=int, default=8, help="rows (tokens)")
@@ -181,6 +182,8 @@ def main(argv=None) -> int:
                         "repeat penalty 1.1 over the last 64) runs")
     p.add_argument("--experts", type=int, default=32)
     p.add_argument("--top", type=int, default=8, help="routed_experts: chosen experts; norm_add: rows a token")
+    p.add_argument("--rank", type=int, default=512, help="latent kernels: the cached latent (512)")
+    p.add_argument("--rot", type=int, default=64, help="latent kernels: the shared rotated key part")
     p.add_argument("--reps", type=int, default=20)
     p.add_argument("--once", action="store_true")
     p.add_argument("--timeline", action="store_true",
@@ -372,6 +375,80 @@ def main(argv=None) -> int:
         run(lambda: ops.state_space(proj, taps, conv_b, state, seq, cu, slots, rate, dt_bias, skip, weight, 1e-5, 8, 1.0, work, y,
                                     mixed, H, G, N, V), args, moved, 5.0 * n * H * N * V,
             f"state_space {b} x {t} tokens, {H} heads of {V} with states of {N} in {G} groups")
+    elif args.op == "forget_recurrence":
+        # `--batch` sequences bring `--tokens` tokens each (1: a decode step): `--heads` heads, states of `--head-dim` squared
+        from llm_b200 import ops
+        b, t, H, D = args.batch, args.tokens, args.heads, args.head_dim
+        n = b * t
+        cu, slots = torch.arange(b + 1, dtype=torch.int32, device=DEV) * t, torch.arange(b, dtype=torch.int32, device=DEV)
+        proj = torch.randn(n, 3 * H * D, device=DEV).to(bf16)
+        bias, lower, weight = torch.ones(H * D, device=DEV), torch.rand(H * D, device=DEV) * 0.9, torch.ones(D, device=DEV)
+        state = torch.zeros(b, H * D * D, device=DEV)
+        work = torch.empty(n, ops.forget_recurrence_work_width(H, D, D), device=DEV)
+        o, mixed = torch.empty(n, H * D, device=DEV), torch.empty(n, H * D, device=DEV, dtype=bf16)
+        moved = proj.numel() * 2 + mixed.numel() * 2 + state.numel() * 8
+        run(lambda: ops.forget_recurrence(proj, bias, lower, state, cu, slots, weight, 1e-5, work, o, mixed, H, D, D,
+                                          single_tokens=t == 1), args, moved, 5.0 * n * H * D * D,
+            f"forget_recurrence {b} x {t} tokens, {H} heads with states of {D} x {D}")
+    elif args.op in ("latent_attention", "latent_prefill", "latent_write", "head_products"):
+        # latent rows of `--rank` + `--rot`, `--heads` heads of `--head-dim` + `--rot`, values of `--head-dim`. latent_attention:
+        # a decode step of `--batch` sequences at `--context`, or (`--tokens` > 1) the last `--tokens` tokens of each
+        from llm_b200 import ops
+        H, D, C, R = args.heads, args.head_dim, args.rank, args.rot
+        b, t = args.batch, args.tokens
+        n, width = b * t, C + R
+        cu, order = torch.arange(b + 1, dtype=torch.int32, device=DEV) * t, torch.arange(b, dtype=torch.int32, device=DEV)
+        if args.op == "latent_prefill":
+            proj = torch.randn(n, H * (D + R) + width, device=DEV).to(bf16)
+            kv, dense = torch.randn(n, H * 2 * D, device=DEV).to(bf16), torch.randn(n, width, device=DEV).to(bf16)
+            out = torch.empty(n, H * D, device=DEV, dtype=bf16)
+            run(lambda: ops.latent_prefill(proj, kv, dense, H, D, R, D, C, (D + R) ** -0.5, out, cu, t, order), args,
+                (proj.numel() + kv.numel() + dense.numel() + out.numel()) * 2, b * t * t * H * (2.0 * D + R),
+                f"latent_prefill {b} x {t} tokens, {H} heads of {D} + {R}")
+        elif args.op == "head_products":
+            x, w = torch.randn(n, H * D, device=DEV).to(bf16), torch.randn(H, C, D, device=DEV).to(bf16)
+            out = torch.empty(n, H * width, device=DEV, dtype=bf16)
+            run(lambda: ops.head_products(x, D, w, out, width), args, (x.numel() + w.numel() + n * H * C) * 2, 2.0 * n * H * C * D,
+                f"head_products {n} tokens, {H} matrices of {C} x {D}")
+        else:
+            context = max(args.context, t)
+            pages = (context + 63) // 64
+            table = torch.arange(b * pages, dtype=torch.int32, device=DEV).view(b, pages)
+            cache = torch.randn(b * pages, 1, 64, width, device=DEV).to(bf16)
+            pos = torch.arange(context - t, context, dtype=torch.int32, device=DEV).repeat(b)
+            seq = torch.arange(b, dtype=torch.int32, device=DEV).repeat_interleave(t)
+            if args.op == "latent_write":
+                proj = torch.randn(n, H * (D + R) + width, device=DEV).to(bf16)
+                gain, angles = torch.ones(C, device=DEV), torch.rand(context, R, device=DEV)
+                queries, dense = torch.empty(n, H * width, device=DEV, dtype=bf16), torch.empty(n, width, device=DEV, dtype=bf16)
+                form = dict(queries=queries) if t == 1 else dict(dense=dense)
+                run(lambda: ops.latent_write(proj, H, D, R, C, gain, 1e-5, angles, True, pos, seq, table, pages, cache, **form), args,
+                    n * (H * R * 4 + width * (4 if t == 1 else 6)), 0.0, f"latent_write {n} tokens")
+            else:
+                q, out = torch.randn(n, H * width, device=DEV).to(bf16), torch.empty(n, H * C, device=DEV, dtype=bf16)
+                lens = torch.full((b,), context, dtype=torch.int32, device=DEV)
+                keys = float(b) * (t * (context - t) + t * (t + 1) / 2)
+                run(lambda: ops.latent_attention(q, cache, table, pages, pos, seq, H, C, R, width ** -0.5, out, decode=t == 1,
+                                                 seq_lens=lens, max_len=context, cu_seqlens=cu, max_new=t, seq_order=order), args,
+                    cache.numel() * 2 + (q.numel() + out.numel()) * 2, 2.0 * keys * H * (2 * C + R),
+                    f"latent_attention {b} x {t} tokens at {context}, {H} heads over rows of {C} + {R}")
+    elif args.op in ("output_norm", "input_conv"):
+        # `--m` tokens of width `--k`, four taps; output_norm: `--top` result rows and one behind, in a step of one token a
+        # sequence with the next input (`--tokens` 1) or alone
+        from llm_b200 import ops
+        m, k, K = args.m, args.k, 4
+        x, y, extra = torch.randn(m, k, device=DEV), torch.randn(m * args.top, k, device=DEV), torch.randn(m, k, device=DEV)
+        gain, taps, out = torch.ones(k, device=DEV), torch.randn(K, k, device=DEV) / 4, torch.empty(m, k, device=DEV, dtype=bf16)
+        if args.op == "input_conv":
+            state, slots = torch.zeros(1, K - 1, k, device=DEV), torch.zeros(1, dtype=torch.int32, device=DEV)
+            cu = torch.tensor([0, m], dtype=torch.int32, device=DEV)
+            run(lambda: ops.input_conv(x, taps, state, cu, slots, out, m), args, m * k * 6, 0.0, f"input_conv {m}x{k}, {K} taps")
+        else:
+            state, slots = torch.zeros(m, K - 1, k, device=DEV), torch.arange(m, dtype=torch.int32, device=DEV)
+            conv = (taps, state, slots, out) if args.tokens == 1 else None
+            run(lambda: ops.output_norm_add_(x, y, gain, 1e-5, "layernorm", args.top, extra=extra, conv=conv), args,
+                m * k * (4 * args.top + 12 + (8 * (K - 1) + 2 if conv else 0)), 0.0,
+                f"output_norm_add {m}x{k}, {args.top} + 1 rows a token{', with the next input' if conv else ''}")
     elif args.op == "routed_experts":
         # `--m` tokens, width `--k`, `--experts` experts of `--n`, `--top` chosen; weights rotate only across experts
         from llm_b200 import ops

@@ -311,12 +311,12 @@ def test_head_products(dtype, case):
 LATENT_CASES = [(3, 11, 6), (4, 80, 16), (2, 128, 64), (20, 40, 8), (40, 64, 32), (16, 256, 64), (33, 512, 64), (1, 512, 128), (70, 96, 32)]
 
 
-@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16, "generic"])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16, "tiles", "generic"])
 @pytest.mark.parametrize("case", LATENT_CASES)
 def test_latent_attention(dtype, case):
     ops = _ops()
-    plainly = dtype == "generic"
-    dtype = torch.bfloat16 if plainly else dtype
+    without = {"tiles": ("latent_decode_tc",), "generic": ("latent_decode_tc", "latent_tiles")}.get(dtype, ())
+    dtype = torch.bfloat16 if without else dtype
     H, C, R = case
     for lengths, new in BATCHES + [([400, 64, 129], [3, 3, 129]), ([700, 1, 64, 65, 300], [1] * 5)]:
         batch = Batch(lengths, new, seed=3 + len(lengths))
@@ -326,11 +326,34 @@ def test_latent_attention(dtype, case):
         results = []
         for fn in (ops.latent_attention, plain_ops.latent_attention):
             out = torch.zeros((batch.n_tokens, H * C), dtype=dtype, device=DEV)
-            with off(*(("latent_tiles",) if plainly else ())):
+            with off(*without):
                 fn(q, cache, batch.table, batch.width, batch.tok_pos, batch.tok_seq, H, C, R, (C + R) ** -0.5, out, **batch.extra())
             results.append(out)
         torch.cuda.synchronize()
+        ops.check_device_status()
         _close(results[0], results[1], dtype, (case, lengths))
+
+
+def test_latent_decode_with_scores_that_grow():
+    """Scores that rise along the sequence, in some heads and not in others: the exponents' references move again and
+    again, each head's at places of its own."""
+    ops = _ops()
+    for H, C, R, n in ((20, 64, 8, 700), (32, 512, 64, 330), (7, 256, 40, 129)):
+        batch = Batch([n, 64, 1], [1, 1, 1], seed=2)
+        cache, _ = batch.caches(1, C + R, 0, torch.bfloat16, seed=3, std=0.3)
+        for p in range(n):
+            page, row = batch.place(0, p)
+            cache[page, 0, row, :4] = torch.tensor([p / 20.0, -p / 30.0, (p % 97) / 5.0, 1.0])
+        q = torch.zeros((3, H * (C + R)), dtype=torch.bfloat16, device=DEV)
+        heads = q.view(3, H, C + R)
+        for h in range(H):
+            heads[:, h, h % 4] = 1.0 + h / 8.0
+        got, want = (torch.zeros((3, H * C), dtype=torch.bfloat16, device=DEV) for _ in range(2))
+        for fn, out in ((ops.latent_attention, got), (plain_ops.latent_attention, want)):
+            fn(q, cache, batch.table, batch.width, batch.tok_pos, batch.tok_seq, H, C, R, 1.0, out, **batch.extra())
+        torch.cuda.synchronize()
+        ops.check_device_status()
+        _close(got, want, torch.bfloat16, (H, C))
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
@@ -339,9 +362,14 @@ def test_latent_attention_planted_keys(dtype, decode):
     """One row stands out by its rotated part alone (its latent part scores nothing) and the result is its latent part:
     far back, at page borders, the newest, and one beyond the query, which must not be seen."""
     ops = _ops()
-    H, C, R, length = 20, 72, 8, 331
+    for H, C in ((20, 72), (20, 64), (3, 128)):
+        _latent_planted(ops, dtype, decode, H, C)
+
+
+def _latent_planted(ops, dtype, decode, H, C):
+    R, length = 8, 331
     batch = Batch([length, 40], [1, 1] if decode else [length, 40], seed=11)
-    for planted in (0, 1, 63, 64, 255, 256, length - 2, length - 1):
+    for planted in (0, 1, 31, 32, 63, 64, 255, 256, length - 2, length - 1):
         cache, _ = batch.caches(1, C + R, 0, dtype, seed=6, std=0.1)
         page, row = batch.place(0, planted)
         cache[page, 0, row] = 0.0
