@@ -21,6 +21,7 @@
 //          staged in shared memory eight at a time, the next eight requested under the current.
 // finish   o / sqrt(mean(o^2) + eps) * weight * silu(gate) per head, rounded to the run's dtype.
 #include "common.cuh"
+#include "pairs.cuh"
 
 using namespace llmb;
 
@@ -115,25 +116,6 @@ __device__ __forceinline__ void copy4(float* smem, const float* global) {
 __device__ __forceinline__ void copy16(float* smem, const float* global) {
     unsigned s = (unsigned)__cvta_generic_to_shared(smem);
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(s), "l"(global));
-}
-
-// two 32-bit floats in one 64-bit register and the packed arithmetic on them (each half rounded as the scalar form)
-typedef unsigned long long pair_t;
-__device__ __forceinline__ pair_t pack2(float lo, float hi) {
-    pair_t r;
-    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
-    return r;
-}
-__device__ __forceinline__ void unpack2(pair_t v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
-__device__ __forceinline__ pair_t fma2(pair_t a, pair_t b, pair_t c) {
-    pair_t d;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-    return d;
-}
-__device__ __forceinline__ pair_t mul2(pair_t a, pair_t b) {
-    pair_t d;
-    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-    return d;
 }
 
 constexpr int SCAN_THREADS = 128;

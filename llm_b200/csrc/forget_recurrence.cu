@@ -9,15 +9,16 @@
 // contiguous).
 //
 // Every column of S is a recurrence of its own, with a decay per row; a warp holds several columns of one head, lane l
-// the state rows l, l + 32, .. of each; per token it fades, writes and sums S q over its rows (a lane's rows in rising
-// order, then the lanes as a butterfly), so a token's result depends on nothing but the sequence before it, and is the
-// same bits in either form:
+// the pairs of state rows 2 l, 2 l + 1, then 64 further, .. of each, as packed 32-bit values (one instruction a pair);
+// per token it fades, writes and sums S q over its rows (even and odd rows in rising order, the two added, then the lanes
+// as a butterfly), so a token's result depends on nothing but the sequence before it, and is the same bits in either form:
 //
 // steps with more than one token a sequence: prepare (gates into a 32-bit work row [f | q | v] per token), scan (a block
 //     holds 32 columns; tokens staged in shared memory a chunk at a time, the next chunk requested under the current; the
 //     partial sums of several tokens meet in one butterfly), finish (the heads' norm, rounded to the run's dtype).
 // steps of one token a sequence: ONE launch, a block per head and sequence: the head's state is requested before the
 //     kernel in front has ended (nothing else in a step touches it), then gates, update, read-out and norm.
+#include "pairs.cuh"
 #include "scan.cuh"
 
 using namespace llmb;
@@ -31,7 +32,22 @@ __device__ __forceinline__ float forget(float z, float bias, float low) {
     float s = 1.0f / (1.0f + expf(-(z + bias)));
     return fmaf(1.0f - low, s, low);
 }
-__device__ __forceinline__ float update(float s, float f, float write, float v) { return fmaf(f, s, __fmul_rn(write, v)); }
+// two rows of a column: f s + (1 - f) v
+__device__ __forceinline__ pair_t update(pair_t s, pair_t f, pair_t write, pair_t v) { return fma2(f, s, mul2(write, v)); }
+// two neighbouring rows of a column, from n on, of which `rows` exist (an even number of rows is read and written in pairs)
+__device__ __forceinline__ pair_t load_rows(const float* column, int n, int rows) {
+    if (n >= rows) return 0ull;
+    if (rows % 2 == 0) return *reinterpret_cast<const pair_t*>(column + n);
+    return pack2(column[n], n + 1 < rows ? column[n + 1] : 0.f);
+}
+__device__ __forceinline__ void store_rows(float* column, int n, int rows, pair_t v) {
+    if (n >= rows) return;
+    if (rows % 2 == 0) { *reinterpret_cast<pair_t*>(column + n) = v; return; }
+    float lo, hi;
+    unpack2(v, lo, hi);
+    column[n] = lo;
+    if (n + 1 < rows) column[n + 1] = hi;
+}
 
 template <typename T, int VEC>
 __global__ void __launch_bounds__(THREADS)
@@ -61,7 +77,7 @@ forget_prepare_kernel(const T* __restrict__ proj, int ld, const float* __restric
     }
 }
 
-// PER: state rows a lane holds of each column (D <= 32 * PER). A block: WARPS warps of COLS columns each, the columns
+// PER: pairs of state rows a lane holds of each column (D <= 64 * PER). A block: WARPS warps of COLS columns each, the columns
 // [blockIdx.x * TILE, + TILE) of head blockIdx.y for sequence blockIdx.z.
 template <int PER, int COLS, int WARPS>
 __global__ void __launch_bounds__(WARPS * 32)
@@ -71,7 +87,7 @@ forget_scan_kernel(const float* __restrict__ work, int work_ld, float* __restric
     constexpr int TILE = WARPS * COLS;         // columns a block holds
     constexpr int GROUP = 32 / COLS;           // tokens whose partial sums meet in one butterfly
     constexpr int CHUNK = GROUP > 8 ? GROUP : 8;   // tokens staged at a time
-    extern __shared__ __align__(16) float staged[];      // [2][CHUNK][row]: f (D) | q (D) | v (TILE)
+    extern __shared__ __align__(16) float staged[];      // [2][CHUNK][row]: f (E) | q (E) | v (TILE), E: D rounded up to even
     griddep_launch();
     griddep_wait();
     int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -79,16 +95,14 @@ forget_scan_kernel(const float* __restrict__ work, int work_ld, float* __restric
     int tile0 = blockIdx.x * TILE, v0 = tile0 + warp * COLS;
     int first = cu_seqlens[seq], n_new = cu_seqlens[seq + 1] - first;
     if (n_new <= 0) return;
-    const int row = (2 * D + TILE + 3) / 4 * 4;
+    const int E = (D + 1) & ~1, row = (2 * E + TILE + 3) / 4 * 4;
     const int keys = H * D, f_at = head * D, q_at = keys + head * D, v_at = 2 * keys + head * V + tile0;
     float* S = state + (long long)slot_ids[seq] * state_stride + (size_t)head * D * V;   // [V, D]
-    float s[PER][COLS];
+    pair_t s[PER][COLS];
 #pragma unroll
-    for (int i = 0; i < PER; ++i) {
-        int n = lane + 32 * i;
+    for (int i = 0; i < PER; ++i)
 #pragma unroll
-        for (int c = 0; c < COLS; ++c) s[i][c] = (n < D && v0 + c < V) ? S[(size_t)(v0 + c) * D + n] : 0.f;
-    }
+        for (int c = 0; c < COLS; ++c) s[i][c] = v0 + c < V ? load_rows(S + (size_t)(v0 + c) * D, 2 * lane + 64 * i, D) : 0ull;
     auto request = [&](int chunk) {
         float* to = staged + (chunk & 1) * CHUNK * row;
         int t0 = chunk * CHUNK, count = min(CHUNK, n_new - t0);
@@ -108,31 +122,41 @@ forget_scan_kernel(const float* __restrict__ work, int work_ld, float* __restric
                 const float* from = work + (size_t)(first + t0 + t) * work_ld;
                 float* row_to = to + t * row;
                 for (int r = threadIdx.x; r < 2 * D; r += WARPS * 32)
-                    copy4(row_to + r, from + (r < D ? f_at + r : q_at + r - D));
+                    copy4(row_to + (r < D ? r : E + r - D), from + (r < D ? f_at + r : q_at + r - D));
                 for (int r = threadIdx.x; r < TILE; r += WARPS * 32)
-                    if (tile0 + r < V) copy4(row_to + 2 * D + r, from + v_at + r);
+                    if (tile0 + r < V) copy4(row_to + 2 * E + r, from + v_at + r);
             }
         }
         copies_commit();
     };
     // one token of a group: fade, write, and the lane's share of S q for each column
     auto token = [&](const float* tok, float (&sums)[32], int j, bool live) {
-        float v[COLS];
+        pair_t v[COLS], acc[COLS];
 #pragma unroll
-        for (int c = 0; c < COLS; ++c) v[c] = (live && v0 + c < V) ? tok[2 * D + warp * COLS + c] : 0.f;
-#pragma unroll
-        for (int c = 0; c < COLS; ++c) sums[j * COLS + c] = 0.f;
+        for (int c = 0; c < COLS; ++c) {
+            float value = (live && v0 + c < V) ? tok[2 * E + warp * COLS + c] : 0.f;
+            v[c] = pack2(value, value);
+            acc[c] = 0ull;
+        }
 #pragma unroll
         for (int i = 0; i < PER; ++i) {
-            int n = lane + 32 * i;
-            bool in = live && n < D;
-            float f = in ? tok[n] : 1.f, q = in ? tok[D + n] : 0.f;      // (beyond the step: nothing fades or is written)
-            float write = 1.0f - f;
+            int n = 2 * lane + 64 * i;
+            // (beyond the step or the state nothing fades, is written or read)
+            float2 f = live && n < D ? *reinterpret_cast<const float2*>(tok + n) : make_float2(1.f, 1.f);
+            float2 q = live && n < D ? *reinterpret_cast<const float2*>(tok + E + n) : make_float2(0.f, 0.f);
+            if (n + 1 >= D) { f.y = 1.f; q.y = 0.f; }
+            pair_t ff = pack2(f.x, f.y), qq = pack2(q.x, q.y), write = pack2(1.0f - f.x, 1.0f - f.y);
 #pragma unroll
             for (int c = 0; c < COLS; ++c) {
-                s[i][c] = update(s[i][c], f, write, v[c]);
-                sums[j * COLS + c] = fmaf(s[i][c], q, sums[j * COLS + c]);
+                s[i][c] = update(s[i][c], ff, write, v[c]);
+                acc[c] = fma2(s[i][c], qq, acc[c]);
             }
+        }
+#pragma unroll
+        for (int c = 0; c < COLS; ++c) {
+            float even, odd;
+            unpack2(acc[c], even, odd);
+            sums[j * COLS + c] = even + odd;
         }
     };
     int n_chunks = (n_new + CHUNK - 1) / CHUNK;
@@ -164,12 +188,10 @@ forget_scan_kernel(const float* __restrict__ work, int work_ld, float* __restric
         __syncthreads();                   // the stage is requested again two chunks on
     }
 #pragma unroll
-    for (int i = 0; i < PER; ++i) {
-        int n = lane + 32 * i;
+    for (int i = 0; i < PER; ++i)
 #pragma unroll
         for (int c = 0; c < COLS; ++c)
-            if (n < D && v0 + c < V) S[(size_t)(v0 + c) * D + n] = s[i][c];
-    }
+            if (v0 + c < V) store_rows(S + (size_t)(v0 + c) * D, 2 * lane + 64 * i, D, s[i][c]);
 }
 
 // The factor of a head's norm: a warp sums the squares, its lanes the elements in strides of 32.
@@ -203,41 +225,53 @@ forget_step_kernel(const T* __restrict__ proj, int ld, const float* __restrict__
                    float* __restrict__ state, long long state_stride, const int* __restrict__ cu_seqlens,
                    const int* __restrict__ slot_ids, const float* __restrict__ weight, float eps, T* __restrict__ mixed,
                    int mixed_ld, int H, int D, int V) {
-    extern __shared__ __align__(16) float shared[];      // f (D) | q (D) | v (V) | o (V)
+    extern __shared__ __align__(16) float shared[];      // f (E) | q (E) | v (V) | o (V), E: D rounded up to even
     griddep_launch();
     int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     int head = blockIdx.x, seq = blockIdx.y, v0 = warp * STEP_COLS;
     size_t t = cu_seqlens[seq];
     float* S = state + (long long)slot_ids[seq] * state_stride + (size_t)head * D * V;   // [V, D]
-    float s[PER][STEP_COLS];
+    pair_t s[PER][STEP_COLS];
 #pragma unroll
-    for (int i = 0; i < PER; ++i) {
-        int n = lane + 32 * i;
+    for (int i = 0; i < PER; ++i)
 #pragma unroll
-        for (int c = 0; c < STEP_COLS; ++c) s[i][c] = (n < D && v0 + c < V) ? S[(size_t)(v0 + c) * D + n] : 0.f;
-    }
+        for (int c = 0; c < STEP_COLS; ++c) s[i][c] = v0 + c < V ? load_rows(S + (size_t)(v0 + c) * D, 2 * lane + 64 * i, D) : 0ull;
     griddep_wait();
     const T* in = proj + t * ld;
-    int keys = H * D;
+    int keys = H * D, E = (D + 1) & ~1;
     for (int c = threadIdx.x; c < 2 * D + V; c += blockDim.x) {
         if (c < D) shared[c] = forget(to_float(in[keys + head * D + c]), bias[head * D + c], lower[head * D + c]);
-        else if (c < 2 * D) shared[c] = silu(to_float(in[head * D + c - D]));
-        else shared[c] = to_float(in[2 * keys + head * V + c - 2 * D]);
+        else if (c < 2 * D) shared[E + c - D] = silu(to_float(in[head * D + c - D]));
+        else shared[2 * E + c - 2 * D] = to_float(in[2 * keys + head * V + c - 2 * D]);
     }
     __syncthreads();
-    float sums[STEP_COLS], v[STEP_COLS];
+    float sums[STEP_COLS];
+    pair_t v[STEP_COLS], acc[STEP_COLS];
 #pragma unroll
-    for (int c = 0; c < STEP_COLS; ++c) { sums[c] = 0.f; v[c] = v0 + c < V ? shared[2 * D + v0 + c] : 0.f; }
+    for (int c = 0; c < STEP_COLS; ++c) {
+        float value = v0 + c < V ? shared[2 * E + v0 + c] : 0.f;
+        v[c] = pack2(value, value);
+        acc[c] = 0ull;
+    }
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
-        int n = lane + 32 * i;
-        float f = n < D ? shared[n] : 1.f, q = n < D ? shared[D + n] : 0.f, write = 1.0f - f;
+        int n = 2 * lane + 64 * i;
+        float2 f = n < D ? *reinterpret_cast<const float2*>(shared + n) : make_float2(1.f, 1.f);
+        float2 q = n < D ? *reinterpret_cast<const float2*>(shared + E + n) : make_float2(0.f, 0.f);
+        if (n + 1 >= D) { f.y = 1.f; q.y = 0.f; }
+        pair_t ff = pack2(f.x, f.y), qq = pack2(q.x, q.y), write = pack2(1.0f - f.x, 1.0f - f.y);
 #pragma unroll
         for (int c = 0; c < STEP_COLS; ++c) {
-            s[i][c] = update(s[i][c], f, write, v[c]);
-            sums[c] = fmaf(s[i][c], q, sums[c]);
-            if (n < D && v0 + c < V) S[(size_t)(v0 + c) * D + n] = s[i][c];
+            s[i][c] = update(s[i][c], ff, write, v[c]);
+            acc[c] = fma2(s[i][c], qq, acc[c]);
+            if (v0 + c < V) store_rows(S + (size_t)(v0 + c) * D, n, D, s[i][c]);
         }
+    }
+#pragma unroll
+    for (int c = 0; c < STEP_COLS; ++c) {
+        float even, odd;
+        unpack2(acc[c], even, odd);
+        sums[c] = even + odd;
     }
     // eight sums over the lanes: the same tree of lane pairs as in the scan
     fold<4, 16>(sums, lane);
@@ -246,7 +280,7 @@ forget_step_kernel(const T* __restrict__ proj, int ld, const float* __restrict__
     float total = sums[0];
     total += __shfl_xor_sync(0xffffffffu, total, 2);
     total += __shfl_xor_sync(0xffffffffu, total, 1);
-    float* o = shared + 2 * D + V;
+    float* o = shared + 2 * E + V;
     if ((lane & 3) == 0 && v0 + (lane >> 2) < V) o[v0 + (lane >> 2)] = total;
     __syncthreads();
     float factor = head_factor(o, V, eps);
@@ -268,25 +302,25 @@ LLMB_EXPORT int llmb_forget_recurrence(const void* proj, int ld, int dtype, cons
     if (n_tokens == 0) return LLMB_OK;
     LLMB_REQUIRE(H > 0 && D > 0 && V > 0 && D <= 512, "forget_recurrence: %d heads with states of %d x %d (up to 512 rows are built)", H, D, V);
     LLMB_REQUIRE(n_seqs > 0 && n_seqs <= 65535 && H <= 65535, "forget_recurrence: bad sizes");
-    LLMB_REQUIRE(ld >= 2 * H * D + H * V && work_ld >= 2 * H * D + H * V && state_stride >= (long long)H * D * V,
-                 "forget_recurrence: rows too short");
+    LLMB_REQUIRE(ld >= 2 * H * D + H * V && work_ld >= 2 * H * D + H * V && state_stride >= (long long)H * D * V &&
+                 (D % 2 || (state_stride % 2 == 0 && ((size_t)state % 8) == 0)),
+                 "forget_recurrence: rows too short (or a state of an even number of rows off an 8-byte boundary)");
     LLMB_REQUIRE(dtype == LLMB_DTYPE_F32 || dtype == LLMB_DTYPE_BF16, "forget_recurrence: unknown dtype %d", dtype);
     typedef __nv_bfloat16 B;
     int warps = ceil_div(V, STEP_COLS);
     // (1,024 threads leave 64 registers each: wide states of many rows take the other form)
     if (single && n_tokens == n_seqs && warps <= 32 && D <= 256 && !(D > 128 && warps > 16)) {
-        size_t smem = sizeof(float) * (size_t)(2 * D + 2 * V);
+        size_t smem = sizeof(float) * (size_t)(2 * D + 2 + 2 * V);
 #define LLMB_STEP_AS(T, PER, MOST)                                                                                        \
         LLMB_CUDA(llmb::launch(forget_step_kernel<T, PER, MOST>, dim3(H, n_seqs), dim3(warps * 32), smem, stream, true,         \
                                (const T*)proj, ld, bias, lower, state, state_stride, cu_seqlens, slot_ids, weight, eps,   \
                                (T*)mixed, mixed_ld, H, D, V))
 #define LLMB_STEP(T)                                  \
         do {                                          \
-            if (D <= 32) LLMB_STEP_AS(T, 1, 1024);    \
-            else if (D <= 64) LLMB_STEP_AS(T, 2, 1024); \
-            else if (D <= 128 && warps > 16) LLMB_STEP_AS(T, 4, 1024); \
-            else if (D <= 128) LLMB_STEP_AS(T, 4, 512); \
-            else LLMB_STEP_AS(T, 8, 512);             \
+            if (D <= 64) LLMB_STEP_AS(T, 1, 1024);    \
+            else if (D <= 128 && warps > 16) LLMB_STEP_AS(T, 2, 1024); \
+            else if (D <= 128) LLMB_STEP_AS(T, 2, 512); \
+            else LLMB_STEP_AS(T, 4, 512);             \
         } while (0)
         if (dtype == LLMB_DTYPE_F32) LLMB_STEP(float); else LLMB_STEP(B);
 #undef LLMB_STEP
@@ -307,7 +341,7 @@ LLMB_EXPORT int llmb_forget_recurrence(const void* proj, int ld, int dtype, cons
     int cols = few ? 8 : 2, scan_warps = few ? 4 : 16;
     int tile = scan_warps * cols, chunk = 32 / cols > 8 ? 32 / cols : 8;
     dim3 grid(ceil_div(V, tile), H, n_seqs);
-    size_t smem = sizeof(float) * 2 * chunk * ((2 * D + tile + 3) / 4 * 4);
+    size_t smem = sizeof(float) * 2 * chunk * ((2 * ((D + 1) & ~1) + tile + 3) / 4 * 4);
     int vectors = D % 4 == 0 && V % 4 == 0 && work_ld % 4 == 0 && ((size_t)work % 16) == 0;
 #define LLMB_SCAN_AS(PER, COLS, WARPS)                                                                                    \
     do {                                                                                                                  \
@@ -322,11 +356,10 @@ LLMB_EXPORT int llmb_forget_recurrence(const void* proj, int ld, int dtype, cons
         if (few) LLMB_SCAN_AS(PER, 8, 4);                   \
         else LLMB_SCAN_AS(PER, 2, 16);                      \
     } while (0)
-    if (D <= 32) LLMB_SCAN(1);
-    else if (D <= 64) LLMB_SCAN(2);
-    else if (D <= 128) LLMB_SCAN(4);
-    else if (D <= 256) LLMB_SCAN(8);
-    else LLMB_SCAN_AS(16, 8, 4);
+    if (D <= 64) LLMB_SCAN(1);
+    else if (D <= 128) LLMB_SCAN(2);
+    else if (D <= 256) LLMB_SCAN(4);
+    else LLMB_SCAN_AS(8, 8, 4);
 #undef LLMB_SCAN
 #undef LLMB_SCAN_AS
     if (dtype == LLMB_DTYPE_F32)

@@ -711,19 +711,29 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __nv
         const bool live = lane < NH && head0 + lane < H;
         const __nv_bfloat16* row_q = q + ((size_t)seq * H + head0 + (live ? lane : 0)) * (C + R);
 #pragma unroll 1
-        for (int c = 0; c < pieces; ++c) {
-            uint32_t r[32];
+        for (int c0 = 0; c0 < pieces; c0 += 3) {                     // three pieces' loads in flight
+            uint4 v[3][8];
 #pragma unroll
-            for (int i = 0; i < 8; ++i) {
-                uint4 v = make_uint4(0u, 0u, 0u, 0u);
-                if (live && c * 64 + i * 8 < C + R) v = *reinterpret_cast<const uint4*>(row_q + c * 64 + i * 8);
-                r[4 * i] = v.x; r[4 * i + 1] = v.y; r[4 * i + 2] = v.z; r[4 * i + 3] = v.w;
+            for (int c = 0; c < 3; ++c)
+#pragma unroll
+                for (int i = 0; i < 8; ++i) {
+                    int at = (c0 + c) * 64 + i * 8;
+                    v[c][i] = live && at < C + R ? *reinterpret_cast<const uint4*>(row_q + at) : make_uint4(0u, 0u, 0u, 0u);
+                }
+#pragma unroll
+            for (int c = 0; c < 3; ++c) {
+                if (c0 + c >= pieces) break;
+#pragma unroll
+                for (int half = 0; half < 2; ++half) {
+                    uint32_t r[16];
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        r[4 * i] = v[c][half * 4 + i].x; r[4 * i + 1] = v[c][half * 4 + i].y;
+                        r[4 * i + 2] = v[c][half * 4 + i].z; r[4 * i + 3] = v[c][half * 4 + i].w;
+                    }
+                    tmem_st16(tmem_base + Q_COL + (c0 + c) * 32 + half * 16, r);
+                }
             }
-            uint32_t lo[16], hi[16];
-#pragma unroll
-            for (int i = 0; i < 16; ++i) { lo[i] = r[i]; hi[i] = r[16 + i]; }
-            tmem_st16(tmem_base + Q_COL + c * 32, lo);
-            tmem_st16(tmem_base + Q_COL + c * 32 + 16, hi);
         }
         tmem_st_wait();
         tcgen05_fence_before();
@@ -870,29 +880,33 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __nv
 }  // namespace decode
 
 // block (row): the slices' weighted values, maxima (base-2 units) and sums merged in slice order
+constexpr int MAX_SPLITS = 32;
 __global__ void __launch_bounds__(128)
 latent_combine_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_stats, __nv_bfloat16* __restrict__ out,
                       int C, int n_splits) {
     griddep_launch();
     griddep_wait();
+    __shared__ float shares[MAX_SPLITS];
     size_t row = blockIdx.x;
-    float m = -INFINITY, total = 0.f;
-    for (int s = 0; s < n_splits; ++s) m = fmaxf(m, part_stats[(row * n_splits + s) * 2]);
-    for (int s = 0; s < n_splits; ++s) {
-        float ms = part_stats[(row * n_splits + s) * 2];
-        total += ms == -INFINITY ? 0.f : part_stats[(row * n_splits + s) * 2 + 1] * exp2f(ms - m);
+    const float* stats = part_stats + row * n_splits * 2;
+    if (threadIdx.x < 32) {                                // a lane a slice: its share of the result
+        int s = threadIdx.x;
+        float ms = s < n_splits ? stats[2 * s] : -INFINITY, m = warp_max(ms);
+        float weight = ms == -INFINITY ? 0.f : exp2f(ms - m);
+        float total = warp_sum(s < n_splits ? stats[2 * s + 1] * weight : 0.f);
+        if (s < n_splits) shares[s] = weight / total;
     }
-    float inv = 1.0f / total;
+    __syncthreads();
     for (int c = threadIdx.x * 4; c < C; c += 128 * 4) {
         float v[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 8
         for (int s = 0; s < n_splits; ++s) {
-            float ms = part_stats[(row * n_splits + s) * 2];
-            float weight = ms == -INFINITY ? 0.f : exp2f(ms - m);
             float4 a = *reinterpret_cast<const float4*>(part_acc + (row * n_splits + s) * C + c);
-            v[0] = fmaf(a.x, weight, v[0]); v[1] = fmaf(a.y, weight, v[1]);
-            v[2] = fmaf(a.z, weight, v[2]); v[3] = fmaf(a.w, weight, v[3]);
+            float share = shares[s];
+            v[0] = fmaf(a.x, share, v[0]); v[1] = fmaf(a.y, share, v[1]);
+            v[2] = fmaf(a.z, share, v[2]); v[3] = fmaf(a.w, share, v[3]);
         }
-        __nv_bfloat162 lo = __floats2bfloat162_rn(v[0] * inv, v[1] * inv), hi = __floats2bfloat162_rn(v[2] * inv, v[3] * inv);
+        __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
         *reinterpret_cast<uint2*>(out + row * C + c) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
     }
 }
@@ -933,7 +947,7 @@ LLMB_EXPORT int llmb_latent_attention(const void* q, const void* cache, const in
     if (n_seqs == 0 || max_new == 0) return LLMB_OK;
     LLMB_REQUIRE(H > 0 && C > 0 && R > 0 && C % 8 == 0 && R % 8 == 0 && C <= 512 && C + R <= 640,
                  "latent_attention: rows of %d + %d (multiples of 8, up to 512 and 640 in all)", C, R);
-    LLMB_REQUIRE(n_seqs <= 65535 && ring_pages > 0 && n_splits >= 1 && scale > 0.f, "latent_attention: bad sizes");
+    LLMB_REQUIRE(n_seqs <= 65535 && ring_pages > 0 && n_splits >= 1 && n_splits <= MAX_SPLITS && scale > 0.f, "latent_attention: bad sizes");
     LLMB_REQUIRE(((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(out)) & 15) == 0,
                  "latent_attention: operands must be 16-byte aligned");
     LLMB_REQUIRE(n_splits == 1 || (scratch && scratch_floats >= llmb_latent_scratch_floats(n_tokens, H, C, n_splits)),
@@ -994,7 +1008,7 @@ LLMB_EXPORT int llmb_latent_decode_tc(const void* q, const void* cache, int n_pa
     if (n_seqs == 0) return LLMB_OK;
     LLMB_REQUIRE(H > 0 && (C == 64 || C == 128 || C == 256 || C == 512) && R > 0 && R <= 64 && R % 8 == 0,
                  "latent_decode_tc: rows of %d + %d (64, 128, 256 or 512, a multiple of 8 up to 64)", C, R);
-    LLMB_REQUIRE(n_seqs <= 65535 && n_pages > 0 && ring_pages > 0 && n_splits >= 1 && scale > 0.f, "latent_decode_tc: bad sizes");
+    LLMB_REQUIRE(n_seqs <= 65535 && n_pages > 0 && ring_pages > 0 && n_splits >= 1 && n_splits <= MAX_SPLITS && scale > 0.f, "latent_decode_tc: bad sizes");
     LLMB_REQUIRE(((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(out)) & 15) == 0,
                  "latent_decode_tc: operands must be 16-byte aligned");
     LLMB_REQUIRE(n_splits == 1 || (scratch && scratch_floats >= llmb_latent_scratch_floats(n_seqs, H, C, n_splits)),

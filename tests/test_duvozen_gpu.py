@@ -154,7 +154,7 @@ def _recurrence_inputs(H, D, V, n, slots, dtype, seed):
     bias = (1.0 + 2.0 * torch.randn(H * D, generator=gen)).to(DEV)
     lower = (0.9 * torch.rand(H * D, generator=gen)).to(DEV)
     weight = (1.0 + 0.3 * torch.randn(V, generator=gen)).to(DEV)
-    state = torch.randn((slots, H * D * V + 3), generator=gen).to(DEV)
+    state = torch.randn((slots, H * D * V + 4), generator=gen).to(DEV)
     return proj, bias, lower, weight, state
 
 
