@@ -72,6 +72,13 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_float<__nv_bfloat16>(f
 }
 
 __device__ __forceinline__ void griddep_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+// The same pointer, known to the compiler only from here on. What the kernel in front wrote is to be read through it, behind
+// griddep_wait(): through a const __restrict__ parameter the compiler may take the data for constant during the kernel and
+// move the load in front of the wait (a load in the wait's own basic block did move).
+template <typename T> __device__ __forceinline__ const T* behind_wait(const T* p) {
+    asm volatile("" : "+l"(p) : : "memory");
+    return p;
+}
 __device__ __forceinline__ void griddep_launch() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
 
 __device__ __forceinline__ float warp_sum(float v) {

@@ -55,6 +55,7 @@ forget_prepare_kernel(const T* __restrict__ proj, int ld, const float* __restric
                       float* __restrict__ work, int work_ld, int keys, int values) {
     griddep_launch();
     griddep_wait();
+    proj = behind_wait(proj);
     size_t t = blockIdx.x;
     const T* in = proj + t * ld;
     float* out = work + t * work_ld;
@@ -90,6 +91,7 @@ forget_scan_kernel(const float* __restrict__ work, int work_ld, float* __restric
     extern __shared__ __align__(16) float staged[];      // [2][CHUNK][row]: f (E) | q (E) | v (TILE), E: D rounded up to even
     griddep_launch();
     griddep_wait();
+    work = behind_wait(work);
     int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     int head = blockIdx.y, seq = blockIdx.z;
     int tile0 = blockIdx.x * TILE, v0 = tile0 + warp * COLS;
@@ -208,6 +210,7 @@ forget_finish_kernel(const float* __restrict__ o, const float* __restrict__ weig
                      int mixed_ld, int H, int V) {
     griddep_launch();
     griddep_wait();
+    o = behind_wait(o);
     size_t t = blockIdx.x;
     for (int head = threadIdx.x >> 5; head < H; head += THREADS / 32) {
         const float* row = o + t * H * V + head * V;
@@ -237,6 +240,7 @@ forget_step_kernel(const T* __restrict__ proj, int ld, const float* __restrict__
 #pragma unroll
         for (int c = 0; c < STEP_COLS; ++c) s[i][c] = v0 + c < V ? load_rows(S + (size_t)(v0 + c) * D, 2 * lane + 64 * i, D) : 0ull;
     griddep_wait();
+    proj = behind_wait(proj);
     const T* in = proj + t * ld;
     int keys = H * D, E = (D + 1) & ~1;
     for (int c = threadIdx.x; c < 2 * D + V; c += blockDim.x) {

@@ -133,6 +133,7 @@ head_products_kernel(const T* __restrict__ x, int ldx, int x_head, const T* __re
     __shared__ float xs[16][33], ws[64][33];
     griddep_launch();
     griddep_wait();
+    x = behind_wait(x);
     int head = blockIdx.z, t0 = blockIdx.y * 16, n0 = blockIdx.x * 64;
     const T* wh = w + (size_t)head * N * K;
     int tx = threadIdx.x & 63, ty = threadIdx.x >> 6;          // output n0 + tx of the tokens ty, ty + 4, ..
@@ -709,7 +710,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __nv
         griddep_wait();
         // the queries, a lane a head, into tensor memory (zeros beyond the head count and beyond the row)
         const bool live = lane < NH && head0 + lane < H;
-        const __nv_bfloat16* row_q = q + ((size_t)seq * H + head0 + (live ? lane : 0)) * (C + R);
+        const __nv_bfloat16* row_q = behind_wait(q) + ((size_t)seq * H + head0 + (live ? lane : 0)) * (C + R);
 #pragma unroll 1
         for (int c0 = 0; c0 < pieces; c0 += 3) {                     // three pieces' loads in flight
             uint4 v[3][8];
@@ -886,6 +887,8 @@ latent_combine_kernel(const float* __restrict__ part_acc, const float* __restric
                       int C, int n_splits) {
     griddep_launch();
     griddep_wait();
+    part_acc = behind_wait(part_acc);
+    part_stats = behind_wait(part_stats);
     __shared__ float shares[MAX_SPLITS];
     size_t row = blockIdx.x;
     const float* stats = part_stats + row * n_splits * 2;

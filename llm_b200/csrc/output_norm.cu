@@ -75,6 +75,7 @@ layernorm_kernel(const float* __restrict__ x, const float* __restrict__ gain, co
     __shared__ float scratch[THREADS / 32];
     griddep_launch();
     griddep_wait();
+    x = behind_wait(x);
     size_t r = blockIdx.x;
     const float* in = x + (size_t)(rows ? rows[r] : (int)r) * width;
     float total = 0.f, mean, factor;
@@ -105,6 +106,8 @@ output_norm_add_kernel(const float* __restrict__ y, int terms, const float* __re
     __shared__ float scratch[THREADS / 32];
     griddep_launch();
     griddep_wait();
+    y = behind_wait(y);
+    extra = behind_wait(extra);
     size_t t = blockIdx.x;
     float total = 0.f, mean, factor;
     for (int c = threadIdx.x * VEC; c < width; c += THREADS * VEC) {
@@ -163,6 +166,7 @@ input_conv_kernel(const float* __restrict__ x, const float* __restrict__ taps, i
                   TOut* __restrict__ h, int width) {
     griddep_launch();
     griddep_wait();
+    x = behind_wait(x);
     const int K = TAPS > 0 ? TAPS : n_taps;
     int b = blockIdx.z, c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
     int first = cu_seqlens[b], n = cu_seqlens[b + 1] - first;
@@ -177,19 +181,26 @@ input_conv_kernel(const float* __restrict__ x, const float* __restrict__ taps, i
         for (int j = 0; j < TAPS; ++j) w[j] = load<VEC>(taps + (size_t)j * width + c);
 #pragma unroll
         for (int j = 1; j < TAPS; ++j) held[j] = row_at(begin - TAPS + j);
-        for (int i = begin; i < end; ++i) {
+        for (int i0 = begin; i0 < end; i0 += 4) {
+            Pack<VEC> rows[4];                                // four rows in flight
 #pragma unroll
-            for (int j = 0; j + 1 < TAPS; ++j) held[j] = held[j + 1];
-            held[TAPS - 1] = row_at(i);
-            Pack<VEC> out;
+            for (int k = 0; k < 4; ++k) rows[k] = row_at(min(i0 + k, end - 1));
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) {
-                float acc = 0.f;
+            for (int k = 0; k < 4; ++k) {
+                if (i0 + k >= end) break;
 #pragma unroll
-                for (int j = 0; j < TAPS; ++j) acc = fmaf(w[j].v[e], held[j].v[e], acc);
-                out.v[e] = held[TAPS - 1].v[e] + acc;
+                for (int j = 0; j + 1 < TAPS; ++j) held[j] = held[j + 1];
+                held[TAPS - 1] = rows[k];
+                Pack<VEC> out;
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) {
+                    float acc = 0.f;
+#pragma unroll
+                    for (int j = 0; j < TAPS; ++j) acc = fmaf(w[j].v[e], held[j].v[e], acc);
+                    out.v[e] = held[TAPS - 1].v[e] + acc;
+                }
+                store(h + (size_t)(first + i0 + k) * width + c, out);
             }
-            store(h + (size_t)(first + i) * width + c, out);
         }
     } else {
         for (int i = begin; i < end; ++i) {
@@ -216,6 +227,7 @@ template <typename TOut>
 __global__ void cast_kernel(const float* __restrict__ x, TOut* __restrict__ h, long long n) {
     griddep_launch();
     griddep_wait();
+    x = behind_wait(x);
     long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i < n) h[i] = from_float<TOut>(x[i]);
 }

@@ -687,6 +687,29 @@ def test_dense_feed_forwards_in_both_dtypes(tmp_path, dtype):
     engine.check()
 
 
+@pytest.mark.parametrize("heads", [8, 24, 40])
+@pytest.mark.parametrize("rank", [64, 128, 256, 512])
+def test_decode_steps_whose_kernels_follow_closely(tmp_path, heads, rank):
+    """A model of latent layers alone, decoded as a batch through captured steps: every kernel starts while the one in
+    front of it ends, so a load in front of the wait for it would read the step before."""
+    from llm_b200.engine import Entry
+    from tiny_duvozen import _latent
+
+    def latent_only(config):
+        config["layers"] = [{"type": "latent_attention", "mlp": None,
+                             "mixer": _latent(heads, 64, 64, 24, rank, 10000.0, (4.0, 100, 8.0, 1.0))}] * 2
+    config, weights, engine = _setup(tmp_path, "Q", torch.bfloat16, latent_only)
+    lengths = (129, 190, 40)
+    seqs = [random_tokens(n + 12, config["vocab"], n) for n in lengths]
+    expected = [plain.forward(config, weights, s) for s in seqs]
+    slots = engine.acquire(3)
+    engine.step([Entry(s, q[:n], []) for s, q, n in zip(slots, seqs, lengths)])
+    for k in range(12):
+        logits = engine.step([Entry(s, [q[n + k]], [0]) for s, q, n in zip(slots, seqs, lengths)])
+        _check_logits(logits, torch.stack([e[n + k] for e, n in zip(expected, lengths)]), torch.bfloat16, k)
+    assert engine.graph_replays > 5
+
+
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 def test_long_decoding_passes_page_edges(tmp_path, dtype):
     """One token a step from the first on, 300 steps: pages fill and follow each other, the recurrences' states and the
