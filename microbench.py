@@ -9,6 +9,11 @@
     python microbench.py gated_recurrence --batch 1 --tokens 2048 --k 4096
     python microbench.py routed_experts --m 2048 --k 4096 --n 1792 --experts 32 --top 8 [--variant narrow|wide128]
     python microbench.py norm_add --m 2048 --k 4096 --top 8
+    python microbench.py forget_recurrence --batch 64 --tokens 1
+    python microbench.py latent_attention --batch 64 --tokens 1 --context 8192 [--rank 256 --rot 32]
+    python microbench.py latent_prefill | latent_write | head_products --batch 1 --tokens 2048
+    python microbench.py output_norm --m 8 --tokens 1 --top 8        # --tokens 1: with the next part's input
+    python microbench.py input_conv --m 2048
     LLMB_NVCC_FLAGS=-DLLMB_TRACE python microbench.py linear --m 8 --n 6144 --k 4096 --timeline
     LLMB_NVCC_FLAGS=-DLLMB_TRACE python microbench.py attention_prefill --tokens 2048 --timeline
 
