@@ -30,7 +30,8 @@
 // * optional, applied where the result is written (by the block itself with one slice, else by the
 //   combining kernel), in 32-bit: `sinks` [heads] (e^sink joins the head's denominator), `gate`
 //   [sequences, heads] (times sigmoid(gate)), `out_scale`. When the value cache IS the key cache, a
-//   page is fetched once and both products read the same tile.
+//   page is fetched once and both products read the same tile;
+// * `bias` [heads, span]: bias[h, min(distance, span - 1)] is added to the scaled score.
 //
 // Refused (the generic kernel serves them): head sizes other than 32, 64, 96, 128, 32-bit caches.
 #include "common.cuh"
@@ -88,7 +89,7 @@ attention_decode_split_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
                               __nv_bfloat16* __restrict__ out, int out_stride,
                               int n_heads, int n_kv_heads, float scale_log2, int window, int chunks,
                               const float* __restrict__ sinks, const __nv_bfloat16* __restrict__ gate,
-                              int gate_stride, float out_scale, float cap_log2) {
+                              int gate_stride, float out_scale, float cap_log2, const float* __restrict__ bias, int span) {
     constexpr int LDS = D + PAD;
     const bool values_are_keys = k_cache == v_cache;
     constexpr int PAGE_ELEMS = LLMB_PAGE * LDS;
@@ -180,6 +181,8 @@ attention_decode_split_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
 #pragma unroll
         for (int i = 0; i < 4; ++i) acc[n][i] = 0.f;
     float run_max = -INFINITY, run_sum = 0.f;      // for head row g (this lane's keys only for the sum)
+    const float* near_bias = bias ? bias + (size_t)(head_base + min(g, group - 1)) * span : nullptr;
+    float far_bias = bias ? near_bias[span - 1] * 1.4426950408889634f : 0.f;
 
     for (int i = 0; i < n_units; ++i) {
         // the newest page, fetched late, is in the last unit of its slice and the youngest group
@@ -214,9 +217,14 @@ attention_decode_split_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
         float v[4] = {s0[0], s0[1], s1[0], s1[1]};
         int key[4] = {first_key + 2 * t, first_key + 2 * t + 1, first_key + 8 + 2 * t, first_key + 9 + 2 * t};
         float local_max = -INFINITY;
+        float added[4] = {far_bias, far_bias, far_bias, far_bias};
+        if (bias && len - 1 - (first_key + 15) < span - 1) {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) added[j] = near_bias[max(0, min(len - 1 - key[j], span - 1))] * 1.4426950408889634f;
+        }
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-            float scaled = v[j] * scale_log2;
+            float scaled = fmaf(v[j], scale_log2, added[j]);
             // a soft cap c bounds the scaled score, c tanh(s / c); in base-2 units both carry the factor log2(e)
             if (cap_log2 > 0.f) scaled = cap_log2 * tanhf(scaled / cap_log2);
             v[j] = (key[j] < len && key[j] >= oldest) ? scaled : -INFINITY;
@@ -318,7 +326,7 @@ static int launch(const void* q, int q_stride, const void* k_cache, const void* 
                   const int* block_table, int table_stride, int ring_pages, const int* seq_lens,
                   const int* seq_order, void* out, int out_stride, float* scratch, int n_seqs, int n_heads,
                   int n_kv_heads, float scale, int window, const float* sinks, const void* gate, int gate_stride,
-                  float out_scale, float softcap, int n_splits, cudaStream_t stream) {
+                  float out_scale, float softcap, const float* bias, int span, int n_splits, cudaStream_t stream) {
     constexpr int LDS = D + PAD;
     constexpr int STAGES = stages_for<D>();
     size_t stage_bytes = (size_t)STAGES * pages_per_stage<D>() * 2 * LLMB_PAGE * LDS * sizeof(__nv_bfloat16);
@@ -339,7 +347,7 @@ static int launch(const void* q, int q_stride, const void* k_cache, const void* 
                  (const __nv_bfloat16*)v_cache, block_table, table_stride, ring_pages, seq_lens, seq_order,
                  part_acc, part_stats, (__nv_bfloat16*)out, out_stride, n_heads, n_kv_heads, scale * 1.4426950408889634f,
                  window, chunks, sinks, (const __nv_bfloat16*)gate, gate_stride, out_scale,
-                 softcap > 0.f ? softcap * 1.4426950408889634f : 0.f);
+                 softcap > 0.f ? softcap * 1.4426950408889634f : 0.f, bias, span);
     int code = check_launch("attention_decode_window_split");
     if (code || n_splits == 1) return code;
     llmb::launch(attention_decode_combine_kernel<D>, dim3(n_heads, n_seqs), D >= 128 ? 128 : 64, 0, stream, true,
@@ -374,7 +382,8 @@ LLMB_EXPORT int llmb_attention_decode_window(const void* q, int q_stride, const 
                                       int out_stride, float* scratch, long long scratch_floats, int n_seqs,
                                       int n_heads, int n_kv_heads, int head_dim, float scale,
                                       int window, const float* sinks, const void* gate, int gate_stride,
-                                      float out_scale, float softcap, int n_splits, cudaStream_t stream) {
+                                      float out_scale, float softcap, const float* bias, int span, int n_splits,
+                                      cudaStream_t stream) {
     if (n_seqs == 0) return LLMB_OK;
     int code = llmb_attention_decode_window_supports(n_heads, n_kv_heads, head_dim, window);
     if (code) return code;
@@ -385,9 +394,10 @@ LLMB_EXPORT int llmb_attention_decode_window(const void* q, int q_stride, const 
     LLMB_REQUIRE(scratch != nullptr && scratch_floats >= llmb_attention_decode_window_scratch_floats(
                                                              n_seqs, n_heads, head_dim, n_splits),
                  "attention_decode_window: scratch too small");
+    LLMB_REQUIRE(!bias || (span > 0 && softcap <= 0.f), "attention_decode_window: a bias with a soft cap, or an empty one");
 #define ARGS q, q_stride, k_cache, v_cache, block_table, table_stride, ring_pages, seq_lens, seq_order, out, \
              out_stride, scratch, n_seqs, n_heads, n_kv_heads, scale, window, sinks, gate, gate_stride, out_scale, \
-             softcap, n_splits, stream
+             softcap, bias, span, n_splits, stream
     switch (head_dim) {
         case 32: return launch<32>(ARGS);
         case 64: return launch<64>(ARGS);

@@ -35,6 +35,7 @@ constexpr int WARPS = 4;
 // value cache IS the key cache (a mixer whose cached rows serve as both), a row is loaded once; values narrower
 // than keys are then a row's first elements.
 // `softcap` > 0 bounds a score before the softmax: s <- softcap * tanh(s / softcap), after the scale.
+// `bias` [heads, span]: bias[h, min(p - j, span - 1)] is added to the score of key j behind the scale.
 // Values may be wider or narrower than keys (`value_dim`; the value cache then has rows of that size and
 // the result rows hold n_heads * value_dim elements).
 template <typename T, int AHEAD, int MAX_PER_LANE>
@@ -45,7 +46,7 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, const T* __restr
                          const int* __restrict__ tok_seq, T* __restrict__ out, int out_stride,
                          int n_heads, int n_kv_heads, int head_dim, float scale, int window,
                          const float* __restrict__ sinks, const T* __restrict__ gate, int gate_stride,
-                         float out_scale, float softcap, int value_dim) {
+                         float out_scale, float softcap, int value_dim, const float* __restrict__ bias, int span) {
     int t = blockIdx.x, head = blockIdx.y;
     const bool values_are_keys = k_cache == v_cache;
     int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -95,6 +96,7 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, const T* __restr
             }
             float score = warp_sum(dot) * scale;
             if (softcap > 0.f) score = softcap * tanhf(score / softcap);
+            if (bias) score += bias[(size_t)head * span + min(pos - (j0 + u * WARPS), span - 1)];
             float new_max = fmaxf(running_max, score);
             float rescale = expf(running_max - new_max);    // exp(-inf) = 0 on the first key
             float p = expf(score - new_max);
@@ -149,6 +151,7 @@ LLMB_EXPORT int llmb_attention_generic(const void* q, int q_stride, const void* 
                                        int n_tokens, int n_heads, int n_kv_heads, int head_dim,
                                        float scale, int window, const float* sinks, const void* gate,
                                        int gate_stride, float out_scale, float softcap, int value_dim,
+                                       const float* bias, int span,
                                        cudaStream_t stream) {
     if (n_tokens == 0) return LLMB_OK;
     if (value_dim <= 0) value_dim = head_dim;
@@ -157,7 +160,7 @@ LLMB_EXPORT int llmb_attention_generic(const void* q, int q_stride, const void* 
     LLMB_REQUIRE(k_cache != v_cache || value_dim <= head_dim, "attention_generic: values that are the keys are not longer than they are");
     LLMB_REQUIRE(n_heads > 0 && n_kv_heads > 0 && n_heads % n_kv_heads == 0,
                  "attention_generic: %d heads are no multiple of %d kv heads", n_heads, n_kv_heads);
-    LLMB_REQUIRE(n_heads <= 65535 && ring_pages > 0 && window >= 0, "attention_generic: bad sizes");
+    LLMB_REQUIRE(n_heads <= 65535 && ring_pages > 0 && window >= 0 && (!bias || (span > 0 && softcap <= 0.f)), "attention_generic: bad sizes");
     dim3 grid(n_tokens, n_heads);
     bool few = (long long)n_tokens * n_heads < 4096;       // the result is the same either way
     bool wide = head_dim > LLMB_MAX_HEAD_DIM || value_dim > LLMB_MAX_HEAD_DIM;              // twice the registers a lane: only where the head needs them
@@ -165,7 +168,7 @@ LLMB_EXPORT int llmb_attention_generic(const void* q, int q_stride, const void* 
     attention_generic_kernel<T, AHEAD, PER><<<grid, WARPS * 32, 0, stream>>>(                            \
         (const T*)q, q_stride, (const T*)k_cache, (const T*)v_cache, block_table, table_stride,         \
         ring_pages, tok_pos, tok_seq, (T*)out, out_stride, n_heads, n_kv_heads, head_dim, scale, window, \
-        sinks, (const T*)gate, gate_stride, out_scale, softcap, value_dim)
+        sinks, (const T*)gate, gate_stride, out_scale, softcap, value_dim, bias, span)
 #define LLMB_GENERIC(T, AHEAD)                                                                          \
     do {                                                                                                \
         if (head_dim > 512 || value_dim > 512) LLMB_GENERIC_AS(T, 1, GENERIC_MAX_HEAD_DIM / 32);         \

@@ -28,7 +28,9 @@
 //   element, and a row whose first pages hold nothing it sees keeps a maximum of -inf without NaN.
 // * optional, all in the epilogue and in 32-bit: `sinks` [heads] (e^sink joins the head's
 //   denominator: no key, no value, not scaled), `gate` [T, heads] (the head's result times
-//   sigmoid(gate)), `out_scale`. When the value cache IS the key cache (a mixer whose cached rows
+//   sigmoid(gate)), `out_scale`. `bias` [heads, span]: bias[h, min(p - j, span - 1)] is added to the
+//   scaled score of key j; a page whose keys are all span - 1 or further behind every query of a warp adds one number
+//   inside the exponent's multiply-add. When the value cache IS the key cache (a mixer whose cached rows
 //   serve as both), a page is fetched once and both products read the same tile.
 //
 // Refused (the generic kernel serves them): 32-bit caches, head sizes other than 32, 64, 96, 128.
@@ -51,7 +53,7 @@ __device__ __forceinline__ float fast_exp2(float x) {
     return y;
 }
 
-template <int D>
+template <int D, bool BIAS>
 __global__ void __launch_bounds__(WARPS * 32, 3)          // three blocks per SM: at most 170 registers
 attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
                          const __nv_bfloat16* __restrict__ k_cache,
@@ -61,7 +63,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
                          __nv_bfloat16* __restrict__ out, int out_stride, int n_heads,
                          int n_kv_heads, float scale_log2, int window, const float* __restrict__ sinks,
                          const __nv_bfloat16* __restrict__ gate, int gate_stride, float out_scale,
-                         float cap_raw) {
+                         float cap_raw, const float* __restrict__ bias, int span) {
     constexpr int LDS = D + PAD;
     const bool values_are_keys = k_cache == v_cache;
     constexpr int PAGE_ELEMS = LLMB_PAGE * LDS;
@@ -164,6 +166,25 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
 #pragma unroll
                 for (int i = 0; i < 4; ++i) s[nb][i] = cap_raw * tanhf(s[nb][i] * inv_cap);
         }
+        // A bias by distance: near keys take theirs here, in raw units (the scale is positive); to far ones one number
+        // belongs, which enters where the maxima and the exponents are formed.
+        float far_raw = 0.f;
+        if constexpr (BIAS) {
+            const float* mine = bias + (size_t)head * span;
+            float inv_scale = 1.4426950408889634f / scale_log2;
+            if (start + tile * BQ + warp * 16 - (key0 + LLMB_PAGE - 1) >= span - 1) {
+                far_raw = mine[span - 1] * inv_scale;
+            } else {
+#pragma unroll
+                for (int nb = 0; nb < 8; ++nb)
+#pragma unroll
+                    for (int i = 0; i < 2; ++i) {
+                        int key = key0 + nb * 8 + 2 * t + i;
+                        s[nb][i] = fmaf(mine[max(0, min(pos0 - key, span - 1))], inv_scale, s[nb][i]);
+                        s[nb][2 + i] = fmaf(mine[max(0, min(pos1 - key, span - 1))], inv_scale, s[nb][2 + i]);
+                    }
+            }
+        }
         // Maxima are kept on the raw scores (the scale is positive); the scale and log2(e) are
         // applied inside the exponent with one fused multiply-add per score.
         bool diagonal = key0 + LLMB_PAGE - 1 > start + tile * BQ + warp * 16;   // some key may be hidden
@@ -189,12 +210,13 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
         local1 = fmaxf(local1, __shfl_xor_sync(0xffffffffu, local1, 2));
         // Without a window key 0 is visible to every row, so after page 0 both maxima are finite. With one, a
         // row may have seen nothing yet: its maximum stays -inf, and a reference of 0 keeps every term 0.
+        if constexpr (BIAS) { local0 += far_raw; local1 += far_raw; }
         float new0 = fmaxf(max0, local0), new1 = fmaxf(max1, local1);
         float ref0 = new0 == -INFINITY ? 0.f : new0, ref1 = new1 == -INFINITY ? 0.f : new1;
         float rescale0 = fast_exp2((max0 - ref0) * scale_log2), rescale1 = fast_exp2((max1 - ref1) * scale_log2);
         max0 = new0;
         max1 = new1;
-        float shift0 = ref0 * scale_log2, shift1 = ref1 * scale_log2;
+        float shift0 = (ref0 - far_raw) * scale_log2, shift1 = (ref1 - far_raw) * scale_log2;
         float add0 = 0.f, add1 = 0.f;
 #pragma unroll
         for (int nb = 0; nb < 8; ++nb) {
@@ -272,21 +294,24 @@ static int launch(const void* q, int q_stride, const void* k_cache, const void* 
                   const int* block_table, int table_stride, int ring_pages, const int* cu_seqlens,
                   const int* seq_lens, void* out, int out_stride, int n_seqs, int max_new, int n_heads,
                   int n_kv_heads, float scale, int window, const float* sinks, const void* gate, int gate_stride,
-                  float out_scale, float softcap, cudaStream_t stream) {
+                  float out_scale, float softcap, const float* bias, int span, cudaStream_t stream) {
     constexpr int LDS = D + PAD;
     size_t smem = (size_t)STAGES * 2 * LLMB_PAGE * LDS * sizeof(__nv_bfloat16);
     static bool configured = false;
     if (!configured) {
-        LLMB_CUDA(cudaFuncSetAttribute(attention_prefill_kernel<D>,
+        LLMB_CUDA(cudaFuncSetAttribute(attention_prefill_kernel<D, false>,
+                                       cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        LLMB_CUDA(cudaFuncSetAttribute(attention_prefill_kernel<D, true>,
                                        cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         configured = true;
     }
     dim3 grid(n_heads, (max_new + BQ - 1) / BQ, n_seqs);
-    attention_prefill_kernel<D><<<grid, WARPS * 32, smem, stream>>>(
+    auto kernel = bias ? attention_prefill_kernel<D, true> : attention_prefill_kernel<D, false>;
+    kernel<<<grid, WARPS * 32, smem, stream>>>(
         (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache,
         block_table, table_stride, ring_pages, cu_seqlens, seq_lens, (__nv_bfloat16*)out, out_stride,
         n_heads, n_kv_heads, scale * 1.4426950408889634f, window, sinks, (const __nv_bfloat16*)gate, gate_stride,
-        out_scale, softcap > 0.f ? softcap / scale : 0.f);
+        out_scale, softcap > 0.f ? softcap / scale : 0.f, bias, span);
     return check_launch("attention_prefill");
 }
 
@@ -308,9 +333,11 @@ LLMB_EXPORT int llmb_attention_prefill(const void* q, int q_stride, const void* 
                                        void* out, int out_stride, int n_seqs, int max_new,
                                        int n_heads, int n_kv_heads, int head_dim, float scale,
                                        int window, const float* sinks, const void* gate, int gate_stride,
-                                       float out_scale, float softcap, cudaStream_t stream) {
+                                       float out_scale, float softcap, const float* bias, int span,
+                                       cudaStream_t stream) {
     if (n_seqs == 0 || max_new == 0) return LLMB_OK;
-    LLMB_REQUIRE(softcap <= 0.f || scale > 0.f, "attention_prefill: a soft cap needs a positive scale");
+    LLMB_REQUIRE((softcap <= 0.f && !bias) || scale > 0.f, "attention_prefill: a soft cap or a bias needs a positive scale");
+    LLMB_REQUIRE(!bias || (span > 0 && softcap <= 0.f), "attention_prefill: a bias with a soft cap, or an empty one");
     int code = llmb_attention_prefill_supports(n_heads, n_kv_heads, head_dim, window);
     if (code) return code;
     LLMB_REQUIRE(n_seqs <= 65535 && max_new / BQ < 65535 && ring_pages > 0, "attention_prefill: bad sizes");
@@ -319,7 +346,7 @@ LLMB_EXPORT int llmb_attention_prefill(const void* q, int q_stride, const void* 
                  "attention_prefill: q and out must be 4-byte aligned with even row strides");
 #define ARGS q, q_stride, k_cache, v_cache, block_table, table_stride, ring_pages, cu_seqlens, seq_lens, \
              out, out_stride, n_seqs, max_new, n_heads, n_kv_heads, scale, window, sinks, gate, gate_stride, \
-             out_scale, softcap, stream
+             out_scale, softcap, bias, span, stream
     switch (head_dim) {
         case 32: return launch<32>(ARGS);
         case 64: return launch<64>(ARGS);

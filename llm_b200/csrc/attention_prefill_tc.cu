@@ -49,7 +49,10 @@
 //
 // The key block's keys beyond a query's own position are masked by value (-inf), so the
 // diagonal needs no special path; blocks wholly above the tile's diagonal are never loaded.
-// A sink (e^sink in a head's denominator, without a key) joins in the epilogue.
+// A sink (e^sink in a head's denominator, without a key) joins in the epilogue. A bias by distance (a table
+// [heads, span], bias[h, min(p - j, span - 1)] added to the scaled score) is added in registers in the key blocks that hold
+// keys less than span - 1 back from a warp's rows; to all others one number belongs, which rides in the multiply-add of the
+// exponent.
 // All waits are bounded by a clock limit and report through the status word of this library.
 #include "tc.cuh"
 
@@ -111,14 +114,15 @@ __device__ __forceinline__ void tmem_st32(uint32_t taddr, const uint32_t (&r)[32
 }
 // HD: head dimension, 64 or 128 (one or two 64-column pieces per tile). Two blocks fit on an SM
 // (96 KB of shared memory, 256 columns of tensor memory, at most 168 registers).
-template <int HD>
+template <int HD, bool BIAS>
 __global__ void __launch_bounds__(THREADS, 2)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, const int* __restrict__ block_table,
                             int table_stride, int ring_pages, const int* __restrict__ cu_seqlens,
                             const int* __restrict__ seq_lens, const int* __restrict__ seq_order,
                             __nv_bfloat16* __restrict__ out, int out_stride,
-                            int n_heads, int n_kv_heads, float scale_log2, const float* __restrict__ sinks, int* status) {
+                            int n_heads, int n_kv_heads, float scale_log2, const float* __restrict__ sinks,
+                            const float* __restrict__ bias, int span, int* status) {
     constexpr int PIECES = HD / 64;
     constexpr int Q_BYTES = PIECES * Q_PIECE;         // the block's queries
     constexpr int KV_BYTES = PIECES * KV_PIECE;       // the K or the V of one key block
@@ -263,6 +267,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         int pos = start + q_index;
         uint32_t lane_addr = tmem_base + ((uint32_t)(quarter * 32) << 16);
         float run_max = -INFINITY, run_sum = 0.f;
+        // a bias in raw units (the scale is positive): that of far keys, and the table for near ones
+        const float to_raw = BIAS ? 1.4426950408889634f / scale_log2 : 0.f;
+        const float* near_bias = BIAS ? bias + (size_t)head * span : nullptr;
+        const float far_bias = BIAS ? near_bias[span - 1] * to_raw : 0.f;
         bool ok = true;
         LAPS_BEGIN
         for (int kb = 0; kb < n_blocks && ok; ++kb) {
@@ -294,8 +302,22 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             };
             tmem_ld32_wait(ra);
             tmem_ld32_wait(rb);
+            float far_raw = 0.f;
+            if constexpr (BIAS) {
+                if (start + tile * BQ + quarter * 32 - (key0 + BKV - 1) >= span - 1) {     // (the same answer in the whole warp)
+                    far_raw = far_bias;
+                } else {
+                    int back = pos - key0;
+#pragma unroll
+                    for (int j = 0; j < 32; ++j) {
+                        ra[j] = __float_as_uint(fmaf(near_bias[max(0, min(back - j, span - 1))], to_raw, __uint_as_float(ra[j])));
+                        rb[j] = __float_as_uint(fmaf(near_bias[max(0, min(back - 32 - j, span - 1))], to_raw, __uint_as_float(rb[j])));
+                    }
+                }
+            }
             row_max(ra, 0);
             row_max(rb, 32);
+            if constexpr (BIAS) block_max += far_raw;
             LAP(1);
             // The exponent's reference moves only when the block's maximum exceeds it by more than
             // 2^8 (softmax does not depend on the reference; probabilities up to 256 are as exact in
@@ -306,7 +328,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             bool move = kb == 0 || (block_max - run_max) * scale_log2 > 8.f;
             float new_max = move ? block_max : run_max;      // finite for a real row: key 0 is visible
             float alpha = (move && kb > 0) ? fast_exp2((run_max - new_max) * scale_log2) : 1.f;
-            float shift = new_max * scale_log2;
+            float shift = (new_max - far_raw) * scale_log2;
             run_max = new_max;
             // probabilities, written over the scores' first columns as bfloat16 pairs (every score of
             // the buffer is in a register by now)
@@ -437,40 +459,44 @@ template <int HD>
 int launch(const CUtensorMap& map_q, const CUtensorMap& map_k, const CUtensorMap& map_v,
            const int* block_table, int table_stride, int ring_pages, const int* cu_seqlens,
            const int* seq_lens, const int* seq_order, void* out, int out_stride, int n_seqs, int max_new, int n_heads,
-           int n_kv_heads, float scale, const float* sinks, cudaStream_t stream) {
+           int n_kv_heads, float scale, const float* sinks, const float* bias, int span, cudaStream_t stream) {
     constexpr int Q_BYTES = (HD / 64) * Q_PIECE, KV_BYTES = (HD / 64) * KV_PIECE;
     // never less than 80 KB, so that no third block lands on an SM and waits for tensor memory
     size_t smem = 1024 + (size_t)Q_BYTES + 4 * KV_BYTES + 16 * 8 + 16;
     if (smem < 80 * 1024) smem = 80 * 1024;
     static bool configured = false;
     if (!configured) {
-        LLMB_CUDA(cudaFuncSetAttribute(attention_prefill_tc_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        LLMB_CUDA(cudaFuncSetAttribute(attention_prefill_tc_kernel<HD, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        LLMB_CUDA(cudaFuncSetAttribute(attention_prefill_tc_kernel<HD, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         configured = true;
     }
     int* status = status_word();
     int* status_dev = nullptr;
     if (status) cudaHostGetDevicePointer((void**)&status_dev, status, 0);
     dim3 grid(n_heads, (max_new + BQ - 1) / BQ, n_seqs);
-    llmb::launch(attention_prefill_tc_kernel<HD>, grid, THREADS, smem, stream, true,
+    llmb::launch(bias ? attention_prefill_tc_kernel<HD, true> : attention_prefill_tc_kernel<HD, false>, grid, THREADS, smem, stream, true,
                  map_q, map_k, map_v, block_table, table_stride, ring_pages, cu_seqlens, seq_lens, seq_order,
-                 (__nv_bfloat16*)out, out_stride, n_heads, n_kv_heads, scale * 1.4426950408889634f, sinks, status_dev);
+                 (__nv_bfloat16*)out, out_stride, n_heads, n_kv_heads, scale * 1.4426950408889634f, sinks, bias, span, status_dev);
     return check_launch("attention_prefill_tc");
 }
 }  // namespace
 
 // q: the fused projection of the new tokens [n_tokens, q_stride] (queries in its first columns);
 // k_cache, v_cache: one layer of the paged cache [n_pages, n_kv_heads, 64, head_dim]; the rest as in
-// llmb_attention_prefill; sinks float32 [n_heads] or null: e^sink is one more term of a head's softmax denominator. out must be 16-byte aligned with a row stride that is a multiple of 8.
+// llmb_attention_prefill; sinks float32 [n_heads] or null: e^sink is one more term of a head's softmax denominator;
+// bias float32 [n_heads, span] or null. out must be 16-byte aligned with a row stride that is a multiple of 8.
 LLMB_EXPORT int llmb_attention_prefill_tc(const void* q, int q_stride, int n_tokens, const void* k_cache,
                                           const void* v_cache, int n_pages, const int* block_table,
                                           int table_stride, int ring_pages, const int* cu_seqlens,
                                           const int* seq_lens, const int* seq_order, void* out, int out_stride, int n_seqs,
                                           int max_new, int n_heads, int n_kv_heads, int head_dim,
-                                          float scale, int window, const float* sinks, cudaStream_t stream) {
+                                          float scale, int window, const float* sinks, const float* bias, int span,
+                                          cudaStream_t stream) {
     if (n_seqs == 0 || max_new == 0) return LLMB_OK;
     int code = llmb_attention_prefill_tc_supports(n_heads, n_kv_heads, head_dim, window);
     if (code) return code;
     LLMB_REQUIRE(n_seqs <= 65535 && max_new / BQ < 65535 && ring_pages > 0 && n_pages > 0, "attention_prefill_tc: bad sizes");
+    LLMB_REQUIRE(!bias || (span > 0 && scale > 0.f), "attention_prefill_tc: a bias needs its table and a positive scale");
     LLMB_REQUIRE(q_stride % 8 == 0 && out_stride % 8 == 0 && (reinterpret_cast<uintptr_t>(q) & 15) == 0 &&
                  (reinterpret_cast<uintptr_t>(out) & 15) == 0 && (reinterpret_cast<uintptr_t>(k_cache) & 15) == 0 &&
                  (reinterpret_cast<uintptr_t>(v_cache) & 15) == 0,
@@ -482,9 +508,9 @@ LLMB_EXPORT int llmb_attention_prefill_tc(const void* q, int q_stride, int n_tok
     if ((code = make_map_2d(&map_v, v_cache, cache_rows, head_dim, head_dim, 64, LLMB_PAGE))) return code;
     if (head_dim == 64)
         return launch<64>(map_q, map_k, map_v, block_table, table_stride, ring_pages, cu_seqlens, seq_lens, seq_order, out,
-                          out_stride, n_seqs, max_new, n_heads, n_kv_heads, scale, sinks, stream);
+                          out_stride, n_seqs, max_new, n_heads, n_kv_heads, scale, sinks, bias, span, stream);
     return launch<128>(map_q, map_k, map_v, block_table, table_stride, ring_pages, cu_seqlens, seq_lens, seq_order, out,
-                       out_stride, n_seqs, max_new, n_heads, n_kv_heads, scale, sinks, stream);
+                       out_stride, n_seqs, max_new, n_heads, n_kv_heads, scale, sinks, bias, span, stream);
 }
 
 // the packed doors of the launching entry points (common.cuh)

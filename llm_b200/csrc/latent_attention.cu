@@ -3,7 +3,9 @@
 //
 // latent_write    one block per token of the projection [q: H x (D | R) | c (C) | r (R)]: c / sqrt(mean(c^2) + eps) * gain, r
 //                 rotated, both into the token's cache row (and, optionally, a dense row); the rotated part of every
-//                 query head, either into the last R columns of its latent query [C | R] or in place.
+//                 query head, either into the last R columns of its latent query [C | R] or in place. Where the queries pass
+//                 a latent of their own, the launch behind the first product norms that latent and writes the cache row, and
+//                 a second one, behind the queries' product, rotates the query heads.
 // head_products   out[t, h, :] = W_h x[t, h, :] with a matrix per head: queries into the latent space, results out of it.
 // latent_attention_tiles (bfloat16)  softmax attention of the new tokens' latent queries [T, H, C + R] over the cached
 //                 rows. All heads share the row, so (token, head) pairs are the rows of the tiles: a block takes 16, 32 or 64
@@ -14,6 +16,7 @@
 //                 Shared memory rows are swizzled by 16-byte pieces (piece ^ row % 8).
 // latent_decode_tc (bfloat16)  the same for a step of one token a sequence on tcgen05, with the rows by TMA: see there.
 //
+// `sinks` [H] (optional): e^sink[h] is one more term of a head's denominator, without key or value, not scaled.
 // Norm, rotation, scores, weights and sums are 32-bit (weights are rounded as the operand of P V, whose sum is 32-bit).
 // A query at position p sees the keys j <= p.
 #include "common.cuh"
@@ -53,9 +56,23 @@ __device__ __forceinline__ float rotated(const T* x, int d, const float* angles,
     return first ? v * c - other * s : v * c + other * s;
 }
 
+// 1 / root mean square of the block's row of n elements.
+template <typename T>
+__device__ __forceinline__ float row_factor(const T* x, int n, float eps, float* scratch) {
+    float sq = 0.f;
+    for (int d = threadIdx.x; d < n; d += THREADS) {
+        float v = to_float(x[d]);
+        sq = fmaf(v, v, sq);
+    }
+    return 1.0f / sqrtf(block_sum(sq, scratch) / (float)n + eps);
+}
+
+// Three parts, each optional: the queries' latent (the first q_rank columns of u, normed, into cq), the cached row (c_at >= 0: the
+// columns [c | r] of u from there on), and the rotated parts of the query heads in `heads` (which may be u).
 template <typename T>
 __global__ void __launch_bounds__(THREADS)
-latent_write_kernel(T* __restrict__ u, int ld, int H, int D, int R, int C, const float* __restrict__ gain, float eps,
+latent_write_kernel(const T* u, int ld, int c_at, int q_rank, const float* __restrict__ q_gain, T* __restrict__ cq, T* heads,
+                    int heads_ld, int H, int D, int R, int C, const float* __restrict__ gain, float eps,
                     const float* __restrict__ table, int n_rot, int interleaved, const int* __restrict__ tok_pos,
                     const int* __restrict__ tok_seq, const int* __restrict__ block_table, int table_stride, int ring_pages,
                     T* __restrict__ cache, int write_cache, T* __restrict__ queries, T* __restrict__ dense) {
@@ -63,26 +80,30 @@ latent_write_kernel(T* __restrict__ u, int ld, int H, int D, int R, int C, const
     griddep_launch();
     griddep_wait();
     size_t t = blockIdx.x;
-    T* in = u + t * ld;
-    const T* c_in = in + H * (D + R);
+    const T* row = u + t * ld;
     int pos = tok_pos[t], width = C + R;
     const float* angles = table + (size_t)pos * n_rot;
-    float sq = 0.f;
-    for (int d = threadIdx.x; d < C; d += THREADS) {
-        float v = to_float(c_in[d]);
-        sq = fmaf(v, v, sq);
+    if (q_rank > 0) {
+        float factor = row_factor(row, q_rank, eps, scratch);
+        for (int d = threadIdx.x; d < q_rank; d += THREADS)
+            cq[t * q_rank + d] = from_float<T>(to_float(row[d]) * factor * q_gain[d]);
     }
-    float factor = 1.0f / sqrtf(block_sum(sq, scratch) / (float)C + eps);
-    T* to = nullptr;
-    if (write_cache) {
-        size_t page = (size_t)block_table[(size_t)tok_seq[t] * table_stride + (pos / LLMB_PAGE) % ring_pages];
-        to = cache + (page * LLMB_PAGE + pos % LLMB_PAGE) * width;
+    if (c_at >= 0) {
+        const T* c_in = row + c_at;
+        float factor = row_factor(c_in, C, eps, scratch);
+        T* to = nullptr;
+        if (write_cache) {
+            size_t page = (size_t)block_table[(size_t)tok_seq[t] * table_stride + (pos / LLMB_PAGE) % ring_pages];
+            to = cache + (page * LLMB_PAGE + pos % LLMB_PAGE) * width;
+        }
+        for (int d = threadIdx.x; d < width; d += THREADS) {
+            T v = from_float<T>(d < C ? to_float(c_in[d]) * factor * gain[d] : rotated(c_in + C, d - C, angles, n_rot, interleaved));
+            if (to) to[d] = v;
+            if (dense) dense[t * width + d] = v;
+        }
     }
-    for (int d = threadIdx.x; d < width; d += THREADS) {
-        T v = from_float<T>(d < C ? to_float(c_in[d]) * factor * gain[d] : rotated(c_in + C, d - C, angles, n_rot, interleaved));
-        if (to) to[d] = v;
-        if (dense) dense[t * width + d] = v;
-    }
+    if (!heads) return;
+    T* in = heads + t * heads_ld;
     if (queries) {
         for (int i = threadIdx.x; i < H * R; i += THREADS) {
             int head = i / R, d = i % R;
@@ -102,19 +123,23 @@ latent_write_kernel(T* __restrict__ u, int ld, int H, int D, int R, int C, const
     }
 }
 
-// u [T, ld]: H query heads of D + R, then C + R columns; gain float32 [C]; table float32 [positions, n_rot] (or null: no
-// rotation); cache [pages, 1, 64, C + R]; queries [T, H, C + R] (or null: query heads rotate in place); dense [T, C + R] or null.
-LLMB_EXPORT int llmb_latent_write(void* u, int ld, int dtype, int H, int D, int R, int C, const float* gain, float eps,
+// u [T, ld]: [queries' latent (q_rank) ..] and from column c_at on [c (C) | r (R)] (c_at < 0: not there); heads [T, heads_ld]: H query
+// heads of D + R (null: none; it may be u); q_gain float32 [q_rank] and cq [T, q_rank] with q_rank > 0; gain float32 [C]; table
+// float32 [positions, n_rot] (or null: no rotation); cache [pages, 1, 64, C + R]; queries [T, H, C + R] (or null: query heads
+// rotate in place); dense [T, C + R] or null.
+LLMB_EXPORT int llmb_latent_write(const void* u, int ld, int dtype, int c_at, int q_rank, const float* q_gain, void* cq, void* heads,
+                                  int heads_ld, int H, int D, int R, int C, const float* gain, float eps,
                                   const float* table, int n_rot, int interleaved, const int* tok_pos, const int* tok_seq,
                                   const int* block_table, int table_stride, int ring_pages, void* cache, int write_cache,
                                   void* queries, void* dense, int n_tokens, cudaStream_t stream) {
     if (n_tokens == 0) return LLMB_OK;
-    LLMB_REQUIRE(H > 0 && D > 0 && R > 0 && C > 0 && ld >= H * (D + R) + C + R && gain && ring_pages > 0, "latent_write: bad sizes");
+    LLMB_REQUIRE(H > 0 && D > 0 && R > 0 && C > 0 && ring_pages > 0 && (c_at < 0 || (gain && u && ld >= c_at + C + R)) &&
+                 (q_rank <= 0 || (q_gain && cq && u && ld >= q_rank)) && (!heads || heads_ld >= H * (D + R)), "latent_write: bad sizes");
     LLMB_REQUIRE(!table || (n_rot > 0 && n_rot % 2 == 0 && n_rot <= R), "latent_write: %d of %d elements rotate", n_rot, R);
 #define LLMB_WRITE(T)                                                                                                     \
-    LLMB_CUDA(llmb::launch(latent_write_kernel<T>, dim3(n_tokens), dim3(THREADS), 0, stream, true, (T*)u, ld, H, D, R, C, gain, \
-                           eps, table, table ? n_rot : 0, interleaved, tok_pos, tok_seq, block_table, table_stride, ring_pages, \
-                           (T*)cache, write_cache, (T*)queries, (T*)dense))
+    LLMB_CUDA(llmb::launch(latent_write_kernel<T>, dim3(n_tokens), dim3(THREADS), 0, stream, true, (const T*)u, ld, c_at, q_rank, \
+                           q_gain, (T*)cq, (T*)heads, heads_ld, H, D, R, C, gain, eps, table, table ? n_rot : 0, interleaved, \
+                           tok_pos, tok_seq, block_table, table_stride, ring_pages, (T*)cache, write_cache, (T*)queries, (T*)dense))
     if (dtype == LLMB_DTYPE_F32) LLMB_WRITE(float);
     else if (dtype == LLMB_DTYPE_BF16) LLMB_WRITE(__nv_bfloat16);
     else return fail(LLMB_ERR_ARGUMENT, "latent_write: unknown dtype %d", dtype);
@@ -281,6 +306,10 @@ __device__ __forceinline__ float fast_exp2(float x) {
     return y;
 }
 
+// What a sink adds to a denominator in units of 2^m (m: the row's reference, base 2). A sink far above every score makes it
+// infinite and the row's result zero, as it should be.
+__device__ __forceinline__ float sink_share(float sink, float m) { return exp2f(fmaf(sink, 1.4426950408889634f, -m)); }
+
 // MT: tiles of 16 rows ((token, head) pairs) a block holds; NT: blocks of 8 value columns a warp holds (C <= 64 NT).
 // Eight warps. S: warp w works on rows [(w % MT) 16, +16) and keys [(w / MT) 8 MT, + 8 MT) of a page.
 // `width` C + R, `row_elems` the elements of a row in shared memory (a multiple of 64, at least width and 64 NT).
@@ -290,7 +319,7 @@ latent_tiles_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
                     const int* __restrict__ block_table, int table_stride, int ring_pages, const int* __restrict__ cu_seqlens,
                     const int* __restrict__ seq_lens, const int* __restrict__ seq_order, __nv_bfloat16* __restrict__ out,
                     float* __restrict__ part_acc, float* __restrict__ part_stats, int H, int C, int width, int row_elems,
-                    float scale_log2) {
+                    float scale_log2, const float* __restrict__ sinks) {
     constexpr int ROWS = 16 * MT, KW = 8 / MT;             // KW: warps that share a row tile's keys
     extern __shared__ __align__(128) unsigned char smem_raw[];
     const int row_bytes = row_elems * 2;
@@ -487,7 +516,11 @@ latent_tiles_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     sum1 += __shfl_xor_sync(0xffffffffu, sum1, 1);
     sum1 += __shfl_xor_sync(0xffffffffu, sum1, 2);
     __syncthreads();
-    if (t4 == 0) { red[k_part * ROWS + row0] = sum0; red[k_part * ROWS + row1] = sum1; }
+    if (t4 == 0) {
+        red[k_part * ROWS + row0] = sum0;
+        red[k_part * ROWS + row1] = sum1;
+        if (k_part == 0) { alphas[row0] = max0; alphas[row1] = max1; }      // (the factors have been read)
+    }
     __syncthreads();
     size_t base = (size_t)first_token * H + row_first;     // the tile's first row among all rows of the step
     if (n_splits > 1 && warp < MT && t4 == 0) {
@@ -512,6 +545,8 @@ latent_tiles_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
             float total = 0.f;
 #pragma unroll
             for (int w = 0; w < KW; ++w) total += red[w * ROWS + r];
+            if (sinks && n_splits == 1)
+                total += sink_share(sinks[(row_first + r) % H], alphas[r] * scale_log2);
             float inv = n_splits == 1 ? 1.0f / total : 1.f;
 #pragma unroll
             for (int n = 0; n < NT; ++n) {
@@ -576,7 +611,8 @@ __global__ void __launch_bounds__(256, 1)
 latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __nv_bfloat16* __restrict__ q,
                         const int* __restrict__ block_table, int table_stride, int ring_pages, const int* __restrict__ seq_lens,
                         const int* __restrict__ seq_order, __nv_bfloat16* __restrict__ out, float* __restrict__ part_acc,
-                        float* __restrict__ part_stats, int H, int R, int stages, float scale_log2, int* status) {
+                        float* __restrict__ part_stats, int H, int R, int stages, float scale_log2,
+                        const float* __restrict__ sinks, int* status) {
     constexpr int pieces = C / 64 + 1, values = (C + 127) / 128;         // of a row; accumulators
     // tensor memory: the queries (two elements a column), the scores, the accumulators
     constexpr uint32_t Q_COL = 0, S_COL = pieces * 32, O_COL = S_COL + KEYS, COLS = 512;
@@ -807,6 +843,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __nv
             mbar_arrive(smem_u32(&p_full[b]));
         }
         // what the result needs, then the signal
+        if (sinks && n_splits == 1 && live) run_sum += sink_share(sinks[head0 + lane], run_max * scale_log2);
         if (lane < NH) { alphas[lane] = run_sum; maxima[lane] = run_max; }
         if (lane == 0) *at_end = 1;
         __threadfence_block();
@@ -884,7 +921,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap map_rows, const __nv
 constexpr int MAX_SPLITS = 32;
 __global__ void __launch_bounds__(128)
 latent_combine_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_stats, __nv_bfloat16* __restrict__ out,
-                      int C, int n_splits) {
+                      int C, int n_splits, int H, const float* __restrict__ sinks) {
     griddep_launch();
     griddep_wait();
     part_acc = behind_wait(part_acc);
@@ -897,6 +934,7 @@ latent_combine_kernel(const float* __restrict__ part_acc, const float* __restric
         float ms = s < n_splits ? stats[2 * s] : -INFINITY, m = warp_max(ms);
         float weight = ms == -INFINITY ? 0.f : exp2f(ms - m);
         float total = warp_sum(s < n_splits ? stats[2 * s + 1] * weight : 0.f);
+        if (sinks) total += sink_share(sinks[row % H], m);
         if (s < n_splits) shares[s] = weight / total;
     }
     __syncthreads();
@@ -946,7 +984,7 @@ LLMB_EXPORT long long llmb_latent_scratch_floats(int n_tokens, int H, int C, int
 LLMB_EXPORT int llmb_latent_attention(const void* q, const void* cache, const int* block_table, int table_stride,
                                       int ring_pages, const int* cu_seqlens, const int* seq_lens, const int* seq_order, void* out,
                                       float* scratch, long long scratch_floats, int n_tokens, int n_seqs, int max_new, int H,
-                                      int C, int R, float scale, int n_splits, cudaStream_t stream) {
+                                      int C, int R, float scale, const float* sinks, int n_splits, cudaStream_t stream) {
     if (n_seqs == 0 || max_new == 0) return LLMB_OK;
     LLMB_REQUIRE(H > 0 && C > 0 && R > 0 && C % 8 == 0 && R % 8 == 0 && C <= 512 && C + R <= 640,
                  "latent_attention: rows of %d + %d (multiples of 8, up to 512 and 640 in all)", C, R);
@@ -972,7 +1010,7 @@ LLMB_EXPORT int llmb_latent_attention(const void* q, const void* cache, const in
         LLMB_CUDA(llmb::launch(latent_tiles_kernel<MT, NT>, grid, dim3(THREADS), p.smem, stream, true,                    \
                                (const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, block_table, table_stride, ring_pages, \
                                cu_seqlens, seq_lens, seq_order, (__nv_bfloat16*)out, part_acc, part_stats, H, C, C + R,   \
-                               p.row_elems, scale * 1.4426950408889634f));                                                \
+                               p.row_elems, scale * 1.4426950408889634f, sinks));                                         \
     } while (0)
 #define LLMB_TILES(MT)                                 \
     do {                                               \
@@ -989,7 +1027,7 @@ LLMB_EXPORT int llmb_latent_attention(const void* q, const void* cache, const in
     int code = check_launch("latent_attention");
     if (code || n_splits == 1) return code;
     LLMB_CUDA(llmb::launch(latent_combine_kernel, dim3(n_tokens * H), dim3(128), 0, stream, true, (const float*)part_acc,
-                           (const float*)part_stats, (__nv_bfloat16*)out, C, n_splits));
+                           (const float*)part_stats, (__nv_bfloat16*)out, C, n_splits, H, sinks));
     return check_launch("latent_attention_combine");
 }
 LLMB_PACKED(llmb_latent_attention)
@@ -1006,8 +1044,8 @@ LLMB_EXPORT int llmb_latent_attention_status() {
 // bfloat16. scratch as in llmb_latent_attention.
 LLMB_EXPORT int llmb_latent_decode_tc(const void* q, const void* cache, int n_pages, const int* block_table, int table_stride,
                                       int ring_pages, const int* seq_lens, const int* seq_order, void* out, float* scratch,
-                                      long long scratch_floats, int n_seqs, int H, int C, int R, float scale, int n_splits,
-                                      cudaStream_t stream) {
+                                      long long scratch_floats, int n_seqs, int H, int C, int R, float scale,
+                                      const float* sinks, int n_splits, cudaStream_t stream) {
     if (n_seqs == 0) return LLMB_OK;
     LLMB_REQUIRE(H > 0 && (C == 64 || C == 128 || C == 256 || C == 512) && R > 0 && R <= 64 && R % 8 == 0,
                  "latent_decode_tc: rows of %d + %d (64, 128, 256 or 512, a multiple of 8 up to 64)", C, R);
@@ -1037,7 +1075,7 @@ LLMB_EXPORT int llmb_latent_decode_tc(const void* q, const void* cache, int n_pa
         }                                                                                                                 \
         LLMB_CUDA(llmb::launch(decode::latent_decode_tc_kernel<NH, CC>, dim3(n_splits, ceil_div(H, NH), n_seqs), dim3(256), s.smem, \
                                stream, true, map_rows, (const __nv_bfloat16*)q, block_table, table_stride, ring_pages, seq_lens, seq_order, \
-                               (__nv_bfloat16*)out, part_acc, part_stats, H, R, s.stages, scale * 1.4426950408889634f, status_dev)); \
+                               (__nv_bfloat16*)out, part_acc, part_stats, H, R, s.stages, scale * 1.4426950408889634f, sinks, status_dev)); \
     } while (0)
 #define LLMB_DECODE(NH)                               \
     do {                                              \
@@ -1053,7 +1091,7 @@ LLMB_EXPORT int llmb_latent_decode_tc(const void* q, const void* cache, int n_pa
     code = check_launch("latent_decode_tc");
     if (code || n_splits == 1) return code;
     LLMB_CUDA(llmb::launch(latent_combine_kernel, dim3(n_seqs * H), dim3(128), 0, stream, true, (const float*)part_acc,
-                           (const float*)part_stats, (__nv_bfloat16*)out, C, n_splits));
+                           (const float*)part_stats, (__nv_bfloat16*)out, C, n_splits, H, sinks));
     return check_launch("latent_attention_combine");
 }
 LLMB_PACKED(llmb_latent_decode_tc)

@@ -5,6 +5,7 @@
 //     q    [T, ld]: head h's query in columns h (D + R) .. (rotated)
 //     kv   [T, H (D + V)]: head h's unrotated key, then its value, in columns h (D + V) ..
 //     rows [T, C + R]: the shared rotated key part in the last R columns
+// With `sinks` (float32 [H], optional) e^sink is one more term of a head's denominator, without key or value, not scaled.
 //
 // One block serves 256 queries of one head of one sequence as two tiles of 128 (the rows of tensor memory), which share
 // the keys and values that come by TMA in blocks of 64 tokens:
@@ -60,7 +61,7 @@ __global__ void __launch_bounds__(THREADS, 1)
 latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
                          const __grid_constant__ CUtensorMap map_r, const int* __restrict__ cu_seqlens,
                          const int* __restrict__ seq_order, __nv_bfloat16* __restrict__ out, int out_stride, int R,
-                         float scale_log2, int* status) {
+                         float scale_log2, const float* __restrict__ sinks, int* status) {
     constexpr int PIECES = D / 64 + 1, V_PIECES = V / 64;
     constexpr int Q_BYTES = PIECES * Q_PIECE, K_BYTES = PIECES * KV_PIECE, V_BYTES = V_PIECES * KV_PIECE;
     extern __shared__ __align__(1024) unsigned char smem_raw[];
@@ -300,6 +301,8 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         if (ok) {
             __syncwarp();
             tcgen05_fence_after();
+            // (a sink far above every score makes the denominator infinite and the result zero, as it should be)
+            if (sinks) run_sum += fast_exp2(fmaf(sinks[head], 1.4426950408889634f, -run_max * scale_log2));
             float inv = 1.0f / run_sum;
             __nv_bfloat16* o = out + (size_t)(first_token + pos) * out_stride + (size_t)head * V;
 #pragma unroll 1
@@ -347,7 +350,7 @@ namespace {
 template <int D, int V>
 int launch(const CUtensorMap& map_q, const CUtensorMap& map_kv, const CUtensorMap& map_r, const int* cu_seqlens,
            const int* seq_order, void* out, int out_stride, int n_seqs, int max_new, int H, int R, float scale,
-           cudaStream_t stream) {
+           const float* sinks, cudaStream_t stream) {
     constexpr size_t smem = smem_bytes<D, V>() < 120 * 1024 ? 120 * 1024 : smem_bytes<D, V>();     // one block an SM: it takes all of tensor memory
     static bool configured = false;
     if (!configured) {
@@ -359,7 +362,7 @@ int launch(const CUtensorMap& map_q, const CUtensorMap& map_kv, const CUtensorMa
     if (status) cudaHostGetDevicePointer((void**)&status_dev, status, 0);
     dim3 grid(H, ceil_div(max_new, TILES * BQ), n_seqs);
     LLMB_CUDA(llmb::launch(latent_prefill_tc_kernel<D, V>, grid, dim3(THREADS), smem, stream, true, map_q, map_kv, map_r, cu_seqlens,
-                           seq_order, (__nv_bfloat16*)out, out_stride, R, scale * 1.4426950408889634f, status_dev));
+                           seq_order, (__nv_bfloat16*)out, out_stride, R, scale * 1.4426950408889634f, sinks, status_dev));
     return check_launch("latent_prefill_tc");
 }
 }  // namespace
@@ -368,7 +371,8 @@ int launch(const CUtensorMap& map_q, const CUtensorMap& map_kv, const CUtensorMa
 // step starts at its first token.
 LLMB_EXPORT int llmb_latent_prefill_tc(const void* q, int ldq, const void* kv, const void* rows, int n_tokens,
                                        const int* cu_seqlens, const int* seq_order, void* out, int out_stride, int n_seqs,
-                                       int max_new, int H, int D, int R, int V, int C, float scale, cudaStream_t stream) {
+                                       int max_new, int H, int D, int R, int V, int C, float scale, const float* sinks,
+                                       cudaStream_t stream) {
     if (n_seqs == 0 || max_new == 0) return LLMB_OK;
     LLMB_REQUIRE((D == 64 || D == 128) && (V == 64 || V == 128) && R > 0 && R <= 64 && R % 8 == 0 && C % 8 == 0 && H > 0,
                  "latent_prefill_tc: heads of %d + %d with values of %d over a latent of %d", D, R, V, C);
@@ -382,7 +386,7 @@ LLMB_EXPORT int llmb_latent_prefill_tc(const void* q, int ldq, const void* kv, c
     if ((code = make_map_2d(&map_q, q, n_tokens, (long long)H * (D + R), ldq, 64, BQ))) return code;
     if ((code = make_map_2d(&map_kv, kv, n_tokens, (long long)H * (D + V), (long long)H * (D + V), 64, BKV))) return code;
     if ((code = make_map_2d(&map_r, (const __nv_bfloat16*)rows + C, n_tokens, R, C + R, 64, BKV))) return code;
-#define GO(DD, VV) return launch<DD, VV>(map_q, map_kv, map_r, cu_seqlens, seq_order, out, out_stride, n_seqs, max_new, H, R, scale, stream)
+#define GO(DD, VV) return launch<DD, VV>(map_q, map_kv, map_r, cu_seqlens, seq_order, out, out_stride, n_seqs, max_new, H, R, scale, sinks, stream)
     if (D == 64 && V == 64) GO(64, 64);
     if (D == 64) GO(64, 128);
     if (V == 64) GO(128, 64);

@@ -16,6 +16,8 @@
 // With mix_cache the values are blended before they are cached: v <- (1 - mix) v + mix * first, where
 // `first` is the row that another layer's value cache (mix_cache, with its own page table and ring) holds
 // for the same token, key/value head and element; that layer must have written the step's tokens before.
+// With `q_scale` (a table [positions]) the queries are multiplied by the number of their position, behind the norm. k_width may
+// be 0: queries alone (a mixer that reads another layer's keys).
 #include "common.cuh"
 
 using namespace llmb;
@@ -45,7 +47,8 @@ norm_rope_cache_write_kernel(const T* __restrict__ u, int u_stride, int q_width,
                              int q_out_stride, const int* __restrict__ block_table, int table_stride, int ring_pages,
                              T* __restrict__ k_cache, int k_heads, T* __restrict__ v_cache, int v_heads,
                              int write_cache, int v_source, int norm_unit, const T* __restrict__ mix_cache,
-                             const int* __restrict__ mix_table, int mix_table_stride, int mix_ring, float mix) {
+                             const int* __restrict__ mix_table, int mix_table_stride, int mix_ring, float mix,
+                             const float* __restrict__ q_scale) {
     extern __shared__ float row[];         // [q_width + k_width]
     __shared__ float scratch[THREADS / 32];
     griddep_launch();
@@ -86,6 +89,7 @@ norm_rope_cache_write_kernel(const T* __restrict__ u, int u_stride, int q_width,
     __syncthreads();
     int pos = tok_pos[t];
     const float* angles = rope_table ? rope_table + (size_t)pos * n_rot : nullptr;
+    float warm = q_scale ? q_scale[pos] : 1.f;
     int half = n_rot / 2;
     size_t page = 0;
     int slot_row = pos % LLMB_PAGE;
@@ -107,7 +111,7 @@ norm_rope_cache_write_kernel(const T* __restrict__ u, int u_stride, int q_width,
             }
         }
         if (is_q) {
-            q_out[(size_t)t * q_out_stride + local] = from_float<T>(v);
+            q_out[(size_t)t * q_out_stride + local] = from_float<T>(q_scale ? v * warm : v);
         } else {
             int head = local / k_dim, d = local % k_dim;
             k_cache[((page * k_heads + head) * LLMB_PAGE + slot_row) * k_dim + d] = from_float<T>(v);
@@ -140,9 +144,9 @@ LLMB_EXPORT int llmb_norm_rope_cache_write(const void* u, int u_stride, int dtyp
                                            int table_stride, int ring_pages, void* k_cache, int k_heads, void* v_cache,
                                            int v_heads, int write_cache, int v_source, int norm_unit,
                                            const void* mix_cache, const int* mix_table, int mix_table_stride,
-                                           int mix_ring, float mix, int n_tokens, cudaStream_t stream) {
+                                           int mix_ring, float mix, const float* q_scale, int n_tokens, cudaStream_t stream) {
     if (n_tokens == 0) return LLMB_OK;
-    LLMB_REQUIRE(q_width > 0 && k_width > 0 && v_width >= 0 && k_heads > 0 && k_width % k_heads == 0,
+    LLMB_REQUIRE(q_width > 0 && v_width >= 0 && ((k_width == 0 && !write_cache) || (k_width > 0 && k_heads > 0 && k_width % k_heads == 0)),
                  "norm_rope_cache_write: bad widths %d / %d / %d with %d key heads", q_width, k_width, v_width, k_heads);
     LLMB_REQUIRE(v_width == 0 || (v_heads > 0 && v_width % v_heads == 0 && v_cache),
                  "norm_rope_cache_write: %d value columns do not fit %d heads", v_width, v_heads);
@@ -168,7 +172,7 @@ LLMB_EXPORT int llmb_norm_rope_cache_write(const void* u, int u_stride, int dtyp
                                rope_table ? n_rot : 0, rot_unit > 0 ? rot_unit : 1, interleaved, tok_pos, tok_seq,   \
                                (T*)q_out, q_out_stride, block_table, table_stride, ring_pages, (T*)k_cache, k_heads, \
                                (T*)v_cache, v_heads, write_cache, v_source, norm_unit, (const T*)mix_cache,          \
-                               mix_table, mix_table_stride, mix_ring, mix));                                        \
+                               mix_table, mix_table_stride, mix_ring, mix, q_scale));                               \
     } while (0)
     if (dtype == LLMB_DTYPE_F32) LLMB_NORM_ROPE(float);
     else if (dtype == LLMB_DTYPE_BF16) LLMB_NORM_ROPE(__nv_bfloat16);

@@ -11,6 +11,8 @@
 //          router may have more outputs than there are experts: the last ones are pass-through experts without
 //          matrices whose result is the token's own row h (times the weight); a small kernel writes those rows,
 //          the plan and the products see only the assignments of experts that have matrices.
+//          With `groups` > 1 (scoring 1) the outputs form that many equal groups of neighbours; only outputs of the `keep`
+//          groups with the largest single score can be chosen (the lower group wins a tie).
 //          `scoring` 2: scores s = sigmoid(z), the `top` largest chosen, weights s as they are.
 //          `weight_scale` multiplies every weight (a constant in front of the whole feed-forward).
 // plan     counts the assignments of every expert, lists them grouped by expert (inside an expert in rising
@@ -19,7 +21,9 @@
 //          the host: the product kernels are launched with the largest possible tile count and blocks beyond the
 //          plan's count leave at once, so a step can be captured and replayed.
 // up       for every tile: act[s, :] = silu(W_gate,e h_t) * (W_up,e h_t) for the rows s of the sorted list
-//          (h_t gathered through the list), one weight matrix [2 F, K] per expert (gate rows, then up).
+//          (h_t gathered through the list), one weight matrix [2 F, K] per expert (gate rows, then up). With a limit the
+//          activation is the clamped one instead: g <- min(g, limit), u <- clamp(u, -limit, limit),
+//          g sigmoid(alpha g) (u + 1).
 // down     for every tile: y[t * top + k, :] = weight[t, k] * (W_down,e act[s, :]), 32-bit, written at the
 //          assignment's own index; the sum over k is taken by the kernel behind (fixed order).
 // With the weight on the expert's input instead of its result, up applies it to its 32-bit sums (W (w h) = w W h) in
@@ -46,6 +50,17 @@ LLMB_DEFINE_LAST_ERROR(llmb_routed_experts)
 constexpr int MAX_TOP = 64;
 constexpr int TILE_M = 32;
 
+// What joins the gate and up sums: limit < 0: silu(g) u; else clamped.
+struct Activation { float limit, alpha; };
+__device__ __forceinline__ float activated(float g, float u, Activation act) {
+    if (act.limit >= 0.f) {
+        g = fminf(g, act.limit);
+        u = fminf(fmaxf(u, -act.limit), act.limit);
+        return g / (1.0f + expf(-act.alpha * g)) * (u + 1.0f);
+    }
+    return g / (1.0f + expf(-g)) * u;
+}
+
 __device__ __forceinline__ void load4(const float* p, float (&x)[4]) {
     float4 v = *reinterpret_cast<const float4*>(p);
     x[0] = v.x; x[1] = v.y; x[2] = v.z; x[3] = v.w;
@@ -63,7 +78,7 @@ template <typename T, int TOK>
 __global__ void __launch_bounds__(512)
 router_kernel(const T* __restrict__ h, int ld, const float* __restrict__ w, const float* __restrict__ bias,
               int hidden, int E, int top, int* __restrict__ ids, float* __restrict__ weights, int n_tokens, int vectors,
-              int scoring, const float* __restrict__ correction, float weight_scale) {
+              int scoring, const float* __restrict__ correction, float weight_scale, int groups, int keep) {
     extern __shared__ float logits[];      // [TOK][E]
     griddep_launch();
     griddep_wait();
@@ -119,12 +134,27 @@ router_kernel(const T* __restrict__ h, int ld, const float* __restrict__ w, cons
         for (int e = 0; e < E; ++e) largest = fmaxf(largest, mine[e]);
         for (int e = 0; e < E; ++e) total += expf(mine[e] - largest);
         for (int e = 0; e < E; ++e) mine[e] = expf(mine[e] - largest) / total;      // scores: never negative
+        if (keep < groups) {
+            // a group's score is its largest score; the outputs of the groups - keep groups with the smallest are closed
+            // (of equal groups the higher one goes first)
+            int size = E / groups;
+            for (int out = groups - keep; out > 0; --out) {
+                int worst = -1;
+                float least = INFINITY;
+                for (int g = 0; g < groups; ++g) {
+                    float peak = -1.f;
+                    for (int e = g * size; e < (g + 1) * size; ++e) peak = fmaxf(peak, mine[e]);
+                    if (peak >= 0.f && peak <= least) { least = peak; worst = g; }
+                }
+                for (int e = worst * size; e < (worst + 1) * size; ++e) mine[e] = -1.f;
+            }
+        }
         float sum = 0.f;
         for (int k = 0; k < top; ++k) {
             int best = 0;
             float value = -INFINITY;
             for (int e = 0; e < E; ++e) {
-                if (mine[e] < 0.f) continue;                  // taken already
+                if (mine[e] < 0.f) continue;                  // taken already, or in a closed group
                 float c = mine[e] + (correction ? correction[e] : 0.f);
                 if (c > value) { value = c; best = e; }
             }
@@ -254,7 +284,7 @@ template <typename T, bool GLU>
 __global__ void __launch_bounds__(256)
 expert_product_kernel(const T* __restrict__ A, int lda, int a_div, const T* __restrict__ W, long long w_stride, int N,
                       int K, const int* __restrict__ sorted, const int* __restrict__ plan, int E, int max_tiles,
-                      T* __restrict__ act, float* __restrict__ y, const float* __restrict__ weights) {
+                      T* __restrict__ act, float* __restrict__ y, const float* __restrict__ weights, Activation activation) {
     __shared__ float As[BK][TILE_M + 1];
     __shared__ float Bs[GLU ? 2 : 1][BK][BN + 1];
     griddep_launch();
@@ -314,7 +344,7 @@ expert_product_kernel(const T* __restrict__ A, int lda, int a_div, const T* __re
                 int col = n0 + tx * 4 + j;
                 if (col < N) {
                     float g = wgt * acc[0][i][j];
-                    act[(long long)s * N + col] = from_float<T>(g / (1.0f + expf(-g)) * (wgt * acc[GLU ? 1 : 0][i][j]));
+                    act[(long long)s * N + col] = from_float<T>(activated(g, wgt * acc[GLU ? 1 : 0][i][j], activation));
                 }
             }
         } else {
@@ -338,7 +368,7 @@ __global__ void __launch_bounds__(128)
 expert_product_tc_kernel(const __nv_bfloat16* __restrict__ A, int lda, int a_div, const __nv_bfloat16* __restrict__ W,
                          long long w_stride, int N, int K, const int* __restrict__ sorted, const int* __restrict__ plan,
                          int E, int max_tiles, __nv_bfloat16* __restrict__ act, float* __restrict__ y,
-                         const float* __restrict__ weights) {
+                         const float* __restrict__ weights, Activation activation) {
     __shared__ __align__(16) __nv_bfloat16 As[2][TILE_M][TC_LD];
     __shared__ __align__(16) __nv_bfloat16 Bs[2][TC_BN][TC_LD];
     griddep_launch();
@@ -425,7 +455,7 @@ expert_product_tc_kernel(const __nv_bfloat16* __restrict__ A, int lda, int a_div
                         if (r < rows && feature < N) {
                             float wgt = weights ? weights[sorted[first + r]] : 1.f;
                             float g = wgt * acc[mi][nj][f];
-                            act[(long long)(first + r) * N + feature] = __float2bfloat16_rn(g / (1.0f + expf(-g)) * (wgt * up[r][c]));
+                            act[(long long)(first + r) * N + feature] = __float2bfloat16_rn(activated(g, wgt * up[r][c], activation));
                         }
                     }
     } else {
@@ -487,7 +517,7 @@ __global__ void __launch_bounds__(G_THREADS, GN == 128 ? 2 : 1)
 expert_product_wide_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                            const int* __restrict__ plan, int E, int max_tiles, int b_rows, int N, int n_kblocks,
                            __nv_bfloat16* __restrict__ act, float* __restrict__ y, const int* __restrict__ sorted,
-                           const float* __restrict__ weights, int* status) {
+                           const float* __restrict__ weights, Activation activation, int* status) {
     constexpr int G_STAGES = stages_of(GN), B_BYTES = GN * GK * 2;
     extern __shared__ __align__(1024) unsigned char smem_raw[];
     unsigned char* base = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -594,7 +624,7 @@ expert_product_wide_kernel(const __grid_constant__ CUtensorMap map_a, const __gr
 #pragma unroll
                     for (int j = 0; j < 16; ++j) {
                         float gate = wgt * __uint_as_float(g[j]);
-                        v[j] = gate / (1.0f + expf(-gate)) * (wgt * __uint_as_float(u[j]));
+                        v[j] = activated(gate, wgt * __uint_as_float(u[j]), activation);
                     }
                     if (vector && n0 + c + 16 <= N) {
                         uint32_t packed[8];
@@ -671,11 +701,13 @@ LLMB_EXPORT long long llmb_routed_experts_plan_ints(int n_tokens, int top, int E
 // int32 [T * top], plan int32 [plan_ints]; act [T * top, F] in `dtype`; y float32 [T * top, hidden]. `tensor_cores`:
 // 0 CUDA cores only, 1 also the mma.sync tiles, 2 also the tcgen05 tiles of 128 rows, which need `gathered`
 // (bfloat16 [T * top, hidden] scratch) and are taken when the step has that scratch, 3: those with 256 accumulator columns.
+// limit < 0: experts with silu; else the clamped activation with that limit and `alpha`.
 LLMB_EXPORT int llmb_routed_experts(const void* h, int ld, int dtype, const float* router, const float* router_bias,
                                     const void* w_up, const void* w_down, int* ids, float* weights, int* sorted,
                                     int* plan, void* act, float* y, void* gathered, int n_tokens, int hidden, int F,
                                     int E, int top, int tensor_cores, int scoring, const float* correction,
-                                    int pass_through, float weight_scale, int weight_on_input, cudaStream_t stream) {
+                                    int pass_through, float weight_scale, int weight_on_input, int groups, int keep,
+                                    float limit, float alpha, cudaStream_t stream) {
     if (n_tokens == 0) return LLMB_OK;
     LLMB_REQUIRE(hidden > 0 && F > 0 && E > 0 && top > 0 && pass_through >= 0 && top <= E + pass_through && top <= MAX_TOP,
                  "routed_experts: %d of %d experts (at most %d are chosen)", top, E + pass_through, MAX_TOP);
@@ -685,6 +717,10 @@ LLMB_EXPORT int llmb_routed_experts(const void* h, int ld, int dtype, const floa
     const float* up_weights = weight_on_input ? weights : nullptr;
     const float* down_weights = weight_on_input ? nullptr : weights;
     int R = E + pass_through;                                  // outputs of the router
+    LLMB_REQUIRE(groups >= 1 && keep >= 1 && keep <= groups && R % groups == 0 && (groups == 1 || (scoring == 1 && !correction)) &&
+                 top <= keep * (R / groups),
+                 "routed_experts: %d of %d groups of %d experts (scores over all of them, no correction)", keep, groups, R);
+    Activation activation = {limit, alpha};
     LLMB_REQUIRE(E <= 2048, "routed_experts: %d experts (up to 2048 are built)", E);
     int n_assign = n_tokens * top;
     int max_tiles = (n_assign + TILE_M - 1) / TILE_M + E;
@@ -702,11 +738,11 @@ LLMB_EXPORT int llmb_routed_experts(const void* h, int ld, int dtype, const floa
         if (n_tokens >= 512)                                                                                       \
             LLMB_CUDA(llmb::launch(router_kernel<T, 4>, dim3((n_tokens + 3) / 4), dim3(128), sizeof(float) * 4 * R, \
                                    stream, true, (const T*)h, ld, router, router_bias, hidden, R, top, ids,       \
-                                   weights, n_tokens, router_vectors, scoring, correction, weight_scale));        \
+                                   weights, n_tokens, router_vectors, scoring, correction, weight_scale, groups, keep));        \
         else                                                                                                       \
             LLMB_CUDA(llmb::launch(router_kernel<T, 1>, dim3(n_tokens), dim3(512), sizeof(float) * R, stream,     \
                                    true, (const T*)h, ld, router, router_bias, hidden, R, top, ids, weights,       \
-                                   n_tokens, router_vectors, scoring, correction, weight_scale));                  \
+                                   n_tokens, router_vectors, scoring, correction, weight_scale, groups, keep));                  \
         if (pass_through > 0)                                                                                      \
             LLMB_CUDA(llmb::launch(pass_through_kernel<T>, dim3(n_assign), dim3(256), 0, stream, true, (const T*)h, \
                                    ld, top, (const int*)ids, (const float*)weights, E, hidden, y));                \
@@ -754,33 +790,33 @@ LLMB_EXPORT int llmb_routed_experts(const void* h, int ld, int dtype, const floa
         auto down = wide256 ? expert_product_wide_kernel<false, 256> : expert_product_wide_kernel<false, 128>;
         LLMB_CUDA(llmb::launch(up, dim3((F + GN / 2 - 1) / (GN / 2), tiles), dim3(G_THREADS), smem, stream, true, map_x, map_up,
                                (const int*)plan, E, max_tiles, 2 * F, F, (hidden + GK - 1) / GK, (B*)act, (float*)nullptr,
-                               (const int*)sorted, up_weights, status_dev));
+                               (const int*)sorted, up_weights, activation, status_dev));
         LLMB_CUDA(llmb::launch(down, dim3((hidden + GN - 1) / GN, tiles), dim3(G_THREADS), smem, stream, true, map_act, map_down,
                                (const int*)plan, E, max_tiles, hidden, hidden, (F + GK - 1) / GK, (B*)nullptr, y,
-                               (const int*)sorted, down_weights, status_dev));
+                               (const int*)sorted, down_weights, activation, status_dev));
     } else if (tc) {
         typedef __nv_bfloat16 B;
         LLMB_CUDA(llmb::launch(expert_product_tc_kernel<true>, dim3((F + 63) / 64, max_tiles), dim3(128), 0, stream, true,
                                (const B*)h, ld, top, (const B*)w_up, up_stride, F, hidden, (const int*)sorted,
-                               (const int*)plan, E, max_tiles, (B*)act, (float*)nullptr, up_weights));
+                               (const int*)plan, E, max_tiles, (B*)act, (float*)nullptr, up_weights, activation));
         LLMB_CUDA(llmb::launch(expert_product_tc_kernel<false>, dim3((hidden + 127) / 128, max_tiles), dim3(128), 0, stream,
                                true, (const B*)act, F, 1, (const B*)w_down, down_stride, hidden, F, (const int*)sorted,
-                               (const int*)plan, E, max_tiles, (B*)nullptr, y, down_weights));
+                               (const int*)plan, E, max_tiles, (B*)nullptr, y, down_weights, activation));
     } else if (dtype == LLMB_DTYPE_F32) {
         LLMB_CUDA(llmb::launch(expert_product_kernel<float, true>, grid_up, dim3(256), 0, stream, true, (const float*)h, ld,
                                top, (const float*)w_up, up_stride, F, hidden, (const int*)sorted, (const int*)plan, E,
-                               max_tiles, (float*)act, (float*)nullptr, up_weights));
+                               max_tiles, (float*)act, (float*)nullptr, up_weights, activation));
         LLMB_CUDA(llmb::launch(expert_product_kernel<float, false>, grid_down, dim3(256), 0, stream, true,
                                (const float*)act, F, 1, (const float*)w_down, down_stride, hidden, F, (const int*)sorted,
-                               (const int*)plan, E, max_tiles, (float*)nullptr, y, down_weights));
+                               (const int*)plan, E, max_tiles, (float*)nullptr, y, down_weights, activation));
     } else {
         typedef __nv_bfloat16 B;
         LLMB_CUDA(llmb::launch(expert_product_kernel<B, true>, grid_up, dim3(256), 0, stream, true, (const B*)h, ld, top,
                                (const B*)w_up, up_stride, F, hidden, (const int*)sorted, (const int*)plan, E, max_tiles,
-                               (B*)act, (float*)nullptr, up_weights));
+                               (B*)act, (float*)nullptr, up_weights, activation));
         LLMB_CUDA(llmb::launch(expert_product_kernel<B, false>, grid_down, dim3(256), 0, stream, true, (const B*)act, F, 1,
                                (const B*)w_down, down_stride, hidden, F, (const int*)sorted, (const int*)plan, E,
-                               max_tiles, (B*)nullptr, y, down_weights));
+                               max_tiles, (B*)nullptr, y, down_weights, activation));
     }
     return check_launch("routed_experts");
 }

@@ -30,6 +30,16 @@ class DecoderModel:
                     0 <= item.cache_of < i and spec.schedule[item.cache_of].cache_of is None):
                 raise FormatError(f"schedule entry {i} reads the cache of entry {item.cache_of}, "
                                   "which is not an earlier entry with a cache of its own")
+        self.streams = int(getattr(spec, "streams", 0))
+        if self.streams:
+            if any(getattr(b, "n_streams", 0) != self.streams for b in spec.blocks):
+                raise FormatError(f"a residual of {self.streams} streams needs every block to work on that many")
+            if any(getattr(item, "add_embedding", False) for item in spec.schedule):
+                raise FormatError("the embedding output cannot be added to a residual of several streams")
+            if not getattr(self.final_norm, "foldable", False):
+                raise FormatError("a residual of several streams needs an RMS norm at the end")
+        elif any(getattr(b, "n_streams", 0) for b in spec.blocks):
+            raise FormatError("blocks that work on several streams need a model whose residual has them")
         self.embedding = None
         self.head = None
         self.dtype = None
@@ -49,6 +59,7 @@ class DecoderModel:
     def libraries(self) -> list:
         """The kernel files a run of this model in its dtype needs (what gets compiled)."""
         names = ["elementwise", "gemm_simt", "gemm_skinny", "gemm_tc"]
+        names += ["streams"] if self.streams else []
         for block in self.blocks:
             names += list(block.libraries)
         names += list(self.final_norm.libraries)
@@ -201,7 +212,10 @@ class DecoderModel:
 
         emit = wanted_by(0)
         scale = getattr(self.spec, "embedding_scale", 1.0)
-        x = ops.embed(tokens, self.embedding, scale=scale, emit=for_product(emit))
+        if self.streams:
+            x = ops.streams_embed(tokens, self.embedding, self.streams, scale=scale)
+        else:
+            x = ops.embed(tokens, self.embedding, scale=scale, emit=for_product(emit))
         # the embedding output, for the runs that add it to the stream again (gathered a second time:
         # every operation of a pass is a launch of this library, so that the pass can be recorded)
         x0 = ops.embed(tokens, self.embedding, scale=scale) if any(added_before(i) for i in range(len(schedule))) else None
@@ -223,7 +237,10 @@ class DecoderModel:
                 emit = None
         if logit_rows.numel() == 0:
             return torch.empty((0, self.spec.vocab), dtype=torch.float32, device=x.device)
-        z = self.final_norm.forward(x, ctx.dtype, rows=logit_rows)
+        if self.streams:                               # the streams' sum, normed
+            z = ops.streams_read(x, None, self.final_norm.gain, self.final_norm.spec.eps, ctx.dtype, rows=logit_rows)
+        else:
+            z = self.final_norm.forward(x, ctx.dtype, rows=logit_rows)
         logits = ops.linear(z, self.head, out_dtype=torch.float32)
         if getattr(self.spec, "logit_scale", 1.0) != 1.0:
             ops.scale_(logits, self.spec.logit_scale)

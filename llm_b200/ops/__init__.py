@@ -417,7 +417,7 @@ def _check_rows(t, n: int, width: int, dtype, what: str):
 def norm_rope_cache_write(u, q_width, k_width, v_width, q_gain, k_gain, eps, rope_table, rot_unit, interleaved,
                           tok_pos, tok_seq, q_out, block_table, ring_pages, k_cache, v_cache, write_cache=True,
                           value_source=None, norm_unit: int = 0, mix_cache=None, mix_table=None, mix_ring: int = 0,
-                          mix: float = 0.0):
+                          mix: float = 0.0, q_scale=None):
     """What lies between a projection and the attention of a mixer that norms whole projections:
     the first q_width columns of `u` are the queries, the next k_width the keys, the next v_width
     the values (u may have more columns). With `q_gain` (float32 [q_width]) the queries of a token
@@ -432,8 +432,12 @@ def norm_rope_cache_write(u, q_width, k_width, v_width, q_gain, k_gain, eps, rop
     `norm_unit` > 0: the norms run over units of that many columns (a head each) with gains of norm_unit
     elements that all units share. `mix_cache` (a value cache of another layer, same shape as `v_cache`, with
     its page table `mix_table` and ring `mix_ring`): the values are blended before they are cached,
-    v <- (1 - mix) v + mix * (the row that cache holds for the same token), in 32-bit, rounded once."""
-    _require_cuda(u, q_gain, k_gain, rope_table, tok_pos, tok_seq, q_out, block_table, k_cache, v_cache, mix_cache, mix_table)
+    v <- (1 - mix) v + mix * (the row that cache holds for the same token), in 32-bit, rounded once.
+
+    `q_scale` (float32 [positions]): the queries are multiplied by the number of their position, behind the norm.
+    k_width == 0 (with v_width == 0 and without `write_cache`): `u` holds queries alone."""
+    _require_cuda(u, q_gain, k_gain, rope_table, tok_pos, tok_seq, q_out, block_table, k_cache, v_cache, mix_cache, mix_table,
+                  q_scale)
     n = q_out.shape[0]
     if value_source is None:
         value_source = q_width + k_width
@@ -458,8 +462,12 @@ def norm_rope_cache_write(u, q_width, k_width, v_width, q_gain, k_gain, eps, rop
                 or q_width % rot_unit or k_width % rot_unit):
             raise KernelError("norm_rope_cache_write: the table of angles must be contiguous float32 [positions, n_rot] "
                               f"with an even n_rot <= {rot_unit}, and the units must divide both widths")
-    if (k_cache.dtype != u.dtype or not k_cache.is_contiguous() or k_cache.shape[1] * k_cache.shape[3] != k_width
-            or k_cache.shape[2] != PAGE):
+    if q_scale is not None and (q_scale.dtype != torch.float32 or q_scale.dim() != 1 or not q_scale.is_contiguous()):
+        raise KernelError("norm_rope_cache_write: the queries' scale must be contiguous float32 [positions]")
+    if k_width == 0 and (write_cache or v_width):
+        raise KernelError("norm_rope_cache_write: without keys nothing is cached")
+    if k_width and (k_cache.dtype != u.dtype or not k_cache.is_contiguous() or k_cache.shape[1] * k_cache.shape[3] != k_width
+                    or k_cache.shape[2] != PAGE):
         raise KernelError(f"norm_rope_cache_write: the key cache {tuple(k_cache.shape)} does not fit keys of {k_width}")
     if v_width and (v_cache is None or v_cache.dtype != u.dtype or not v_cache.is_contiguous()
                     or v_cache.shape[1] * v_cache.shape[3] != v_width or v_cache.shape[2] != PAGE):
@@ -468,10 +476,11 @@ def norm_rope_cache_write(u, q_width, k_width, v_width, q_gain, k_gain, eps, rop
           _c_int(q_width), _c_int(k_width), _c_int(v_width), _ptr(q_gain), _ptr(k_gain), _c_float(eps),
           _ptr(rope_table), _c_int(n_rot), _c_int(rot_unit), _c_int(1 if interleaved else 0), _ptr(tok_pos),
           _ptr(tok_seq), _ptr(q_out), _c_int(q_out.stride(0)), _ptr(block_table), _c_int(block_table.shape[1]),
-          _c_int(ring_pages), _ptr(k_cache), _c_int(k_cache.shape[1]), _ptr(v_cache if v_width else None),
+          _c_int(ring_pages), _ptr(k_cache if k_width else None), _c_int(k_cache.shape[1] if k_width else 0),
+          _ptr(v_cache if v_width else None),
           _c_int(v_cache.shape[1] if v_width else 0), _c_int(1 if write_cache else 0), _c_int(value_source),
           _c_int(norm_unit), _ptr(mix_cache), _ptr(mix_table), _c_int(mix_table.shape[1] if mix_table is not None else 0),
-          _c_int(mix_ring), _c_float(mix), _c_int(n), _stream())
+          _c_int(mix_ring), _c_float(mix), _ptr(q_scale), _c_int(n), _stream())
     return q_out
 
 
@@ -620,6 +629,70 @@ def fill_(x, value: float):
     return x
 
 
+# ----------------------------------------------------------------------------- residual of several streams
+
+MAX_STREAMS = 16       # streams the kernels of csrc/streams.cu take
+
+
+def streams_embed(tokens, table, n_streams: int, scale: float = 1.0):
+    """X[t, s, :] = table[tokens[t], :] * scale for every stream s, float32 [T, n_streams, hidden]."""
+    _require_cuda(tokens, table)
+    n, (vocab, hidden) = tokens.numel(), table.shape
+    out = torch.empty((n, n_streams, hidden), dtype=torch.float32, device=table.device)
+    _call("streams", "llmb_streams_embed", _ptr(tokens), _ptr(table), _c_int(_code(table.dtype)), _ptr(out), _c_int(n),
+          _c_int(n_streams), _c_int(hidden), _c_int(vocab), _c_float(scale), _stream())
+    return out
+
+
+def _check_streams(X, what: str):
+    _require_cuda(X)
+    if X.dtype != torch.float32 or X.dim() != 3 or not X.is_contiguous():
+        raise KernelError(f"{what}: the streams must be contiguous float32 [T, streams, hidden]")
+    return X.shape
+
+
+def _check_vector(t, count: int, what: str):
+    _require_cuda(t)
+    if t.dtype != torch.float32 or t.numel() != count or not t.is_contiguous():
+        raise KernelError(f"{what} must be contiguous float32 with {count} elements")
+
+
+def streams_update_(X, y, terms: int, write, read=None, gain=None, eps: float = 0.0, out=None):
+    """Behind a part: X[t, j] <- sum_s mix[s, j] X[t, s] + spread[j] * sum_k y[t * terms + k], all from the old streams
+    (X float32 [T, S, hidden], y float32 [T * terms, hidden], `write` float32 [S + S * S]: spread, then mix row by row). With
+    `out` [T, hidden] (run dtype) also the next part's input, of the new streams: u = sum_s read[s] X[t, s],
+    out[t] = u / sqrt(mean(u^2) + eps) * gain (`read` float32 [S], `gain` float32 [hidden])."""
+    n, S, hidden = _check_streams(X, "streams_update_")
+    _require_cuda(y, out)
+    if y.dtype != torch.float32 or tuple(y.shape) != (n * terms, hidden) or not y.is_contiguous():
+        raise KernelError(f"streams_update_: the result must be contiguous float32 [{n * terms}, {hidden}]")
+    _check_vector(write, S + S * S, "streams_update_: the weights of the streams")
+    if out is not None:
+        _check_vector(read, S, "streams_update_: the weights of the input")
+        _check_vector(gain, hidden, "streams_update_: the gain")
+        _check_out(out, (n, hidden), out.dtype, "streams_update_")
+    _call("streams", "llmb_streams", _ptr(X), _c_int(S), _ptr(y), _c_int(terms), _ptr(write), _ptr(read if out is not None else None),
+          _ptr(gain if out is not None else None), _c_float(eps), None, _ptr(out), _c_int(_code(out.dtype) if out is not None else 0),
+          _c_int(n), _c_int(hidden), _stream())
+    return out
+
+
+def streams_read(X, read, gain, eps: float, out_dtype, rows=None, out=None):
+    """out[r] = u / sqrt(mean(u^2) + eps) * gain with u = sum_s read[s] X[rows[r] or r, s] (`read` None: the plain sum)."""
+    n, S, hidden = _check_streams(X, "streams_read")
+    _require_cuda(rows, out)
+    count = rows.numel() if rows is not None else n
+    if read is not None:
+        _check_vector(read, S, "streams_read: the weights of the streams")
+    _check_vector(gain, hidden, "streams_read: the gain")
+    _check_out(out, (count, hidden), out_dtype, "streams_read")
+    if out is None:
+        out = torch.empty((count, hidden), dtype=out_dtype, device=X.device)
+    _call("streams", "llmb_streams", _ptr(X), _c_int(S), None, _c_int(0), None, _ptr(read), _ptr(gain), _c_float(eps), _ptr(rows),
+          _ptr(out), _c_int(_code(out_dtype)), _c_int(count), _c_int(hidden), _stream())
+    return out
+
+
 # ----------------------------------------------------------------------------- gated delta rule
 
 def delta_rule_work_width(n_heads: int, n_kv_heads: int, dim: int, vdim: int) -> int:
@@ -755,6 +828,46 @@ def forget_recurrence(proj, f_bias, lower, state, cu_seqlens, slot_ids, norm_wei
     return mixed
 
 
+# ----------------------------------------------------------------------------- recurrence with a fixed decay per head
+
+def decay_recurrence_work_width(n_heads: int, dim: int, vdim: int) -> int:
+    """Floats of a token's 32-bit work row: k, q and v."""
+    return (2 * n_heads * dim + n_heads * vdim + 3) // 4 * 4
+
+
+def decay_recurrence(proj, decays, state, cu_seqlens, slot_ids, norm_weight, eps, work, o, mixed, n_heads, dim, vdim,
+                     single_tokens=False):
+    """Linear attention with one fixed decay per head, behind its projection. `proj` [T, >= 2 H D + 2 H V] (run dtype, rows
+    contiguous) holds per token [q (H D) | k (H D) | v (H V) | gate (H V)]; q, k, v <- silu; per head
+    S_t = decay S_(t-1) + k_t v_t^T, o_t = S_t^T q_t (`decays` float32 [H]); then the concatenated heads
+    o / sqrt(mean(o^2) + eps) * norm_weight * sigmoid(gate) (norm_weight float32 [H V]) into `mixed` [T, H V] (run dtype).
+    `state` float32 [slots, H V D]: S as [H, V, D], read and updated for the slots of the step. `work` float32
+    [T, decay_recurrence_work_width], `o` float32 [T, H V]: scratch. `single_tokens`: every sequence brings exactly one
+    token (token b is sequence b's)."""
+    _require_cuda(proj, decays, state, cu_seqlens, slot_ids, norm_weight, work, o, mixed)
+    n, H, D, V = proj.shape[0], n_heads, dim, vdim
+    if proj.dim() != 2 or proj.shape[1] < 2 * H * (D + V) or proj.stride(1) != 1:
+        raise KernelError(f"decay_recurrence: the projection {tuple(proj.shape)} does not hold {2 * H * (D + V)} columns")
+    _check_rows(mixed, n, H * V, proj.dtype, "decay_recurrence: mixed")
+    for t, shape, what in ((decays, (H,), "decays"), (norm_weight, (H * V,), "norm weight"), (o, (n, H * V), "o")):
+        if t.dtype != torch.float32 or tuple(t.shape) != shape or not t.is_contiguous():
+            raise KernelError(f"decay_recurrence: {what} must be contiguous float32 {shape}")
+    width = decay_recurrence_work_width(H, D, V)
+    if work.dtype != torch.float32 or work.dim() != 2 or work.shape[0] < n or work.shape[1] < width or not work.is_contiguous():
+        raise KernelError(f"decay_recurrence: work must be contiguous float32 [T, >= {width}]")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.shape[1] < H * D * V or state.stride(1) != 1:
+        raise KernelError(f"decay_recurrence: the state must be float32 [slots, >= {H * D * V}]")
+    n_seqs = cu_seqlens.numel() - 1
+    warps = (V + 7) // 8
+    one = single_tokens and n == n_seqs and warps <= 32 and D <= 256 and not (D > 128 and warps > 16)
+    _call("decay_recurrence", "llmb_decay_recurrence", _ptr(proj), _c_int(proj.stride(0)), _c_int(_code(proj.dtype)),
+          _ptr(decays), _ptr(state), ctypes.c_longlong(state.stride(0)), _ptr(cu_seqlens), _ptr(slot_ids),
+          _ptr(norm_weight), _c_float(eps), _ptr(work), _c_int(work.shape[1]), _ptr(o), _ptr(mixed), _c_int(mixed.stride(0)),
+          _c_int(n), _c_int(n_seqs), _c_int(H), _c_int(D), _c_int(V), _c_int(1 if single_tokens else 0), _stream(),
+          kernels=2 if one else 3)
+    return mixed
+
+
 # ----------------------------------------------------------------------------- routed experts
 
 #: how a router scores and weights its outputs (RoutedExpertsSpec.scoring), by the number the kernel takes
@@ -782,7 +895,7 @@ def routed_experts_wide(n_tokens: int, top: int, n_experts: int, hidden: int, in
 
 def routed_experts(h, router, router_bias, w_up, w_down, top: int, ids, weights, order, plan, act, y, gathered=None,
                    scoring: int = 0, correction=None, pass_through: int = 0, weight_scale: float = 1.0,
-                   weight_on_input: bool = False):
+                   weight_on_input: bool = False, groups: int = 1, keep: int = 1, limit: float = -1.0, alpha: float = 1.0):
     """A feed-forward of routed experts on the rows of h [T, hidden] (run dtype). Router logits
     z = router h + router_bias in 32-bit (`router` float32 [E, hidden]); the `top` largest are chosen and
     weighted by the softmax over them. Expert e: W_down,e (silu(W_gate,e h) * (W_up,e h)) with `w_up`
@@ -796,7 +909,11 @@ def routed_experts(h, router, router_bias, w_up, w_down, top: int, ids, weights,
     per output; it takes part in the choice only) are chosen, weights s / (sum of the chosen s + 1e-20).
     `pass_through` > 0: the router has E + pass_through outputs, and the last ones are experts without matrices
     whose result is h itself. `weight_scale` multiplies every weight. `scoring` 2: scores s = sigmoid(z), the `top`
-    largest chosen, weights s as they are. `weight_on_input`: y[t * top + k] = expert(weight[t, k] h[t]) instead."""
+    largest chosen, weights s as they are. `weight_on_input`: y[t * top + k] = expert(weight[t, k] h[t]) instead.
+
+    `groups` > 1 (scoring 1): the outputs form that many equal groups of neighbours, a group's score is its largest, and
+    only outputs of the `keep` best groups can be chosen. `limit` >= 0: the experts' activation is the clamped one,
+    g <- min(g, limit), u <- clamp(u, -limit, limit), g sigmoid(alpha g) (u + 1)."""
     _require_cuda(h, router, router_bias, w_up, w_down, ids, weights, order, plan, act, y, gathered, correction)
     n, hidden = h.shape
     E, two_f, _ = w_up.shape
@@ -825,7 +942,7 @@ def routed_experts(h, router, router_bias, w_up, w_down, top: int, ids, weights,
           _ptr(router_bias), _ptr(w_up), _ptr(w_down), _ptr(ids), _ptr(weights), _ptr(order), _ptr(plan), _ptr(act),
           _ptr(y), _ptr(gathered if wide else None), _c_int(n), _c_int(hidden), _c_int(F), _c_int(E), _c_int(top),
           _c_int(level), _c_int(scoring), _ptr(correction), _c_int(pass_through), _c_float(weight_scale),
-          _c_int(1 if weight_on_input else 0), _stream(),
+          _c_int(1 if weight_on_input else 0), _c_int(groups), _c_int(keep), _c_float(limit), _c_float(alpha), _stream(),
           kernels=(5 if wide else 4) + (1 if pass_through else 0))
     return y
 
@@ -1187,7 +1304,7 @@ def attention_decode_splits(n_seqs: int, n_heads: int, n_kv_heads: int, max_len:
 def attention(qkv, k_cache, v_cache, block_table, ring_pages, tok_pos, tok_seq, n_heads,
               n_kv_heads, head_dim, scale, window=0, out=None, decode=False, seq_lens=None,
               max_len=0, cu_seqlens=None, max_new=0, seq_order=None, sinks=None, gate=None, out_scale=1.0,
-              softcap=0.0, value_dim=None):
+              softcap=0.0, value_dim=None, bias=None):
     """Causal grouped-query attention of the new tokens' queries (the first
     Hq * D columns of `qkv`) over the paged cache, which already holds the new
     tokens' keys and values. Returns [T, Hq * D] in qkv's dtype. `seq_order`
@@ -1200,11 +1317,18 @@ def attention(qkv, k_cache, v_cache, block_table, ring_pages, tok_pos, tok_seq, 
     result. With any of the three, `out` may be a range of columns of a wider buffer. The value
     cache may be the key cache itself (a mixer whose values are its keys). `softcap` > 0 bounds the scaled
     scores before the softmax: s <- softcap * tanh(s / softcap). `value_dim` (default head_dim): the size of a
-    value where it differs from a key's; the result is then [T, Hq * value_dim] (the kernel for any sizes)."""
-    _require_cuda(qkv, k_cache, v_cache, block_table, tok_pos, tok_seq, sinks, gate)
+    value where it differs from a key's; the result is then [T, Hq * value_dim] (the kernel for any sizes).
+    `bias` (float32 [Hq, span], without a soft cap): bias[a, min(p - j, span - 1)] is added to head a's scaled score of
+    the key at position j for the query at position p."""
+    _require_cuda(qkv, k_cache, v_cache, block_table, tok_pos, tok_seq, sinks, gate, bias)
     n = qkv.shape[0]
     value_dim = value_dim or head_dim
-    extras = (sinks is not None or gate is not None or out_scale != 1.0 or softcap > 0.0 or value_dim != head_dim
+    span = 0
+    if bias is not None:
+        if bias.dtype != torch.float32 or bias.dim() != 2 or bias.shape[0] != n_heads or not bias.is_contiguous() or softcap > 0.0:
+            raise KernelError(f"attention: a bias must be contiguous float32 [{n_heads}, span], without a soft cap")
+        span = bias.shape[1]
+    extras = (sinks is not None or bias is not None or gate is not None or out_scale != 1.0 or softcap > 0.0 or value_dim != head_dim
               or (out is not None and not out.is_contiguous()))
     if extras:
         if out is not None:
@@ -1220,8 +1344,8 @@ def attention(qkv, k_cache, v_cache, block_table, ring_pages, tok_pos, tok_seq, 
     variant = tactics.choose_attention(decode, qkv.dtype, n_heads, n_kv_heads, head_dim, window,
                                        cu_seqlens is not None and seq_lens is not None,
                                        qkv.stride(0) % 8 == 0 and qkv.data_ptr() % 16 == 0)
-    # the tcgen05 prefill takes a sink, none of the others
-    sink_only = (sinks is not None and gate is None and out_scale == 1.0 and softcap <= 0.0 and value_dim == head_dim
+    # the tcgen05 prefill takes a sink and a bias, none of the others
+    sink_only = ((sinks is not None or bias is not None) and gate is None and out_scale == 1.0 and softcap <= 0.0 and value_dim == head_dim
                  and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0)
     if extras and variant not in _ATTENTION_WITH_EXTRAS and not (variant == "attention_prefill_tc" and sink_only):
         # the next choice that takes a sink, a gate, a scale and rows inside a wider buffer
@@ -1240,19 +1364,20 @@ def attention(qkv, k_cache, v_cache, block_table, ring_pages, tok_pos, tok_seq, 
               _c_int(block_table.shape[1]), _c_int(ring_pages), _ptr(cu_seqlens), _ptr(seq_lens),
               _ptr(seq_order), _ptr(out), _c_int(out.stride(0)), _c_int(cu_seqlens.numel() - 1),
               _c_int(max_new), _c_int(n_heads), _c_int(n_kv_heads), _c_int(head_dim), _c_float(scale),
-              _c_int(window), _ptr(sinks), _stream())
+              _c_int(window), _ptr(sinks), _ptr(bias), _c_int(span), _stream())
     elif variant == "attention_prefill":
         _call("attention_prefill", "llmb_attention_prefill", _ptr(qkv), _c_int(qkv.stride(0)),
               _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _c_int(block_table.shape[1]),
               _c_int(ring_pages), _ptr(cu_seqlens), _ptr(seq_lens), _ptr(out), _c_int(out.stride(0)),
               _c_int(cu_seqlens.numel() - 1), _c_int(max_new), _c_int(n_heads), _c_int(n_kv_heads),
               _c_int(head_dim), _c_float(scale), _c_int(window), _ptr(sinks), _ptr(gate),
-              _c_int(gate.stride(0) if gate is not None else 0), _c_float(out_scale), _c_float(softcap), _stream())
+              _c_int(gate.stride(0) if gate is not None else 0), _c_float(out_scale), _c_float(softcap), _ptr(bias),
+              _c_int(span), _stream())
     elif variant == "attention_decode":
         # the plain grouped-query case keeps the kernel file it was tuned in; a window, a sink, a gate, a scale, a
         # value cache that is the key cache and groups above 8 run the same kernel with those additions
         plain = (window == 0 and sinks is None and gate is None and out_scale == 1.0 and n_heads // n_kv_heads <= 8
-                 and softcap <= 0.0 and k_cache.data_ptr() != v_cache.data_ptr())
+                 and softcap <= 0.0 and bias is None and k_cache.data_ptr() != v_cache.data_ptr())
         name = "attention_decode" if plain else "attention_decode_window"
         splits = attention_decode_splits(n, n_heads, n_kv_heads, max_len, window)
         lib = load_library(name)
@@ -1275,8 +1400,8 @@ def attention(qkv, k_cache, v_cache, block_table, ring_pages, tok_pos, tok_seq, 
             _call(name, "llmb_attention_decode", *head, _c_int(splits), _stream(), kernels=2 if splits > 1 else 1)
         else:
             _call(name, "llmb_attention_decode_window", *head, _ptr(sinks), _ptr(gate),
-                  _c_int(gate.stride(0) if gate is not None else 0), _c_float(out_scale), _c_float(softcap),
-                  _c_int(splits), _stream(), kernels=2 if splits > 1 else 1)
+                  _c_int(gate.stride(0) if gate is not None else 0), _c_float(out_scale), _c_float(softcap), _ptr(bias),
+                  _c_int(span), _c_int(splits), _stream(), kernels=2 if splits > 1 else 1)
     elif variant == "attention_generic":
         _call("attention_generic", "llmb_attention_generic", _ptr(qkv), _c_int(qkv.stride(0)),
               _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _c_int(block_table.shape[1]),
@@ -1284,7 +1409,7 @@ def attention(qkv, k_cache, v_cache, block_table, ring_pages, tok_pos, tok_seq, 
               _c_int(_code(qkv.dtype)), _c_int(n), _c_int(n_heads), _c_int(n_kv_heads),
               _c_int(head_dim), _c_float(scale), _c_int(window), _ptr(sinks), _ptr(gate),
               _c_int(gate.stride(0) if gate is not None else 0), _c_float(out_scale), _c_float(softcap),
-              _c_int(value_dim), _stream())
+              _c_int(value_dim), _ptr(bias), _c_int(span), _stream())
     else:
         raise KernelError(f"attention: no kernel named {variant}")
     return out
@@ -1305,31 +1430,62 @@ def attention_replay_key(step, n_heads: int, n_kv_heads: int, window: int = 0):
 # ----------------------------------------------------------------------------- latent attention, shared rotated keys
 
 def latent_write(u, n_heads, dim, rot, rank, gain, eps, rope_table, interleaved, tok_pos, tok_seq, block_table, ring_pages,
-                 cache, queries=None, dense=None, write_cache=True):
+                 cache, queries=None, dense=None, write_cache=True, q_rank=0, q_gain=None, cq=None):
     """Behind the projection of a latent attention: `u` [T, >= H (D + R) + C + R] holds per token H query heads of
     [D | R] elements, the latent c (C) and a rotated key part r (R) that all heads share. c / sqrt(mean(c^2) + eps) * gain
     and the rotated r go as one row [C | R] into `cache` [pages, 1, 64, C + R] (unless `write_cache` is False) and, where given, into
     `dense` [T, C + R]. The query heads' last R elements rotate: into the last R columns of `queries` [T, H (C + R)], or,
-    without it, where they are. `rope_table` float32 [positions, n_rot], n_rot <= R, or None. Norm and angles are 32-bit."""
-    _require_cuda(u, gain, rope_table, tok_pos, tok_seq, block_table, cache, queries, dense)
+    without it, where they are. `rope_table` float32 [positions, n_rot], n_rot <= R, or None. Norm and angles are 32-bit.
+
+    With `q_rank` > 0 the first q_rank columns of `u` are the queries' latent instead of query heads: normed with `q_gain`
+    (float32 [q_rank]) into `cq` [T, q_rank]; the query heads come from a product of it (latent_rotate)."""
+    _require_cuda(u, gain, rope_table, tok_pos, tok_seq, block_table, cache, queries, dense, q_gain, cq)
     n, width = u.shape[0], rank + rot
-    if u.dim() != 2 or u.stride(1) != 1 or u.shape[1] < n_heads * (dim + rot) + width:
-        raise KernelError(f"latent_write: u {tuple(u.shape)} does not hold {n_heads} heads of {dim} + {rot} and {rank} + {rot}")
+    front = q_rank if q_rank else n_heads * (dim + rot)
+    if u.dim() != 2 or u.stride(1) != 1 or u.shape[1] < front + width:
+        raise KernelError(f"latent_write: u {tuple(u.shape)} does not hold {front} columns and {rank} + {rot}")
     if gain.dtype != torch.float32 or gain.numel() != rank:
         raise KernelError(f"latent_write: the gain must be float32 [{rank}]")
+    if q_rank and (q_gain is None or cq is None or q_gain.dtype != torch.float32 or q_gain.numel() != q_rank
+                   or tuple(cq.shape) != (n, q_rank) or cq.dtype != u.dtype or not cq.is_contiguous() or queries is not None):
+        raise KernelError(f"latent_write: the queries' latent needs a float32 gain [{q_rank}] and a contiguous result [{n}, {q_rank}]")
     if tuple(cache.shape[1:]) != (1, PAGE, width) or cache.dtype != u.dtype or not cache.is_contiguous():
         raise KernelError(f"latent_write: the cache {tuple(cache.shape)} does not hold rows of {width}")
     for t, shape, what in ((queries, (n, n_heads * width), "queries"), (dense, (n, width), "dense")):
         if t is not None and (tuple(t.shape) != shape or t.dtype != u.dtype or not t.is_contiguous()):
             raise KernelError(f"latent_write: {what} must be contiguous {u.dtype} {shape}")
-    if rope_table is not None and (rope_table.dtype != torch.float32 or not rope_table.is_contiguous()
-                                   or rope_table.shape[1] > rot or rope_table.shape[1] % 2):
-        raise KernelError(f"latent_write: the table of angles must be contiguous float32 [positions, n_rot <= {rot}]")
-    _call("latent_attention", "llmb_latent_write", _ptr(u), _c_int(u.stride(0)), _c_int(_code(u.dtype)), _c_int(n_heads),
-          _c_int(dim), _c_int(rot), _c_int(rank), _ptr(gain), _c_float(eps), _ptr(rope_table),
-          _c_int(rope_table.shape[1] if rope_table is not None else 0), _c_int(1 if interleaved else 0), _ptr(tok_pos),
+    n_rot = _latent_angles(rope_table, rot)
+    _call("latent_attention", "llmb_latent_write", _ptr(u), _c_int(u.stride(0)), _c_int(_code(u.dtype)), _c_int(front),
+          _c_int(q_rank), _ptr(q_gain), _ptr(cq), None if q_rank else _ptr(u), _c_int(u.stride(0)), _c_int(n_heads),
+          _c_int(dim), _c_int(rot), _c_int(rank), _ptr(gain), _c_float(eps), _ptr(rope_table), _c_int(n_rot),
+          _c_int(1 if interleaved else 0), _ptr(tok_pos),
           _ptr(tok_seq), _ptr(block_table), _c_int(block_table.shape[1]), _c_int(ring_pages), _ptr(cache),
           _c_int(1 if write_cache else 0), _ptr(queries), _ptr(dense), _c_int(n), _stream())
+
+
+def _latent_angles(rope_table, rot: int) -> int:
+    if rope_table is None:
+        return 0
+    if (rope_table.dtype != torch.float32 or not rope_table.is_contiguous() or rope_table.shape[1] > rot
+            or rope_table.shape[1] % 2):
+        raise KernelError(f"latent_write: the table of angles must be contiguous float32 [positions, n_rot <= {rot}]")
+    return rope_table.shape[1]
+
+
+def latent_rotate(heads, n_heads, dim, rot, rank, rope_table, interleaved, tok_pos, queries=None):
+    """The rotated parts of the query heads `heads` [T, H (D + R)] alone: into the last R columns of every head of `queries`
+    [T, H (C + R)], or, without it, where they are."""
+    _require_cuda(heads, rope_table, tok_pos, queries)
+    n, width = heads.shape[0], rank + rot
+    if tuple(heads.shape) != (n, n_heads * (dim + rot)) or heads.stride(1) != 1:
+        raise KernelError(f"latent_rotate: {tuple(heads.shape)} are not {n_heads} heads of {dim} + {rot}")
+    if queries is not None and (tuple(queries.shape) != (n, n_heads * width) or queries.dtype != heads.dtype or not queries.is_contiguous()):
+        raise KernelError(f"latent_rotate: queries must be contiguous {heads.dtype} [{n}, {n_heads * width}]")
+    n_rot = _latent_angles(rope_table, rot)
+    _call("latent_attention", "llmb_latent_write", None, _c_int(0), _c_int(_code(heads.dtype)), _c_int(-1), _c_int(0), None, None,
+          _ptr(heads), _c_int(heads.stride(0)), _c_int(n_heads), _c_int(dim), _c_int(rot), _c_int(rank), None, _c_float(0.0),
+          _ptr(rope_table), _c_int(n_rot), _c_int(1 if interleaved else 0), _ptr(tok_pos), None, None, _c_int(0), _c_int(1),
+          None, _c_int(0), _ptr(queries), None, _c_int(n), _stream())
 
 
 def head_products(x, x_head: int, w, out, out_head: int):
@@ -1367,10 +1523,17 @@ def latent_attention_replay_key(step, n_heads: int):
     return (False, max(step.new_counts))
 
 
+def _check_sinks(sinks, n_heads: int, what: str):
+    if sinks is not None:
+        _check_vector(sinks, n_heads, f"{what}: sinks")
+
+
 def latent_attention(queries, cache, block_table, ring_pages, tok_pos, tok_seq, n_heads, rank, rot, scale, out, decode=False,
-                     seq_lens=None, max_len=0, cu_seqlens=None, max_new=0, seq_order=None):
+                     seq_lens=None, max_len=0, cu_seqlens=None, max_new=0, seq_order=None, sinks=None):
     """Causal softmax attention of the new tokens' latent queries [T, H (C + R)] over the cached rows [pages, 1, 64, C + R],
-    whose first C elements are the values: out[t, h * C :] = sum_j softmax_j(scale q_h . row_j) row_j[:C]."""
+    whose first C elements are the values: out[t, h * C :] = sum_j softmax_j(scale q_h . row_j) row_j[:C]. `sinks` (float32
+    [H]): e^sinks[h] is one more term of head h's denominator."""
+    _check_sinks(sinks, n_heads, "latent_attention")
     _require_cuda(queries, cache, block_table, tok_pos, tok_seq, out)
     n, width = queries.shape[0], rank + rot
     if tuple(queries.shape) != (n, n_heads * width) or not queries.is_contiguous():
@@ -1383,7 +1546,8 @@ def latent_attention(queries, cache, block_table, ring_pages, tok_pos, tok_seq, 
         _call("attention_generic", "llmb_attention_generic", _ptr(queries), _c_int(queries.stride(0)), _ptr(cache), _ptr(cache),
               _ptr(block_table), _c_int(block_table.shape[1]), _c_int(ring_pages), _ptr(tok_pos), _ptr(tok_seq), _ptr(out),
               _c_int(out.stride(0)), _c_int(_code(queries.dtype)), _c_int(n), _c_int(n_heads), _c_int(1), _c_int(width),
-              _c_float(scale), _c_int(0), None, None, _c_int(0), _c_float(1.0), _c_float(0.0), _c_int(rank), _stream())
+              _c_float(scale), _c_int(0), _ptr(sinks), None, _c_int(0), _c_float(1.0), _c_float(0.0), _c_int(rank), None, _c_int(0),
+              _stream())
         return out
     splits, scratch = 1, None
     if decode:
@@ -1402,20 +1566,22 @@ def latent_attention(queries, cache, block_table, ring_pages, tok_pos, tok_seq, 
             _call("latent_attention", "llmb_latent_decode_tc", _ptr(queries), _ptr(cache), _c_int(cache.shape[0]),
                   _ptr(block_table), _c_int(block_table.shape[1]), _c_int(ring_pages), _ptr(seq_lens), _ptr(seq_order), _ptr(out),
                   _ptr(scratch), ctypes.c_longlong(scratch.numel()), _c_int(n), _c_int(n_heads), _c_int(rank), _c_int(rot),
-                  _c_float(scale), _c_int(splits), _stream(), kernels=2 if splits > 1 else 1)
+                  _c_float(scale), _ptr(sinks), _c_int(splits), _stream(), kernels=2 if splits > 1 else 1)
             return out
     _call("latent_attention", "llmb_latent_attention", _ptr(queries), _ptr(cache), _ptr(block_table), _c_int(block_table.shape[1]),
           _c_int(ring_pages), _ptr(cu_seqlens), _ptr(seq_lens), _ptr(seq_order), _ptr(out), _ptr(scratch),
           ctypes.c_longlong(scratch.numel() if scratch is not None else 0), _c_int(n), _c_int(cu_seqlens.numel() - 1),
-          _c_int(1 if decode else max_new), _c_int(n_heads), _c_int(rank), _c_int(rot), _c_float(scale), _c_int(splits), _stream(),
+          _c_int(1 if decode else max_new), _c_int(n_heads), _c_int(rank), _c_int(rot), _c_float(scale), _ptr(sinks), _c_int(splits), _stream(),
           kernels=2 if splits > 1 else 1)
     return out
 
 
-def latent_prefill(proj, kv, dense, n_heads, dim, rot, vdim, rank, scale, out, cu_seqlens, max_new, seq_order=None):
+def latent_prefill(proj, kv, dense, n_heads, dim, rot, vdim, rank, scale, out, cu_seqlens, max_new, seq_order=None, sinks=None):
     """Causal softmax attention of packed prompts that all start at their first token, with the keys and values of every
     head formed: head h's queries are columns h (D + R).. of `proj` (rotated), its keys [D columns h (D + V).. of `kv` | the
-    last R columns of `dense` [T, C + R]], its values the V columns behind them in `kv`. Result [T, H V] into `out`."""
+    last R columns of `dense` [T, C + R]], its values the V columns behind them in `kv`. Result [T, H V] into `out`. `sinks` as
+    in latent_attention."""
+    _check_sinks(sinks, n_heads, "latent_prefill")
     _require_cuda(proj, kv, dense, out, cu_seqlens)
     n = proj.shape[0]
     if tuple(kv.shape) != (n, n_heads * (dim + vdim)) or tuple(dense.shape) != (n, rank + rot) or not kv.is_contiguous() \
@@ -1424,7 +1590,7 @@ def latent_prefill(proj, kv, dense, n_heads, dim, rot, vdim, rank, scale, out, c
     _check_rows(out, n, n_heads * vdim, proj.dtype, "latent_prefill: out")
     _call("latent_prefill_tc", "llmb_latent_prefill_tc", _ptr(proj), _c_int(proj.stride(0)), _ptr(kv), _ptr(dense), _c_int(n),
           _ptr(cu_seqlens), _ptr(seq_order), _ptr(out), _c_int(out.stride(0)), _c_int(cu_seqlens.numel() - 1), _c_int(max_new),
-          _c_int(n_heads), _c_int(dim), _c_int(rot), _c_int(vdim), _c_int(rank), _c_float(scale), _stream())
+          _c_int(n_heads), _c_int(dim), _c_int(rot), _c_int(vdim), _c_int(rank), _c_float(scale), _ptr(sinks), _stream())
     return out
 
 

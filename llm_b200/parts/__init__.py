@@ -4,7 +4,8 @@ from .base import (Block, FeedForward, Mixer, Norm, Part, PositionEncoding, Step
                    register_block, register_feed_forward, register_mixer, register_norm,
                    register_position)
 from .attention import AttentionMixer
-from .block import OutputNormBlock, ParallelBlock, PreNormBlock, SandwichBlock
+from .block import OutputNormBlock, ParallelBlock, PreNormBlock, SandwichBlock, StreamsBlock
+from .decay_recurrence import DecayRecurrenceMixer
 from .delta_rule import DeltaRuleMixer
 from .diff_attention import DiffAttentionMixer
 from .feedforward import GatedMlp, Mlp
@@ -28,4 +29,4 @@ __all__ = ["spec", "Block", "FeedForward", "Mixer", "Norm", "Part", "PositionEnc
            "RmsNorm", "Rope", "inverse_frequencies", "TanhNorm", "ProjectedMixer", "LatentAttentionMixer",
            "SigmoidAttentionMixer", "GatedRecurrenceMixer", "SideBySideMixer", "SandwichBlock", "DeltaRuleMixer",
            "GatedAttentionMixer", "Mlp", "RoutedExperts", "StateSpaceMixer", "OutputNormBlock", "LayerNorm",
-           "ForgetRecurrenceMixer", "RotaryLatentMixer"]
+           "ForgetRecurrenceMixer", "RotaryLatentMixer", "StreamsBlock", "DecayRecurrenceMixer"]

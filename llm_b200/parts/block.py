@@ -687,3 +687,177 @@ class OutputNormBlock(Block):
 
 
 register_block("output_norm", OutputNormBlock)
+
+
+class StreamsBlock(Block):
+    """A residual of several streams X [T, n, size] (32-bit): a part reads norm(sum_s in[s] x_s), and its result y and the
+    old streams give the new ones, x_t <- sum_s mix[s, t] x_s + out[t] y (Zhu et al., "Hyper-Connections").
+
+    A part's result is a stream of its own (`y`, possibly several rows a token that the kernel adds in index order). Launches
+    beside the parts': behind each part ONE kernel that forms the new streams and, in the same pass over them, the
+    weighted sum and norm that the next part reads (the feed-forward's, or the first of the block that runs next, which asks
+    for it through `input_emit`); the first part of a model reads the streams by a launch of its own."""
+
+    chains_norms = True
+
+    def __init__(self, spec):
+        self.spec = spec
+        self.mixer_norm = build_norm(spec.mixer_norm)
+        self.mixer = build_mixer(spec.mixer)
+        self.feed_forward = build_feed_forward(spec.feed_forward) if spec.feed_forward is not None else None
+        self.ffn_norm = build_norm(spec.ffn_norm) if self.feed_forward is not None else None
+        if not 1 <= spec.n_streams <= ops.MAX_STREAMS:
+            raise Unsupported(f"a residual of {spec.n_streams} streams (1 to {ops.MAX_STREAMS} are built)")
+        for norm in (self.mixer_norm, self.ffn_norm):
+            if norm is not None and not getattr(norm, "foldable", False):
+                raise Unsupported("a block of several streams needs RMS norms (a gain and an eps) in front of its parts")
+        for part in (self.mixer, self.feed_forward):
+            if part is not None and part.result_extra:
+                raise Unsupported("a block of several streams adds a token's result rows in one run: no row of its own behind them")
+        self.read = [None, None]           # per part: in [n]
+        self.write = [None, None]          # per part: [out (n) | mix (n * n)]
+
+    @property
+    def size(self):
+        return self.spec.mixer_norm.size
+
+    @property
+    def parts(self):
+        return tuple(p for p in (self.mixer_norm, self.mixer, self.ffn_norm, self.feed_forward) if p is not None)
+
+    @property
+    def graph_safe(self):
+        return all(p.graph_safe for p in self.parts)
+
+    @property
+    def libraries(self):
+        return ("streams", "post_norm") + tuple(lib for p in self.parts for lib in p.libraries)
+
+    def _stream_names(self):
+        s = self.spec
+        return [dict(s.mixer_streams)] + ([dict(s.ffn_streams)] if self.feed_forward is not None else [])
+
+    def parameters(self):
+        from ..weights.loader import ParamSpec
+        n, out = self.spec.n_streams, {}
+        for p in self.parts:
+            out.update(p.parameters())
+        for t in self._stream_names():
+            out.update({t["in"]: ParamSpec((n,), "streams"), t["out"]: ParamSpec((n,), "streams"),
+                        t["mix"]: ParamSpec((n, n), "streams")})
+        return out
+
+    def bind(self, tensors, dtype, device):
+        for p in self.parts:
+            p.bind(tensors, dtype, device)
+        for i, t in enumerate(self._stream_names()):
+            self.read[i] = to_float32(tensors[t["in"]], device)
+            self.write[i] = torch.cat([to_float32(tensors[t["out"]], device), to_float32(tensors[t["mix"]], device).reshape(-1)])
+
+    def replay_key(self, step):
+        keys = [p.replay_key(step) for p in self.parts]
+        return None if any(k is None for k in keys) else tuple(keys)
+
+    def prepare(self, max_positions, device):
+        for p in self.parts:
+            p.prepare(max_positions, device)
+
+    def weights(self):
+        return [w for p in self.parts for w in p.weights()] + [w for w in self.read + self.write if w is not None]
+
+    def kernel_shapes(self, dtype, token_counts):
+        return [shape for p in self.parts for shape in p.kernel_shapes(dtype, token_counts)]
+
+    class _Input:
+        """Where the kernel that last updates the streams leaves a part's input: rows (run dtype), filled or not."""
+        __slots__ = ("rows", "read", "gain", "eps", "filled")
+
+        def __init__(self, rows, read, norm):
+            self.rows, self.read, self.gain, self.eps, self.filled = rows, read, norm.gain, norm.spec.eps, False
+
+    @staticmethod
+    def accepts_emit(emit) -> bool:
+        return isinstance(emit, StreamsBlock._Input)
+
+    def input_emit(self, ctx, n_tokens: int, device):
+        return self._input(ctx, 0, n_tokens)
+
+    def _input(self, ctx, which, n):
+        rows = ctx.scratch(("h_first", "h_ffn")[which], (n, self.size), ctx.dtype)
+        if rows is None:
+            rows = torch.empty((n, self.size), dtype=ctx.dtype, device=ctx.device)
+        return StreamsBlock._Input(rows, self.read[which], (self.mixer_norm, self.ffn_norm)[which])
+
+    def scratch_requests(self, n_tokens, dtype):
+        """h_first lives through the whole layer (this layer's last kernel writes the next layer's into it; the mixer
+        has read it by then); y takes a part's result rows."""
+        from ..engine.workspace import BufferRequest
+        mixer = self.mixer.scratch_requests(n_tokens, dtype)
+        ffn = self.feed_forward.scratch_requests(n_tokens, dtype) if self.feed_forward is not None else []
+        mixer_end = 1 + max([r.last_use for r in mixer] + [0])
+        ffn_start = mixer_end + 2
+        ffn_end = ffn_start + max([r.last_use for r in ffn] + [0])
+        terms = max(int(p.result_terms) if p.overwrites else 1 for p in (self.mixer, self.feed_forward) if p is not None)
+        out = [BufferRequest("h_first", (n_tokens, self.size), dtype, 0, ffn_end + 2),
+               BufferRequest("y_part", (n_tokens * terms, self.size), torch.float32, 0, ffn_end + 1)]
+        out += [r.shifted(1, "mixer.") for r in mixer]
+        if self.feed_forward is not None:
+            out.append(BufferRequest("h_ffn", (n_tokens, self.size), dtype, mixer_end + 1, ffn_end))
+            out += [r.shifted(ffn_start, "ffn.") for r in ffn]
+        return out
+
+    def _result(self, ctx, part, n):
+        """(buffer, terms, fresh): where the part's result goes; zeroed where the part adds instead of writing."""
+        terms = int(part.result_terms) if part.overwrites else 1
+        y = ctx.scratch("y_part", (n * terms, self.size), torch.float32)
+        if y is None:
+            y = torch.empty((n * terms, self.size), dtype=torch.float32, device=ctx.device)
+        if not part.overwrites:
+            ops.fill_(y, 0.0)
+        return y, terms, bool(part.overwrites)
+
+    def _join(self, x, y, terms, which, following):
+        """The new streams; where `following` is given, also the next part's input."""
+        if following is None:
+            ops.streams_update_(x, y, terms, self.write[which])
+            return
+        ops.streams_update_(x, y, terms, self.write[which], following.read, following.gain, following.eps, following.rows)
+        following.filled = True
+
+    def forward(self, x, ctx, entry, cache_entry, normed=None, emit_next=None):
+        """x [T, n, size]. `normed`: this block's first input as the block before left it (a filled _Input), or None.
+        `emit_next`: where this block's last kernel leaves the next block's (an _Input, or None)."""
+        views, n = ctx.workspace, x.shape[0]
+
+        def prefixed(prefix):
+            if views is not None:
+                views.prefix = prefix
+
+        if isinstance(normed, StreamsBlock._Input) and normed.filled:
+            h = normed.rows
+        else:
+            first = self._input(ctx, 0, n)
+            h = ops.streams_read(x, first.read, first.gain, first.eps, ctx.dtype, out=first.rows)
+        y, terms, fresh = self._result(ctx, self.mixer, n)
+        prefixed("mixer.")
+        if fresh:
+            self.mixer.forward(h, ctx, entry, cache_entry, y, fresh=True)
+        else:
+            self.mixer.forward(h, ctx, entry, cache_entry, y)
+        prefixed("")
+        if self.feed_forward is None:
+            self._join(x, y, terms, 0, emit_next)
+            return
+        second = self._input(ctx, 1, n)
+        self._join(x, y, terms, 0, second)
+        y, terms, fresh = self._result(ctx, self.feed_forward, n)
+        prefixed("ffn.")
+        if fresh:
+            self.feed_forward.forward(second.rows, ctx, y, fresh=True)
+        else:
+            self.feed_forward.forward(second.rows, ctx, y)
+        prefixed("")
+        self._join(x, y, terms, 1, emit_next)
+
+
+register_block("streams", StreamsBlock)

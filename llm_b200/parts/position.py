@@ -63,6 +63,33 @@ def table_magnitude(scaling: dict | None) -> float:
     return 1.0
 
 
+def distance_bucket(distance: int, rows: int, far: float) -> int:
+    """The row of a table of `rows` learned biases for a key `distance` positions back: one row a distance below
+    half = rows // 2, from there on a logarithmic scale on which `far` is the first distance beyond the table, whose last
+    row serves everything further back (the buckets of Raffel et al., "Exploring the Limits of Transfer Learning with a
+    Unified Text-to-Text Transformer"). A distance that lies on a bucket's edge belongs to the bucket that starts there,
+    whatever the logarithms' rounding."""
+    half = rows // 2
+    if distance < half:
+        return distance
+    steps = math.log(distance / half) / math.log(far / half) * (rows - half)
+    return min(rows - 1, half + math.floor(steps + 1e-9))
+
+
+def distance_rows(rows: int, far: float) -> list:
+    """The bucket of every distance up to the first one that gets the last row (which serves all further ones)."""
+    out = [0]
+    while out[-1] < rows - 1:
+        out.append(distance_bucket(len(out), rows, far))
+    return out
+
+
+def query_temperature(positions: int, coef: float, every: float) -> torch.Tensor:
+    """float32 [positions]: 1 + coef ln(floor((p + 1) / every) + 1), in float64 and rounded once."""
+    p = torch.arange(positions, dtype=torch.float64)
+    return (1.0 + coef * torch.log(torch.floor((p + 1.0) / every) + 1.0)).to(torch.float32)
+
+
 class Rope(PositionEncoding):
     """Holds a float32 table [positions, n] on the device, n = rotary_dim or head_dim: cos
     of position * inv_freq[p] in columns [0, n/2), sin in [n/2, n). Angles are computed in

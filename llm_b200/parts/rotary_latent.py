@@ -28,7 +28,9 @@ class RotaryLatentMixer(ProjectedMixer):
       projected; a query and key then cost head_dim + rot_dim + value_dim products instead of 2 kv_rank + rot_dim.
 
     Launches: the product [q; dkv], ops.latent_write (norm, rotations, cache write), then the form's own, then
-    the output product."""
+    the output product. Where the queries pass a latent of their own (spec.q_rank), the first product is [dq; dkv],
+    ops.latent_write norms that latent too, and a product with W_uq and ops.latent_rotate make the query heads. Learned
+    sinks (spec.sink) are an argument of the attention kernels."""
     libraries = ("elementwise", "gemm_simt", "gemm_skinny", "gemm_tc", "latent_attention", "latent_prefill_tc",
                  "attention_generic")
 
@@ -36,9 +38,11 @@ class RotaryLatentMixer(ProjectedMixer):
         s = spec
         if min(s.n_heads, s.head_dim, s.rot_dim, s.value_dim, s.kv_rank) < 1:
             raise FormatError("a latent attention with rotated keys needs positive sizes")
+        if s.q_rank < 0:
+            raise FormatError(f"a latent of the queries of {s.q_rank} elements")
         self.spec = spec
         self.position = build_position(spec.position)
-        self.w_uk = self.w_uv = self.w_expand = self.c_gain = None
+        self.w_uk = self.w_uv = self.w_expand = self.c_gain = self.w_uq = self.q_gain = self.sinks = None
 
     @property
     def q_width(self):
@@ -51,7 +55,7 @@ class RotaryLatentMixer(ProjectedMixer):
 
     @property
     def in_width(self):
-        return (self.q_width + self.row + 7) // 8 * 8
+        return ((self.spec.q_rank or self.q_width) + self.row + 7) // 8 * 8
 
     @property
     def out_width(self):
@@ -59,20 +63,32 @@ class RotaryLatentMixer(ProjectedMixer):
 
     def parameters(self):
         s, t = self.spec, self.spec.tensor
-        return {t["q"]: ParamSpec((self.q_width, s.hidden)), t["dkv"]: ParamSpec((self.row, s.hidden)),
-                t["dkv_norm"]: ParamSpec((s.kv_rank,), "gain"),
-                t["uk"]: ParamSpec((s.n_heads * s.head_dim, s.kv_rank)),
-                t["uv"]: ParamSpec((s.n_heads * s.value_dim, s.kv_rank)), t["o"]: ParamSpec((s.hidden, self.out_width))}
+        if s.q_rank:
+            out = {t["dq"]: ParamSpec((s.q_rank, s.hidden)), t["dq_norm"]: ParamSpec((s.q_rank,), "gain"),
+                   t["uq"]: ParamSpec((self.q_width, s.q_rank))}
+        else:
+            out = {t["q"]: ParamSpec((self.q_width, s.hidden))}
+        out.update({t["dkv"]: ParamSpec((self.row, s.hidden)), t["dkv_norm"]: ParamSpec((s.kv_rank,), "gain"),
+                    t["uk"]: ParamSpec((s.n_heads * s.head_dim, s.kv_rank)),
+                    t["uv"]: ParamSpec((s.n_heads * s.value_dim, s.kv_rank)), t["o"]: ParamSpec((s.hidden, self.out_width))})
+        if s.sink:
+            out[t["sink"]] = ParamSpec((s.n_heads,), "vector")
+        return out
 
     def bind(self, tensors, dtype, device):
         s, t = self.spec, self.spec.tensor
-        rows = [to_run_dtype(tensors[t[r]], dtype, device) for r in ("q", "dkv")]
+        rows = [to_run_dtype(tensors[t[r]], dtype, device) for r in ("dq" if s.q_rank else "q", "dkv")]
         pad = self.in_width - sum(r.shape[0] for r in rows)
         if pad:
             rows.append(torch.zeros((pad, s.hidden), dtype=dtype, device=device))
         self.w_in = torch.cat(rows).contiguous()
         self.w_out = to_run_dtype(tensors[t["o"]], dtype, device)
         self.c_gain = to_float32(tensors[t["dkv_norm"]], device)
+        if s.q_rank:
+            self.w_uq = to_run_dtype(tensors[t["uq"]], dtype, device)
+            self.q_gain = to_float32(tensors[t["dq_norm"]], device)
+        if s.sink:
+            self.sinks = to_float32(tensors[t["sink"]], device)
         uk = to_run_dtype(tensors[t["uk"]], dtype, device).view(s.n_heads, s.head_dim, s.kv_rank)
         uv = to_run_dtype(tensors[t["uv"]], dtype, device).view(s.n_heads, s.value_dim, s.kv_rank)
         self.w_uk = uk.transpose(1, 2).contiguous()                     # [H, kv_rank, head_dim]
@@ -89,7 +105,7 @@ class RotaryLatentMixer(ProjectedMixer):
         return KvRequest(1, self.row, 0, values_are_keys=True)
 
     def mix_weights(self):
-        return [self.w_uk, self.w_uv]
+        return [w for w in (self.w_uk, self.w_uv, self.w_uq) if w is not None]
 
     def _shape(self, dtype, decode, fresh=False):
         s = self.spec
@@ -112,7 +128,11 @@ class RotaryLatentMixer(ProjectedMixer):
         return ops.latent_attention_replay_key(step, s.n_heads)
 
     def mix_shapes(self, dtype, token_counts):
-        return [(label, "latent_attention", self._shape(dtype, decode, fresh))
+        s = self.spec
+        heads = [(f"query product, {n} tokens", "linear",
+                  dict(m=n, n=self.q_width, k=s.q_rank, in_dtype=dtype, out_dtype=dtype, lda=s.q_rank, aligned=True))
+                 for n in token_counts] if s.q_rank else []
+        return heads + [(label, "latent_attention", self._shape(dtype, decode, fresh))
                 for label, decode, fresh in (("decode latent attention", True, False),
                                              ("prefill latent attention, first tokens", False, True),
                                              ("prefill latent attention, later tokens", False, False))]
@@ -127,6 +147,9 @@ class RotaryLatentMixer(ProjectedMixer):
         if self._can_expand(dtype):
             out += [BufferRequest("latent_rows", (n_tokens, self.row), dtype, 0, 2),
                     BufferRequest("latent_kv", (n_tokens, s.n_heads * (s.head_dim + s.value_dim)), dtype, 1, 2)]
+        if s.q_rank:
+            out += [BufferRequest("latent_cq", (n_tokens, s.q_rank), dtype, 0, 0),
+                    BufferRequest("latent_heads", (n_tokens, self.q_width), dtype, 0, 2)]
         return out
 
     def mix(self, proj, ctx, entry, cache_entry, out, scratch):
@@ -140,24 +163,38 @@ class RotaryLatentMixer(ProjectedMixer):
             t = scratch(name, shape, dtype)
             return t if t is not None else torch.empty(shape, dtype=dtype, device=proj.device)
 
+        interleaved = self.position.interleaved if self.position is not None else True
         write = dict(write_cache=(entry == cache_entry))
-        common = (proj, s.n_heads, s.head_dim, s.rot_dim, s.kv_rank, self.c_gain, s.eps, angles,
-                  self.position.interleaved if self.position is not None else True, ctx.tok_pos, ctx.tok_seq, table, ring, rows)
+        common = (proj, s.n_heads, s.head_dim, s.rot_dim, s.kv_rank, self.c_gain, s.eps, angles, interleaved, ctx.tok_pos,
+                  ctx.tok_seq, table, ring, rows)
+
+        def down(queries=None, dense=None):
+            """From the first product to the query heads (returned): the cached row, its dense copy, the heads' rotated
+            parts (in place, or in `queries`)."""
+            if not s.q_rank:
+                ops.latent_write(*common, queries=queries, dense=dense, **write)
+                return proj
+            cq = buffer("latent_cq", (n, s.q_rank))
+            ops.latent_write(*common, dense=dense, q_rank=s.q_rank, q_gain=self.q_gain, cq=cq, **write)
+            up = ops.linear(cq, self.w_uq, out=buffer("latent_heads", (n, self.q_width)))
+            ops.latent_rotate(up, s.n_heads, s.head_dim, s.rot_dim, s.kv_rank, angles, interleaved, ctx.tok_pos, queries=queries)
+            return up
+
         if entry == cache_entry and self._expands(ctx, dtype):
             dense = buffer("latent_rows", (n, self.row))
-            ops.latent_write(*common, dense=dense, **write)             # the queries are rotated where they are
+            heads = down(dense=dense)                                   # the queries are rotated where they are
             kv = ops.linear(dense[:, :s.kv_rank], self.w_expand,
                             out=buffer("latent_kv", (n, s.n_heads * (s.head_dim + s.value_dim))))
-            ops.latent_prefill(proj, kv, dense, s.n_heads, s.head_dim, s.rot_dim, s.value_dim, s.kv_rank, s.scale, out,
-                               ctx.cu_seqlens, max(ctx.new_counts), ctx.seq_order)
+            ops.latent_prefill(heads, kv, dense, s.n_heads, s.head_dim, s.rot_dim, s.value_dim, s.kv_rank, s.scale, out,
+                               ctx.cu_seqlens, max(ctx.new_counts), ctx.seq_order, sinks=self.sinks)
             return
         queries = buffer("latent_q", (n, s.n_heads * self.row))
-        ops.latent_write(*common, queries=queries, **write)
-        ops.head_products(proj, s.head_dim + s.rot_dim, self.w_uk, queries, self.row)
+        heads = down(queries=queries)
+        ops.head_products(heads, s.head_dim + s.rot_dim, self.w_uk, queries, self.row)
         latent = buffer("latent_o", (n, s.n_heads * s.kv_rank))
         ops.latent_attention(queries, rows, table, ring, ctx.tok_pos, ctx.tok_seq, s.n_heads, s.kv_rank, s.rot_dim, s.scale,
                              latent, decode=ctx.decode, seq_lens=ctx.seq_lens, max_len=ctx.max_len,
-                             cu_seqlens=ctx.cu_seqlens, max_new=max(ctx.new_counts), seq_order=ctx.seq_order)
+                             cu_seqlens=ctx.cu_seqlens, max_new=max(ctx.new_counts), seq_order=ctx.seq_order, sinks=self.sinks)
         ops.head_products(latent, s.kv_rank, self.w_uv, out, s.value_dim)
 
 

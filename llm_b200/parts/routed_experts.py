@@ -31,16 +31,25 @@ class RoutedExperts(FeedForward):
     `scoring` 'sigmoid' weights the chosen experts by their scores sigmoid(z) as they are; `weight_on_input` puts
     the weight on the expert's input, where the epilogue of the gate and up product applies it to its 32-bit sums
     (W (w h) = w W h) and the down product leaves its rows unweighted. `shared`: a feed-forward of its own for every
-    token, one more row a token behind the experts' (`result_extra`) or added into the residual."""
+    token, one more row a token behind the experts' (`result_extra`) or added into the residual.
+
+    `groups` and `keep_groups` restrict the choice to the best groups of neighbours (the router kernel's work too);
+    `activation` 'clamped' is applied where silu is, in the epilogue of the gate and up product."""
     graph_safe = True
     overwrites = True
 
     def __init__(self, spec):
         s = spec
-        if s.activation != "silu":
+        if s.activation not in ("silu", "clamped") or (s.activation == "clamped" and not s.limit >= 0.0):
             raise Unsupported(f"activation '{s.activation}' in routed experts")
         if min(s.hidden, s.intermediate, s.n_experts, s.top) < 1 or s.pass_through < 0 or s.top > s.n_experts + s.pass_through:
             raise FormatError(f"{s.top} of {s.n_experts + max(s.pass_through, 0)} experts cannot be chosen")
+        if s.groups < 1 or not 1 <= s.keep_groups <= s.groups or (s.n_experts + s.pass_through) % s.groups \
+                or s.top > s.keep_groups * ((s.n_experts + s.pass_through) // s.groups):
+            raise FormatError(f"{s.top} of {s.n_experts + s.pass_through} experts cannot be chosen from {s.keep_groups} of "
+                              f"{s.groups} equal groups")
+        if s.groups > 1 and (s.scoring != "all" or s.correction):
+            raise Unsupported("groups of experts need scores over all experts and no correction of the choice")
         if s.scoring not in ops.ROUTER_SCORING:
             raise Unsupported(f"scoring '{s.scoring}' in routed experts (built: {', '.join(ops.ROUTER_SCORING)})")
         if s.correction and s.scoring != "all":
@@ -138,7 +147,9 @@ class RoutedExperts(FeedForward):
         gathered = buffer("expert_in", (a, s.hidden), h.dtype) if wide else None
         ops.routed_experts(h, self.router, self.router_bias, self.w_up, self.w_down, s.top, ids, weights, order, plan,
                            act, rows, gathered, scoring=ops.ROUTER_SCORING.index(s.scoring), correction=self.correction,
-                           pass_through=s.pass_through, weight_scale=s.out_scale, weight_on_input=s.weight_on_input)
+                           pass_through=s.pass_through, weight_scale=s.out_scale, weight_on_input=s.weight_on_input,
+                           groups=s.groups, keep=s.keep_groups, limit=s.limit if s.activation == "clamped" else -1.0,
+                           alpha=s.alpha)
         if not fresh:
             ops.add_terms_(residual, rows, s.top)
         if self.shared is None:

@@ -135,7 +135,9 @@ class RotaryLatentSpec:
     """Attention over one cached latent row per position with a rotated key part that all heads share. A query head
     is [head_dim unrotated | rot_dim rotated] elements of W_q h; W_dkv h is [kv_rank | rot_dim]: the first part,
     RMS-normed (eps), is the latent c, the second the shared rotated key part. Head a's key is [W_uk,a c | shared part],
-    its value W_uv,a c. Only c and the rotated part are cached."""
+    its value W_uv,a c. Only c and the rotated part are cached. With `q_rank` > 0 the queries pass a latent of their own:
+    W_q is W_uq norm(W_dq h) (roles `dq`, `dq_norm`, `uq` instead of `q`). `sink`: one more term e^sink[head] in a head's
+    softmax denominator (role `sink`), without key or value, not scaled."""
     hidden: int
     n_heads: int
     head_dim: int                    # unrotated query / key elements of a head
@@ -145,8 +147,10 @@ class RotaryLatentSpec:
     scale: float                     # multiplies q.k
     eps: float                       # of the latent's norm
     position: Optional[PositionSpec] # of the rotated part (head_dim == rot_dim there)
-    names: tuple                     # sorted (role, tensor name): q, dkv, dkv_norm, uk, uv, o
+    names: tuple                     # sorted (role, tensor name): q, dkv, dkv_norm, uk, uv, o (or dq, dq_norm, uq; + sink)
     kind: str = "rotary_latent_attention"
+    q_rank: int = 0                  # size of the queries' latent (0: none)
+    sink: bool = False
 
     @property
     def tensor(self):
@@ -218,7 +222,13 @@ class GatedAttentionSpec:
     `value_mix` (a name shared by the layers whose values are blended: in every such layer but the one with
     `value_mix_first`, v <- (1 - w) v + w v_first with w one stored number (role `value_mix`) and v_first the
     values that the first such layer computed for the same token; the blended values are what is cached);
-    `out_scale` multiplies the mixer's result."""
+    `out_scale` multiplies the mixer's result; `bias` (the projections of queries, keys and values have one each, roles
+    `q_bias`, `k_bias`, `v_bias`); `unit_norm` (queries and keys are divided by their root mean square per head, without a
+    weight, eps `norm_eps`); `q_temp` = (coef, every): queries at position p are multiplied by
+    1 + coef ln(floor((p + 1) / every) + 1), behind the norm; `distance_bias` = far: a learned number per head and
+    distance bucket (role `rel`, [rows, n_heads]; the tensor decides how many rows) is added to the scaled score, bucket(n) = n for n < rows / 2, else
+    min(rows - 1, rows / 2 + floor(ln(n / (rows / 2)) / ln(far / (rows / 2)) * (rows - rows / 2))); `shared_kv` (the mixer has
+    no projections of keys and values: it reads those of the run that its schedule entry names)."""
     hidden: int
     n_heads: int
     n_kv_heads: int
@@ -240,6 +250,11 @@ class GatedAttentionSpec:
     value_mix_first: bool = False
     out_scale: float = 1.0
     sink: bool = False
+    bias: bool = False
+    unit_norm: bool = False
+    q_temp: Optional[tuple] = None
+    distance_bias: Optional[float] = None
+    shared_kv: bool = False
 
     @property
     def tensor(self):
@@ -285,6 +300,26 @@ class ForgetRecurrenceSpec:
     eps: float
     names: tuple                     # sorted (role, tensor name): q, f, f_bias, lower, v, norm, o
     kind: str = "forget_recurrence"
+
+    @property
+    def tensor(self):
+        return dict(self.names)
+
+
+@dataclass(frozen=True)
+class DecayRecurrenceSpec:
+    """Linear attention with one fixed decay per head (Qin et al., "Lightning Attention-2"; Sun et al., "Retentive
+    Network"): q = silu(W_q h), k = silu(W_k h) (n_heads heads of head_dim), v = silu(W_v h) (n_heads heads of value_dim);
+    per head S_t = decay S_(t-1) + k_t v_t^T, o_t = S_t^T q_t; the concatenated heads are divided by their root mean square
+    (eps), multiplied by a weight per element and by sigmoid(W_g h), then W_o."""
+    hidden: int
+    n_heads: int
+    head_dim: int
+    value_dim: int
+    decay: tuple                     # per head
+    eps: float
+    names: tuple                     # sorted (role, tensor name): q, k, v, gate, norm, o
+    kind: str = "decay_recurrence"
 
     @property
     def tensor(self):
@@ -366,7 +401,11 @@ class RoutedExpertsSpec:
 
     `scoring` 'sigmoid': scores s = sigmoid(z), the `top` largest are chosen, and the weights are the chosen scores
     as they are. `weight_on_input`: the weight multiplies the expert's input instead of its result, expert(w h).
-    `shared` (a GatedMlpSpec): one more feed-forward that every token passes, added to the result."""
+    `shared` (a GatedMlpSpec): one more feed-forward that every token passes, added to the result.
+
+    `groups` > 1 (scoring 'all'): the outputs form that many equal groups of neighbours; a group's score is its largest,
+    and only outputs of the `keep_groups` best groups can be chosen. `activation` 'clamped': g <- min(W_gate h, limit),
+    u <- clamp(W_up h, -limit, limit), down(g sigmoid(alpha g) (u + 1)) with `limit` and `alpha`."""
     hidden: int
     intermediate: int
     n_experts: int
@@ -382,6 +421,10 @@ class RoutedExpertsSpec:
     out_scale: float = 1.0
     weight_on_input: bool = False
     shared: Optional[GatedMlpSpec] = None
+    groups: int = 1
+    keep_groups: int = 1
+    limit: float = 0.0               # of the clamped activation
+    alpha: float = 1.0
 
     @property
     def tensor(self):
@@ -418,6 +461,22 @@ class OutputNormBlockSpec:
     mixer_conv: Optional[str] = None
     ffn_conv: Optional[str] = None
     kind: str = "output_norm"
+
+
+@dataclass(frozen=True)
+class StreamsBlockSpec:
+    """A residual of several streams (Zhu et al., "Hyper-Connections"). For each part: u = sum_s in[s] x_s;
+    y = part(norm(u)); then, all streams at once from the old ones, x_t <- sum_s mix[s, t] x_s + out[t] y.
+    `mixer_streams`, `ffn_streams`: the names of the tensors (in [n], mix [n, n], out [n]). `feed_forward` (with its norm
+    and streams) may be None."""
+    n_streams: int
+    mixer_norm: object
+    mixer: object
+    mixer_streams: tuple
+    ffn_norm: object
+    feed_forward: object
+    ffn_streams: Optional[tuple]
+    kind: str = "streams"
 
 
 @dataclass(frozen=True)
@@ -468,6 +527,8 @@ class ModelSpec:
     embedding_scale: float = 1.0     # multiplies the embedded tokens
     logit_scale: float = 1.0         # multiplies the logits
     logit_softcap: float = 0.0       # c > 0: logits <- c * tanh(logits / c), after the scale
+    streams: int = 0                 # n > 0: the residual is n streams, all equal to the embedding output at first and summed
+                                     # at the end; every block is then one that works on n streams
 
 
 def names(**roles) -> tuple:

@@ -15,13 +15,19 @@ class ParamSpec:
 
     role: 'matrix' (an operand of a matrix product, held in the run dtype),
     'gain' (a norm's weight; 'gain_offset' where it is stored as an offset from 1), 'bias', 'vector',
-    'gate_scalar' (one learned number, shape ())
+    'gate_scalar' (one learned number, shape ()), 'streams' (the weights of a residual's streams)
     and 'taps' (small 32-bit operands: a gate's vector, a short convolution's taps), 'table'
     (integers, held as int32).
-    Gains and biases are held in 32-bit whatever the file stores.
+    Gains and biases are held in 32-bit whatever the file stores. `free` lists the axes whose size the
+    checkpoint decides (`shape` then holds the size of a random model's tensor there).
     """
     shape: tuple
     role: str = "matrix"
+    free: tuple = ()
+
+    def fits(self, shape) -> bool:
+        return len(shape) == len(self.shape) and all(
+            i in self.free or a == b for i, (a, b) in enumerate(zip(shape, self.shape)))
 
 
 def storage_dtype(file_dtype: torch.dtype) -> torch.dtype:
@@ -40,7 +46,7 @@ def check_names(expected: dict, found: dict, where: str = "") -> None:
     missing = [n for n in expected if n not in found]
     unexpected = [n for n in found if n not in expected]
     mismatched = [(n, list(found[n]), list(expected[n].shape))
-                  for n in expected if n in found and tuple(found[n]) != tuple(expected[n].shape)]
+                  for n in expected if n in found and not expected[n].fits(tuple(found[n]))]
     if missing or unexpected or mismatched:
         raise WeightError(missing, unexpected, mismatched, where)
 

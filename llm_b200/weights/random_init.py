@@ -46,7 +46,7 @@ def random_tensors(expected: dict, seed: int, dtype=torch.bfloat16, std: float =
     device that makes it: a model made on the GPU and one written to a folder on the CPU
     from the same seed are the same model. Matrices and biases are N(0, std); gains are
     1 + N(0, gain_noise) (N(0, gain_noise) where the gain is stored as an offset from 1); the taps of a
-    short convolution are N(0, 1 / taps). Values are drawn in 32-bit and rounded once to `dtype`."""
+    short convolution are N(0, 1 / taps); the weights of a residual's n streams are 1 / n + N(0, gain_noise). Values are drawn in 32-bit and rounded once to `dtype`."""
     out = {}
     for name in sorted(expected):
         spec = expected[name]
@@ -60,6 +60,8 @@ def random_tensors(expected: dict, seed: int, dtype=torch.bfloat16, std: float =
             normal_(tensor, tensor_key(seed, name), 0.0, gain_noise)
         elif spec.role == "gate_scalar":                     # one learned number of the order of one half
             normal_(tensor, tensor_key(seed, name), 0.5, gain_noise)
+        elif spec.role == "streams":                         # the weights of a residual's streams: around 1 / their number
+            normal_(tensor, tensor_key(seed, name), 1.0 / max(spec.shape[-1], 1), gain_noise)
         elif spec.role == "taps":                            # a short convolution: taps of the order of 1 / taps
             normal_(tensor, tensor_key(seed, name), 0.0, 1.0 / max(spec.shape[-1], 1))
         else:

@@ -134,10 +134,11 @@ def rope_cache_write(qkv, rope_table, tok_pos, tok_seq, block_table, ring_pages,
 def attention(qkv, k_cache, v_cache, block_table, ring_pages, tok_pos, tok_seq, n_heads,
               n_kv_heads, head_dim, scale, window=0, out=None, decode=False, seq_lens=None,
               max_len=0, cu_seqlens=None, max_new=0, seq_order=None, sinks=None, gate=None, out_scale=1.0,
-              softcap=0.0, value_dim=None):
+              softcap=0.0, value_dim=None, bias=None):
     """`sinks` (float32 [heads]): e^sink is one more term of a head's softmax denominator. `gate`
     ([T, heads]): head a of token t is multiplied by sigmoid(gate[t, a]). `out_scale` multiplies all.
-    `softcap` c > 0: score <- c tanh(score / c). `value_dim`: the size of a value (default head_dim)."""
+    `softcap` c > 0: score <- c tanh(score / c). `value_dim`: the size of a value (default head_dim).
+    `bias` ([heads, span]): bias[a, distance] joins the scaled score, the last column at every further distance."""
     n = qkv.shape[0]
     value_dim = value_dim or head_dim
     result = torch.zeros((n, n_heads * value_dim), dtype=torch.float32, device=qkv.device)
@@ -155,6 +156,8 @@ def attention(qkv, k_cache, v_cache, block_table, ring_pages, tok_pos, tok_seq, 
             scores = (keys[:, h // group, :] @ q[h]) * scale
             if softcap > 0.0:
                 scores = softcap * torch.tanh(scores / softcap)
+            if bias is not None:
+                scores = scores + bias[h, torch.clamp(pos - js, max=bias.shape[1] - 1)]
             if sinks is None:
                 p = torch.softmax(scores, dim=0)
             else:
@@ -186,13 +189,14 @@ def tanh_norm(x, alpha, gain, bias, out_dtype, rows=None, out=None, second=None)
 
 def norm_rope_cache_write(u, q_width, k_width, v_width, q_gain, k_gain, eps, rope_table, rot_unit, interleaved,
                           tok_pos, tok_seq, q_out, block_table, ring_pages, k_cache, v_cache, write_cache=True,
-                          value_source=None, norm_unit=0, mix_cache=None, mix_table=None, mix_ring=0, mix=0.0):
+                          value_source=None, norm_unit=0, mix_cache=None, mix_table=None, mix_ring=0, mix=0.0, q_scale=None):
     """The first q_width columns of u are the queries, the next k_width the keys, the next v_width
     the values (or, with value_source, the v_width columns from there on: q_width makes the values
     the keys as projected). With a gain, queries (keys) are divided by the root mean square of the
     whole segment (or, with norm_unit, of every unit of that many columns, all units sharing a gain of
     that size) and multiplied by the gain; then every unit of rot_unit columns of both rotates. With
-    mix_cache the values become (1 - mix) v + mix * (what that cache holds at the token's place)."""
+    mix_cache the values become (1 - mix) v + mix * (what that cache holds at the token's place). With q_scale the
+    queries of position p are multiplied by q_scale[p]."""
     n = u.shape[0]
     if n == 0:
         return q_out
@@ -210,7 +214,8 @@ def norm_rope_cache_write(u, q_width, k_width, v_width, q_gain, k_gain, eps, rop
             x = _rotate(x.reshape(n, -1, rot_unit), rope_table[pos, :half], rope_table[pos, half:], interleaved)
         return x.reshape(n, width)
 
-    q_out.copy_(segment(0, q_width, q_gain).to(q_out.dtype))
+    warm = 1.0 if q_scale is None else q_scale[pos][:, None]
+    q_out.copy_((segment(0, q_width, q_gain) * warm).to(q_out.dtype))
     if write_cache:
         pages = block_table.long()[tok_seq.long(), (pos // PAGE) % ring_pages]
         rows = pos % PAGE
@@ -385,12 +390,14 @@ def routed_experts_wide(n_tokens, top, n_experts, hidden, intermediate, dtype):
 
 
 def routed_experts(h, router, router_bias, w_up, w_down, top, ids, weights, order, plan, act, y, gathered=None,
-                   scoring=0, correction=None, pass_through=0, weight_scale=1.0, weight_on_input=False):
+                   scoring=0, correction=None, pass_through=0, weight_scale=1.0, weight_on_input=False, groups=1, keep=1,
+                   limit=-1.0, alpha=1.0):
     """Token by token: 32-bit router logits, the `top` largest, the softmax over them, and one row
     weight * expert(h) per choice, in the order of choice (largest logit first). scoring 1: the scores are the
     softmax over all outputs, the choice is by score + correction, the weights are the chosen scores over
     their sum (+ 1e-20). The router's last `pass_through` outputs are experts whose result is h. scoring 2: the weights are the
-    sigmoids of the chosen logits. weight_on_input: expert(weight h) in place of weight * expert(h)."""
+    sigmoids of the chosen logits. weight_on_input: expert(weight h) in place of weight * expert(h). groups: only outputs of
+    the `keep` groups with the largest single score are chosen. limit >= 0: the clamped activation."""
     n, hidden = h.shape
     F = w_up.shape[1] // 2
     x = h.to(torch.float32)
@@ -402,6 +409,11 @@ def routed_experts(h, router, router_bias, w_up, w_down, top, ids, weights, orde
         if scoring == 1:
             scores = torch.softmax(logits[t], 0)
             choice = scores + correction if correction is not None else scores
+            if groups > 1:
+                peaks = torch.sort(scores.view(groups, -1).max(-1).values, descending=True, stable=True).indices
+                choice = choice.view(groups, -1).clone()
+                choice[peaks[keep:]] = -1.0
+                choice = choice.view(-1)
             chosen = torch.sort(choice, descending=True, stable=True).indices[:top]
             share = scores[chosen] / (scores[chosen].sum() + 1e-20) * weight_scale
         elif scoring == 2:
@@ -421,7 +433,12 @@ def routed_experts(h, router, router_bias, w_up, w_down, top, ids, weights, orde
             if weight_on_input:
                 gate_up = gate_up * share[k]
             g, u = gate_up[:F], gate_up[F:]
-            a = (g / (1.0 + torch.exp(-g)) * u).to(h.dtype).to(torch.float32)
+            if limit >= 0.0:
+                g, u = torch.clamp(g, max=limit), torch.clamp(u, -limit, limit)
+                a = g / (1.0 + torch.exp(-alpha * g)) * (u + 1.0)
+            else:
+                a = g / (1.0 + torch.exp(-g)) * u
+            a = a.to(h.dtype).to(torch.float32)
             y[t * top + k] = (1.0 if weight_on_input else share[k]) * (a @ w_down[e].to(torch.float32).T)
     return y
 
@@ -547,27 +564,41 @@ def forget_recurrence(proj, f_bias, lower, state, cu_seqlens, slot_ids, norm_wei
 
 
 def latent_write(u, n_heads, dim, rot, rank, gain, eps, rope_table, interleaved, tok_pos, tok_seq, block_table, ring_pages,
-                 cache, queries=None, dense=None, write_cache=True):
-    n, qw = u.shape[0], n_heads * (dim + rot)
+                 cache, queries=None, dense=None, write_cache=True, q_rank=0, q_gain=None, cq=None):
+    n, qw = u.shape[0], q_rank or n_heads * (dim + rot)
     for t in range(n):
         pos, b = int(tok_pos[t]), int(tok_seq[t])
         row = u[t, qw:qw + rank + rot].to(torch.float32).clone()
+        if q_rank:
+            x = u[t, :q_rank].to(torch.float32)
+            cq[t] = (x / torch.sqrt((x * x).mean() + eps) * q_gain).to(cq.dtype)
         c = row[:rank]
         row[:rank] = c / torch.sqrt((c * c).mean() + eps) * gain
-        q = u[t, :qw].to(torch.float32).view(n_heads, dim + rot).clone()
         if rope_table is not None:
             n_rot = rope_table.shape[1]
             cos, sin = rope_table[pos:pos + 1, :n_rot // 2], rope_table[pos:pos + 1, n_rot // 2:]
             row[rank:rank + n_rot] = _rotate(row[None, None, rank:rank + n_rot], cos, sin, interleaved)[0, 0]
-            q[:, dim:dim + n_rot] = _rotate(q[None, :, dim:dim + n_rot], cos, sin, interleaved)[0]
         if write_cache:
             cache[int(block_table[b, (pos // PAGE) % ring_pages]), 0, pos % PAGE] = row.to(cache.dtype)
         if dense is not None:
             dense[t] = row.to(dense.dtype)
+    if not q_rank:
+        latent_rotate(u[:, :qw], n_heads, dim, rot, rank, rope_table, interleaved, tok_pos, queries)
+
+
+def latent_rotate(heads, n_heads, dim, rot, rank, rope_table, interleaved, tok_pos, queries=None):
+    n = heads.shape[0]
+    for t in range(n):
+        pos = int(tok_pos[t])
+        q = heads[t].to(torch.float32).view(n_heads, dim + rot).clone()
+        if rope_table is not None:
+            n_rot = rope_table.shape[1]
+            cos, sin = rope_table[pos:pos + 1, :n_rot // 2], rope_table[pos:pos + 1, n_rot // 2:]
+            q[:, dim:dim + n_rot] = _rotate(q[None, :, dim:dim + n_rot], cos, sin, interleaved)[0]
         if queries is not None:
             queries.view(n, n_heads, rank + rot)[t, :, rank:] = q[:, dim:].to(queries.dtype)
         else:
-            u[t, :qw] = q.reshape(-1).to(u.dtype)
+            heads[t] = q.reshape(-1).to(heads.dtype)
 
 
 def head_products(x, x_head, w, out, out_head):
@@ -582,20 +613,31 @@ def latent_attention_replay_key(step, n_heads):
     return ()
 
 
+def _sink_softmax(scores, sinks):
+    """Softmax over the last axis with one more term e^sinks[h] in row h's denominator (sinks None: without)."""
+    if sinks is None:
+        return torch.softmax(scores, dim=-1)
+    s = sinks.to(torch.float32).reshape((-1,) + (1,) * (scores.dim() - 1))
+    top = torch.maximum(scores.max(-1, keepdim=True).values, s)
+    e = torch.exp(scores - top)
+    return e / (e.sum(-1, keepdim=True) + torch.exp(s - top))
+
+
 def latent_attention(queries, cache, block_table, ring_pages, tok_pos, tok_seq, n_heads, rank, rot, scale, out, decode=False,
-                     seq_lens=None, max_len=0, cu_seqlens=None, max_new=0, seq_order=None):
+                     seq_lens=None, max_len=0, cu_seqlens=None, max_new=0, seq_order=None, sinks=None):
     n, width = queries.shape[0], rank + rot
     for t in range(n):
         pos, b = int(tok_pos[t]), int(tok_seq[t])
         js = torch.arange(pos + 1, device=queries.device)
         rows = cache[block_table.long()[b, (js // PAGE) % ring_pages], 0, js % PAGE].to(torch.float32)
         q = queries[t].to(torch.float32).view(n_heads, width)
-        p = torch.softmax((q @ rows.T) * scale, dim=-1)
+        p = _sink_softmax((q @ rows.T) * scale, sinks)
         out[t] = (p @ rows[:, :rank]).reshape(-1).to(out.dtype)
     return out
 
 
-def latent_prefill(proj, kv, dense, n_heads, dim, rot, vdim, rank, scale, out, cu_seqlens, max_new, seq_order=None):
+def latent_prefill(proj, kv, dense, n_heads, dim, rot, vdim, rank, scale, out, cu_seqlens, max_new, seq_order=None,
+                   sinks=None):
     """Causal attention of packed prompts that start at their first token, keys and values of every head formed."""
     for b in range(cu_seqlens.numel() - 1):
         lo, hi = int(cu_seqlens[b]), int(cu_seqlens[b + 1])
@@ -605,9 +647,56 @@ def latent_prefill(proj, kv, dense, n_heads, dim, rot, vdim, rank, scale, out, c
         mask = torch.ones((hi - lo, hi - lo), dtype=torch.bool, device=proj.device).tril()
         for h in range(n_heads):
             s = (q[:, h, :dim] @ heads[:, h, :dim].T + q[:, h, dim:] @ shared.T) * scale
-            p = torch.softmax(s.masked_fill(~mask, float("-inf")), dim=-1)
+            p = _sink_softmax(s.masked_fill(~mask, float("-inf"))[None], None if sinks is None else sinks[h:h + 1])[0]
             out[lo:hi, h * vdim:(h + 1) * vdim] = (p @ heads[:, h, dim:]).to(out.dtype)
     return out
+
+
+def decay_recurrence_work_width(n_heads, dim, vdim):
+    return (2 * n_heads * dim + n_heads * vdim + 3) // 4 * 4
+
+
+def decay_recurrence(proj, decays, state, cu_seqlens, slot_ids, norm_weight, eps, work, o, mixed, n_heads, dim, vdim,
+                     single_tokens=False):
+    """Token by token and head by head; S lies in the state as [H, V, D]."""
+    H, D, V = n_heads, dim, vdim
+    u = proj.to(torch.float32)
+    n, keys, values = u.shape[0], H * D, H * V
+    x = u[:, :2 * keys + values]
+    x = x / (1.0 + torch.exp(-x))
+    q, k, v = x[:, :keys].view(n, H, D), x[:, keys:2 * keys].view(n, H, D), x[:, 2 * keys:].view(n, H, V)
+    gate = torch.sigmoid(u[:, 2 * keys + values:2 * (keys + values)])
+    for b in range(cu_seqlens.numel() - 1):
+        slot = int(slot_ids[b])
+        S = state[slot, :H * D * V].view(H, V, D).clone()
+        for t in range(int(cu_seqlens[b]), int(cu_seqlens[b + 1])):
+            S = decays[:, None, None] * S + v[t][:, :, None] * k[t][:, None, :]
+            r = (S * q[t][:, None, :]).sum(-1).reshape(-1)
+            mixed[t] = (r / torch.sqrt((r * r).mean() + eps) * norm_weight * gate[t]).to(mixed.dtype)
+        state[slot, :H * D * V] = S.reshape(-1)
+    return mixed
+
+
+def streams_embed(tokens, table, n_streams, scale=1.0):
+    return (table[tokens.long()].to(torch.float32) * scale)[:, None, :].repeat(1, n_streams, 1)
+
+
+def streams_read(X, read, gain, eps, out_dtype, rows=None, out=None):
+    """The weighted (or plain) sum over the streams, over its root mean square, times the gain."""
+    if rows is not None:
+        X = X[rows.long()]
+    u = X.sum(1) if read is None else (X * read[None, :, None]).sum(1)
+    y = (u / torch.sqrt((u * u).mean(-1, keepdim=True) + eps) * gain).to(out_dtype)
+    return y if out is None else out.copy_(y)
+
+
+def streams_update_(X, y, terms, write, read=None, gain=None, eps=0.0, out=None):
+    """X'_t = sum_s mix[s, t] X_s + spread[t] * (a token's summed rows); write = [spread | mix]."""
+    n, S, hidden = X.shape
+    spread, mix = write[:S], write[S:].view(S, S)
+    total = y.view(n, terms, hidden).sum(1)
+    X.copy_(torch.einsum("st,nsh->nth", mix, X) + spread[None, :, None] * total[:, None, :])
+    return None if out is None else streams_read(X, read, gain, eps, out.dtype, out=out)
 
 
 def softcap_(x, cap):
@@ -823,7 +912,9 @@ OPS = {"embed": embed, "scale_": scale_, "cast_sumsq": cast_sumsq, "rmsnorm": rm
        "output_norm_add_": output_norm_add_, "forget_recurrence": forget_recurrence,
        "forget_recurrence_work_width": forget_recurrence_work_width, "latent_write": latent_write,
        "head_products": head_products, "latent_attention": latent_attention, "latent_prefill": latent_prefill,
-       "latent_attention_replay_key": latent_attention_replay_key}
+       "latent_attention_replay_key": latent_attention_replay_key, "latent_rotate": latent_rotate,
+       "decay_recurrence": decay_recurrence, "decay_recurrence_work_width": decay_recurrence_work_width,
+       "streams_embed": streams_embed, "streams_read": streams_read, "streams_update_": streams_update_}
 
 
 def install(monkeypatch):
