@@ -1,7 +1,7 @@
 """Decode and prefill throughput of the library on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--layers L] [--impl reference]
-    python bench.py --workload llama-2-7b | llama-3.2-1b | 8b-decode512 | guberax | mefolorn | zogapel | zemozen | duvozen
+    python bench.py --workload llama-2-7b | llama-3.2-1b | 8b-decode512 | guberax | mefolorn | zogapel | zemozen | duvozen | renapel
 
 The default run has the layer sizes of a Llama-3.1-8B (32 layers, hidden 4096,
 32 heads over 8 kv heads of 128, feed-forward 14336, vocabulary 128256, llama3
@@ -14,7 +14,7 @@ tokens and 128 new tokens each, a Llama-3.2-1B shape with 64 prompts of 1 to 8,1
 256 new tokens at temperature 0.7 (both through `LLM.generate`, host ids in and out), and the
 Llama-3.1-8B shape decoding 256 tokens after prompts of 512 at batch 1, 8 and 64; `guberax`
 times the Guberax architecture beside Llama at equal layer sizes, `mefolorn` the Mefolorn
-architecture beside both, `zogapel` the Zogapel architecture beside Mefolorn and Llama, `zemozen` the Zemozen architecture beside Zogapel and Llama, `duvozen` the Duvozen architecture beside Zemozen, Mefolorn and Llama. The test names follow the `pp`/`tg`
+architecture beside both, `zogapel` the Zogapel architecture beside Mefolorn and Llama, `zemozen` the Zemozen architecture beside Zogapel and Llama, `duvozen` the Duvozen architecture beside Zemozen, Mefolorn and Llama, `renapel` the Renapel architecture beside Duvozen, Zemozen and Llama. The test names follow the `pp`/`tg`
 split of MythEclipse/llm's bench (apps/cli/src/bench.rs:10-12): prefill alone,
 and decoding alone on a cache that is already filled.
 """
@@ -508,10 +508,29 @@ def workload_duvozen(args):
                    "latent rows 256 + 32, recurrence 32 heads of 64 x 64; vocabulary 128256")
 
 
+def workload_renapel(args):
+    """Renapel beside Duvozen (the library's closest model: latent attention, attention with sinks, a recurrence with a
+    matrix state, routed experts), Zemozen (routed experts in every layer) and Llama at equal layer sizes (the Llama-3.1-8B
+    and Llama-3.2-1B shapes), `--layers` layers of each (at most 8) plus the head. Renapel's layers go linear attention,
+    attention, latent attention, attention over the keys of the second, with four streams and experts in every layer."""
+    from llm_b200.shapes import shape
+    layers = min(args.layers, 8)
+    sizes = [(size, [("llama", shape(llama, layers)), ("zemozen_window2048", shape(zemozen, layers, 2048)),
+                     ("duvozen", shape(duvozen, layers)), ("renapel", shape(renapel, layers))])
+             for size, llama, zemozen, duvozen, renapel in (
+                 ("1b", "llama-3.2-1b", "zemozen-1b", "duvozen-1b", "renapel-1b"),
+                 ("8b", "llama-3.1-8b", "zemozen-8b", "duvozen-8b", "renapel-8b"))]
+    return _beside(args, sizes, "prefill and decode tokens/s, Renapel beside Duvozen, Zemozen and Llama at equal layer sizes, bf16",
+                   "renapel-8b",
+                   "8b: width 4096 in 4 streams, 32/8 heads of 128, 8 of 32 experts of 1792, latent rows 512 + 64, latent of the "
+                   "queries 1536, linear attention 32 heads of 128 x 128; 1b: width 2048, 32/8 heads of 64, experts of 1024, "
+                   "latent rows 256 + 32, latent of the queries 768, linear attention 32 heads of 64 x 64; vocabulary 128256")
+
+
 WORKLOADS = {"llama-2-7b": workload_llama_2_7b, "llama-3.2-1b": workload_llama_3_2_1b,
              "8b-decode512": workload_8b_decode512, "guberax": workload_guberax, "mefolorn": workload_mefolorn,
              "zogapel": workload_zogapel, "zemozen": workload_zemozen,
-             "duvozen": workload_duvozen}
+             "duvozen": workload_duvozen, "renapel": workload_renapel}
 
 
 

@@ -142,6 +142,33 @@ SHAPES["duvozen-8b"] = _duvozen(4096, 32, 8, 128, 14336, 128256, 32, (64, 512), 
 SHAPES["duvozen-1b"] = _duvozen(2048, 32, 8, 64, 8192, 128256, 16, (32, 256), 32, 8)
 
 
+def _renapel(width, heads, kv_heads, dim, ff, vocab, layers, latent, experts, top):
+    """A Renapel configuration whose layers match a Llama shape in size (width, heads, head size, vocabulary): four streams
+    and a pattern of four layers, linear attention (states of head size x head size), attention with a bias by distance (up to
+    128 back), latent attention (the Llama shape's heads as the unrotated part; `latent` = rotated part, cached latent and
+    the queries' latent), and attention over the keys and values of the one before. Every layer has routed experts in
+    4 groups of which 2 stay, whose `top` chosen ones together are as wide as the Llama shape's feed-forward."""
+    rot_dim, kv_rank, q_rank = latent
+    base = {"heads": heads, "dim": dim, "vdim": dim}
+    lightning = {**base, "decay": [1.0 - 2.0 ** (-1.0 - 7.0 * h / heads) for h in range(heads)]}
+    attention = {**base, "kv_heads": kv_heads, "scale": dim ** -0.5, "bias_max": 128, "q_temp": {"coef": 0.2, "every": 1024}}
+    latent_mixer = {**base, "rot_dim": rot_dim, "kv_rank": kv_rank, "q_rank": q_rank, "scale": (dim + rot_dim) ** -0.5,
+                    "rot": {"base": 500000.0, "dims": rot_dim}}
+    routed = {"kind": "moe", "expert": {"ff": ff // top, "limit": 7.0},
+              "router": {"experts": experts, "top": top, "scale": 2.5, "groups": {"count": 4, "keep": 2}}}
+    kinds = [("lightning", lightning), ("attention", attention), ("latent_attention", latent_mixer), ("attention", attention)]
+    out = []
+    for i in range(layers):
+        kind, mixer = kinds[i % 4]
+        out.append({"type": kind, "mixer": {**mixer, "kv_from": i - 2} if i % 4 == 3 else mixer, "mlp": routed})
+    return {"architecture": "Renapel", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "streams": 4, "layers": out}
+
+
+# the layer sizes of llama-3.1-8b and llama-3.2-1b; 8 of 32 experts; cached rows of 512 + 64 and 256 + 32
+SHAPES["renapel-8b"] = _renapel(4096, 32, 8, 128, 14336, 128256, 32, (64, 512, 1536), 32, 8)
+SHAPES["renapel-1b"] = _renapel(2048, 32, 8, 64, 8192, 128256, 16, (32, 256, 768), 32, 8)
+
+
 def shape(name: str, layers: int | None = None, window: int | None = None) -> dict:
     """A copy of the named shape's config.json, optionally with fewer layers (and, for a shape
     with windowed attention, another window)."""

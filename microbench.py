@@ -14,6 +14,9 @@
     python microbench.py latent_prefill | latent_write | head_products --batch 1 --tokens 2048
     python microbench.py output_norm --m 8 --tokens 1 --top 8        # --tokens 1: with the next part's input
     python microbench.py input_conv --m 2048
+    python microbench.py decay_recurrence --batch 64 --tokens 1
+    python microbench.py streams --m 2048 --streams 4 --top 8
+    python microbench.py attention_decode | attention_prefill --bias 128     # a bias by distance, up to 128 back
     LLMB_NVCC_FLAGS=-DLLMB_TRACE python microbench.py linear --m 8 --n 6144 --k 4096 --timeline
     LLMB_NVCC_FLAGS=-DLLMB_TRACE python microbench.py attention_prefill --tokens 2048 --timeline
 
@@ -159,7 +162,7 @@ def phase_sums(fn, label: str) -> int:
 
 def main(argv=None) -> int:
     p = argparse.ArgumentParser(description=__doc__.split("\n")[0])
-    p.add_argument("op", choices=["forget_recurrence", "latent_attention", "latent_prefill", "head_products", "latent_write",
+    p.add_argument("op", choices=["decay_recurrence", "streams", "forget_recurrence", "latent_attention", "latent_prefill", "head_products", "latent_write",
                                   "output_norm", "input_conv", "delta_rule", "gated_recurrence", "state_space", "routed_experts", "norm_add",
                                   "linear", "attention_decode", "attention_prefill", "rmsnorm",
                                   "swiglu", "rope", "sample"])
@@ -189,6 +192,8 @@ def main(argv=None) -> int:
     p.add_argument("--top", type=int, default=8, help="routed_experts: chosen experts; norm_add: rows a token")
     p.add_argument("--rank", type=int, default=512, help="latent kernels: the cached latent (512)")
     p.add_argument("--rot", type=int, default=64, help="latent kernels: the shared rotated key part")
+    p.add_argument("--streams", type=int, default=4)
+    p.add_argument("--bias", type=int, default=0, help="attention: the span of a bias by distance (with sinks)")
     p.add_argument("--reps", type=int, default=20)
     p.add_argument("--once", action="store_true")
     p.add_argument("--timeline", action="store_true",
@@ -268,12 +273,13 @@ def main(argv=None) -> int:
         vc = torch.randn(n_pages, hkv, 64, d, device=DEV, dtype=bf16)
         table = torch.arange(n_pages, dtype=torch.int32, device=DEV).view(batch, pages_per)
         lens = torch.full((batch,), ctx, dtype=torch.int32, device=DEV)
+        extra = dict(bias=torch.randn(hq, args.bias, device=DEV), sinks=torch.zeros(hq, device=DEV)) if args.bias else {}
         if decode:
             qkv = torch.randn(batch, (hq + 2 * hkv) * d, device=DEV, dtype=bf16)
             pos = torch.full((batch,), ctx - 1, dtype=torch.int32, device=DEV)
             seq = torch.arange(batch, dtype=torch.int32, device=DEV)
             fn = lambda: attention(qkv, kc, vc, table, pages_per, pos, seq, hq, hkv, d, d ** -0.5, 0,
-                                   decode=True, seq_lens=lens, max_len=ctx)
+                                   decode=True, seq_lens=lens, max_len=ctx, **extra)
             if args.timeline:
                 return timeline(fn, f"attention_decode batch={batch} context={ctx} heads={hq}/{hkv} D={d}",
                                 "attention_decode")
@@ -285,7 +291,7 @@ def main(argv=None) -> int:
             seq = torch.zeros(ctx, dtype=torch.int32, device=DEV)
             cu = torch.tensor([0, ctx], dtype=torch.int32, device=DEV)
             fn = lambda: attention(qkv, kc, vc, table, pages_per, pos, seq, hq, hkv, d, d ** -0.5, 0,
-                                   seq_lens=lens, max_len=ctx, cu_seqlens=cu, max_new=ctx)
+                                   seq_lens=lens, max_len=ctx, cu_seqlens=cu, max_new=ctx, **extra)
             args.reps = min(args.reps, 5)
             if args.timeline:
                 return phase_sums(fn, f"attention_prefill tokens={ctx} heads={hq}/{hkv} D={d}")
@@ -395,6 +401,31 @@ def main(argv=None) -> int:
         run(lambda: ops.forget_recurrence(proj, bias, lower, state, cu, slots, weight, 1e-5, work, o, mixed, H, D, D,
                                           single_tokens=t == 1), args, moved, 5.0 * n * H * D * D,
             f"forget_recurrence {b} x {t} tokens, {H} heads with states of {D} x {D}")
+    elif args.op == "decay_recurrence":
+        # as forget_recurrence
+        from llm_b200 import ops
+        b, t, H, D = args.batch, args.tokens, args.heads, args.head_dim
+        n = b * t
+        cu, slots = torch.arange(b + 1, dtype=torch.int32, device=DEV) * t, torch.arange(b, dtype=torch.int32, device=DEV)
+        proj = torch.randn(n, 4 * H * D, device=DEV).to(bf16)
+        decays, weight = torch.linspace(0.5, 0.999, H, device=DEV), torch.ones(H * D, device=DEV)
+        state = torch.zeros(b, H * D * D, device=DEV)
+        work = torch.empty(n, ops.decay_recurrence_work_width(H, D, D), device=DEV)
+        o, mixed = torch.empty(n, H * D, device=DEV), torch.empty(n, H * D, device=DEV, dtype=bf16)
+        moved = proj.numel() * 2 + mixed.numel() * 2 + state.numel() * 8
+        run(lambda: ops.decay_recurrence(proj, decays, state, cu, slots, weight, 1e-5, work, o, mixed, H, D, D,
+                                         single_tokens=t == 1), args, moved, 5.0 * n * H * D * D,
+            f"decay_recurrence {b} x {t} tokens, {H} heads with states of {D} x {D}")
+    elif args.op == "streams":
+        # `--m` tokens of width `--k` in `--streams` streams, `--top` result rows a token, with the next part's input
+        from llm_b200 import ops
+        m, k, S = args.m, args.k, args.streams
+        X, y = torch.randn(m, S, k, device=DEV), torch.randn(m * args.top, k, device=DEV)
+        write = torch.cat([torch.ones(S), torch.eye(S).reshape(-1)]).to(DEV) * 0.9
+        read, gain = torch.ones(S, device=DEV) / S, torch.ones(k, device=DEV)
+        h = torch.empty(m, k, device=DEV, dtype=bf16)
+        run(lambda: ops.streams_update_(X, y, args.top, write, read, gain, 1e-5, h), args,
+            X.numel() * 8 + y.numel() * 4 + h.numel() * 2, 0.0, f"streams {m} tokens x {S} of {k}, {args.top} rows a token")
     elif args.op in ("latent_attention", "latent_prefill", "latent_write", "head_products"):
         # latent rows of `--rank` + `--rot`, `--heads` heads of `--head-dim` + `--rot`, values of `--head-dim`. latent_attention:
         # a decode step of `--batch` sequences at `--context`, or (`--tokens` > 1) the last `--tokens` tokens of each
