@@ -360,8 +360,10 @@ expert_product_kernel(const T* __restrict__ A, int lda, int a_div, const T* __re
 // ---------------------------------------------------------------------------------------------- tensor cores
 
 // 32 rows x 128 columns a block of four warps (a warp: 32 x 32), k in steps of 32 through shared memory
-// (cp.async, two stages); for GLU the 128 columns are 64 gate and the 64 up columns of the same features.
-constexpr int TC_BN = 128, TC_BK = 32, TC_LD = TC_BK + 8;
+// (cp.async, a ring of stages: a decode step streams the experts' matrices, and what a block has in flight sets its rate);
+// for GLU the 128 columns are 64 gate and the 64 up columns of the same features.
+constexpr int TC_BN = 128, TC_BK = 32, TC_LD = TC_BK + 8, TC_STAGES = 4;
+constexpr size_t TC_SMEM = sizeof(__nv_bfloat16) * TC_STAGES * (TILE_M + TC_BN) * TC_LD;
 
 template <bool GLU>
 __global__ void __launch_bounds__(128)
@@ -369,8 +371,9 @@ expert_product_tc_kernel(const __nv_bfloat16* __restrict__ A, int lda, int a_div
                          long long w_stride, int N, int K, const int* __restrict__ sorted, const int* __restrict__ plan,
                          int E, int max_tiles, __nv_bfloat16* __restrict__ act, float* __restrict__ y,
                          const float* __restrict__ weights, Activation activation) {
-    __shared__ __align__(16) __nv_bfloat16 As[2][TILE_M][TC_LD];
-    __shared__ __align__(16) __nv_bfloat16 Bs[2][TC_BN][TC_LD];
+    extern __shared__ __align__(16) unsigned char stages_raw[];
+    auto As = reinterpret_cast<__nv_bfloat16 (*)[TILE_M][TC_LD]>(stages_raw);
+    auto Bs = reinterpret_cast<__nv_bfloat16 (*)[TC_BN][TC_LD]>(stages_raw + sizeof(__nv_bfloat16) * TC_STAGES * TILE_M * TC_LD);
     griddep_launch();
     griddep_wait();
     int tile = blockIdx.y;
@@ -396,20 +399,25 @@ expert_product_tc_kernel(const __nv_bfloat16* __restrict__ A, int lda, int a_div
             long long w_row = GLU ? (long long)((n >> 6) * N + feature) : (long long)feature;
             if (feature < N) cp_async16(&Bs[stage][n][piece], We + w_row * K + k0 + piece);
         }
-        cp_async_commit();
     };
     // rows and columns that are never loaded must read as zeros
-    for (int i = threadIdx.x; i < 2 * TILE_M * TC_LD; i += 128) (&As[0][0][0])[i] = __float2bfloat16(0.f);
-    for (int i = threadIdx.x; i < 2 * TC_BN * TC_LD; i += 128) (&Bs[0][0][0])[i] = __float2bfloat16(0.f);
-    __syncthreads();
+    if (rows < TILE_M || n0 + FEATURES > N) {
+        for (int i = threadIdx.x; i < (int)(TC_SMEM / 16); i += 128) reinterpret_cast<uint4*>(stages_raw)[i] = make_uint4(0u, 0u, 0u, 0u);
+        __syncthreads();
+    }
     float acc[2][4][4] = {};               // [row block of 16][column block of 8][fragment]
     int n_k = K / TC_BK;
-    request(0, 0);
+#pragma unroll
+    for (int st = 0; st < TC_STAGES - 1; ++st) {
+        if (st < n_k) request(st, st * TC_BK);
+        cp_async_commit();
+    }
     for (int kb = 0; kb < n_k; ++kb) {
-        int stage = kb & 1;
-        if (kb + 1 < n_k) { request(stage ^ 1, (kb + 1) * TC_BK); cp_async_wait<1>(); }
-        else cp_async_wait<0>();
-        __syncthreads();
+        int stage = kb % TC_STAGES;
+        cp_async_wait<TC_STAGES - 2>();
+        __syncthreads();                   // step kb has landed, and everyone is done with step kb - 1, whose stage is requested again
+        if (kb + TC_STAGES - 1 < n_k) request((kb + TC_STAGES - 1) % TC_STAGES, (kb + TC_STAGES - 1) * TC_BK);
+        cp_async_commit();
 #pragma unroll
         for (int ks = 0; ks < TC_BK; ks += 16) {
             uint32_t a[2][4], b[2][4];
@@ -427,12 +435,12 @@ expert_product_tc_kernel(const __nv_bfloat16* __restrict__ A, int lda, int a_div
                     mma_bf16(acc[mi][ni * 2 + 1], a[mi][0], a[mi][1], a[mi][2], a[mi][3], b[ni][2], b[ni][3]);
                 }
         }
-        __syncthreads();
     }
     // accumulator element (mi, nj, f): row mi * 16 + lane / 4 + (f / 2) * 8, column warp * 32 + nj * 8 + (lane % 4) * 2 + f % 2
     if (GLU) {
         // gate columns live in warps 0-1, up columns in warps 2-3: exchanged through shared memory
-        __shared__ float up[TILE_M][64 + 1];
+        __syncthreads();                   // the stages have been read
+        auto up = reinterpret_cast<float (*)[64 + 1]>(stages_raw);
         if (warp >= 2)
 #pragma unroll
             for (int mi = 0; mi < 2; ++mi)
@@ -796,10 +804,16 @@ LLMB_EXPORT int llmb_routed_experts(const void* h, int ld, int dtype, const floa
                                (const int*)sorted, down_weights, activation, status_dev));
     } else if (tc) {
         typedef __nv_bfloat16 B;
-        LLMB_CUDA(llmb::launch(expert_product_tc_kernel<true>, dim3((F + 63) / 64, max_tiles), dim3(128), 0, stream, true,
+        static bool configured = false;
+        if (!configured) {
+            LLMB_CUDA(cudaFuncSetAttribute(expert_product_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC_SMEM));
+            LLMB_CUDA(cudaFuncSetAttribute(expert_product_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC_SMEM));
+            configured = true;
+        }
+        LLMB_CUDA(llmb::launch(expert_product_tc_kernel<true>, dim3((F + 63) / 64, max_tiles), dim3(128), TC_SMEM, stream, true,
                                (const B*)h, ld, top, (const B*)w_up, up_stride, F, hidden, (const int*)sorted,
                                (const int*)plan, E, max_tiles, (B*)act, (float*)nullptr, up_weights, activation));
-        LLMB_CUDA(llmb::launch(expert_product_tc_kernel<false>, dim3((hidden + 127) / 128, max_tiles), dim3(128), 0, stream,
+        LLMB_CUDA(llmb::launch(expert_product_tc_kernel<false>, dim3((hidden + 127) / 128, max_tiles), dim3(128), TC_SMEM, stream,
                                true, (const B*)act, F, 1, (const B*)w_down, down_stride, hidden, F, (const int*)sorted,
                                (const int*)plan, E, max_tiles, (B*)nullptr, y, down_weights, activation));
     } else if (dtype == LLMB_DTYPE_F32) {

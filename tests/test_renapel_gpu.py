@@ -36,7 +36,7 @@ def test_streams(dtype, case):
     width, S, terms = case
     gen = torch.Generator().manual_seed(width + S)
     new = lambda *shape: torch.randn(shape, generator=gen).to(DEV)
-    for n in (1, 9, 70):
+    for n in (1, 9, 300):
         X, y, write, read, gain = new(n, S, width), new(n * terms, width), new(S + S * S), new(S), 1.0 + 0.3 * new(width)
         for wanted in (True, False):
             got, want = X.clone(), X.clone()
@@ -56,6 +56,22 @@ def test_streams(dtype, case):
         tokens = torch.randint(0, 50, (n,), generator=gen).to(torch.int32).to(DEV)
         table = new(50, width).to(dtype)
         assert torch.equal(ops.streams_embed(tokens, table, S, 0.5), plain_ops.streams_embed(tokens, table, S, 0.5))
+
+
+@pytest.mark.parametrize("width", [2048, 4096, 6148])
+def test_streams_give_a_token_the_same_bits_in_any_step(width):
+    """Steps of few and of many tokens take different launches: a token's streams and its input are equal to the last bit."""
+    ops = _ops()
+    S, n = 4, 300
+    gen = torch.Generator().manual_seed(width)
+    new = lambda *shape: torch.randn(shape, generator=gen).to(DEV)
+    X, y, write, read, gain = new(n, S, width), new(n * 2, width), new(S + S * S), new(S), new(width)
+    whole, part = X.clone(), X[:7].clone()
+    out, few = torch.zeros((n, width), device=DEV), torch.zeros((7, width), device=DEV)
+    ops.streams_update_(whole, y, 2, write, read, gain, 1e-5, out)
+    ops.streams_update_(part, y[:14].contiguous(), 2, write, read, gain, 1e-5, few)
+    assert torch.equal(whole[:7], part) and torch.equal(out[:7], few)
+    assert torch.equal(ops.streams_read(whole, read, gain, 1e-5, torch.float32), out)
 
 
 def test_streams_mix_from_the_first_index_to_the_second():
