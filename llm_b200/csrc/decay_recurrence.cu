@@ -12,6 +12,11 @@
 // steps of one token a sequence: a block per head and sequence requests the head's state before the kernel in front has
 //     ended (nothing else in a step touches it), then silu, update and read-out; finish.
 // Both sum in the same order.
+// bfloat16 steps of many tokens (sizes in llmb_decay_recurrence): with one decay per head the tokens of a chunk can be taken
+//     together, and the work is matrix products (chunk_kernel below): prepare writes bfloat16 rows, the chunks replace the
+//     scan, finish. The state stays 32-bit: where it, or anything else of 32 bits, is an operand of a product, it
+//     enters as three bfloat16 parts that add up to its 24 bits.
+#include "mma.cuh"
 #include "row_scan.cuh"
 
 using namespace llmb;
@@ -22,15 +27,15 @@ constexpr int THREADS = 256;
 
 __device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
 
-template <typename T, int VEC>
+template <typename T, int VEC, typename TWork>
 __global__ void __launch_bounds__(THREADS)
-decay_prepare_kernel(const T* __restrict__ proj, int ld, float* __restrict__ work, int work_ld, int keys, int values) {
+decay_prepare_kernel(const T* __restrict__ proj, int ld, TWork* __restrict__ work, int work_ld, int keys, int values) {
     griddep_launch();
     griddep_wait();
     proj = behind_wait(proj);
     size_t t = blockIdx.x;
     const T* in = proj + t * ld;
-    float* out = work + t * work_ld;
+    TWork* out = work + t * work_ld;
     for (int c = threadIdx.x * VEC; c < 2 * keys + values; c += THREADS * VEC) {
         T raw[VEC];
         float r[VEC];
@@ -40,10 +45,231 @@ decay_prepare_kernel(const T* __restrict__ proj, int ld, float* __restrict__ wor
         int to = c < keys ? keys + c : c < 2 * keys ? c - keys : c;          // k in front of q
 #pragma unroll
         for (int i = 0; i < VEC; ++i) r[i] = silu(to_float(raw[i]));
-        if constexpr (VEC == 4) *reinterpret_cast<float4*>(out + to) = make_float4(r[0], r[1], r[2], r[3]);
-        else out[to] = r[0];
+        if constexpr (VEC == 4 && sizeof(TWork) == 2) *reinterpret_cast<uint2*>(out + to) = make_uint2(pack_bf16(r[0], r[1]), pack_bf16(r[2], r[3]));
+        else if constexpr (VEC == 4) *reinterpret_cast<float4*>(out + to) = make_float4(r[0], r[1], r[2], r[3]);
+        else out[to] = from_float<TWork>(r[0]);
     }
 }
+
+// ---------------------------------------------------------------------------------------------- chunks of tokens
+
+// With b = decay, for the token i of a chunk that starts from the state S:
+//     o_i = b^(i + 1) S^T q_i + sum_{j <= i} b^(i - j) (q_i . k_j) v_j,      S' = b^n S + sum_j b^(n - 1 - j) k_j v_j^T
+// (n tokens in the chunk). A block takes 32 columns of a head's state for one sequence, eight warps (mma.sync, 32-bit
+// accumulation): warp w holds the state's rows 16 w .. in registers as 32-bit accumulators of the second formula, and works on
+// the rows 16 (w % 4) .. and columns 16 (w / 4) .. of the chunk's results. q, k and v are bfloat16 as they are; the state, the
+// weights b^(i - j) (q_i . k_j) and the faded values are split into three bfloat16 parts. The chunks' rows come by
+// cp.async, the next under the current.
+namespace chunk {
+
+constexpr int C = 64, VT = 32, WARPS = 8, LDV = VT + 8;
+
+__device__ __forceinline__ void split3(float x, float& a, float& b, float& c) {
+    a = __bfloat162float(__float2bfloat16_rn(x));
+    float r = x - a;
+    b = __bfloat162float(__float2bfloat16_rn(r));
+    c = r - b;                                               // (rounded when it is packed)
+}
+// two neighbouring values as packed parts
+__device__ __forceinline__ void split_pair(float lo, float hi, uint32_t (&part)[3]) {
+    float a0, b0, c0, a1, b1, c1;
+    split3(lo, a0, b0, c0);
+    split3(hi, a1, b1, c1);
+    part[0] = pack_bf16(a0, a1);
+    part[1] = pack_bf16(b0, b1);
+    part[2] = pack_bf16(c0, c1);
+}
+
+template <int D>
+constexpr size_t smem_bytes() {
+    return sizeof(__nv_bfloat16) * (2 * 2 * C * (D + 8) + 2 * C * LDV + 3 * D * LDV + 3 * C * LDV) + sizeof(float) * (C + 4);
+}
+
+template <int D>
+__global__ void __launch_bounds__(WARPS * 32, 1)
+decay_chunk_kernel(const __nv_bfloat16* __restrict__ work, int work_ld, float* __restrict__ state, long long state_stride,
+                   const int* __restrict__ cu_seqlens, const int* __restrict__ slot_ids, const float* __restrict__ decays,
+                   float* __restrict__ o, int H, int V) {
+    typedef __nv_bfloat16 B;
+    constexpr int LDD = D + 8;
+    extern __shared__ __align__(16) unsigned char raw[];
+    auto Ks = reinterpret_cast<B (*)[C][LDD]>(raw);                                  // [2]
+    auto Qs = reinterpret_cast<B (*)[C][LDD]>(raw + sizeof(B) * 2 * C * LDD);        // [2]
+    auto Vs = reinterpret_cast<B (*)[C][LDV]>(raw + sizeof(B) * 4 * C * LDD);        // [2]
+    auto Sp = reinterpret_cast<B (*)[D][LDV]>(raw + sizeof(B) * (4 * C * LDD + 2 * C * LDV));                 // [3] the state's parts
+    auto Vp = reinterpret_cast<B (*)[C][LDV]>(raw + sizeof(B) * (4 * C * LDD + 2 * C * LDV + 3 * D * LDV));    // [3] the faded values'
+    float* power = reinterpret_cast<float*>(raw + sizeof(B) * (4 * C * LDD + 2 * C * LDV + 3 * D * LDV + 3 * C * LDV));   // [C + 1] b^n
+    griddep_launch();
+    int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+    int head = blockIdx.y, seq = blockIdx.z, v0 = blockIdx.x * VT;
+    int first = cu_seqlens[seq], n_new = cu_seqlens[seq + 1] - first;
+    if (tid == 0) {
+        double b = decays[head], p = 1.0;
+        for (int n = 0; n <= C; ++n) { power[n] = (float)p; p *= b; }
+    }
+    float* S = state + (long long)slot_ids[seq] * state_stride + (size_t)head * D * V;   // [V, D]
+    const bool owns = warp * 16 < D;
+    float s[4][4];                                           // rows warp * 16 + g, + 8; columns nt * 8 + 2 t4, + 1
+#pragma unroll
+    for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+        for (int f = 0; f < 4; ++f) {
+            int d = warp * 16 + g + (f >> 1) * 8, v = v0 + nt * 8 + 2 * t4 + (f & 1);
+            s[nt][f] = owns && n_new > 0 && v < V ? S[(size_t)v * D + d] : 0.f;
+        }
+    griddep_wait();
+    if (n_new <= 0) return;
+    work = behind_wait(work);
+    const int keys = H * D;
+    const B* k_from = work + (size_t)first * work_ld + head * D;
+    const B* v_from = work + (size_t)first * work_ld + 2 * keys + head * V + v0;
+    auto request = [&](int chunk) {                          // rows beyond the step's tokens become zeros
+        int st = chunk & 1, t0 = chunk * C, count = min(C, n_new - t0);
+        const uint4 none = make_uint4(0u, 0u, 0u, 0u);
+        for (int i = tid; i < C * (D / 8); i += WARPS * 32) {
+            int r = i / (D / 8), c = i % (D / 8) * 8;
+            if (r < count) {
+                cp_async16(&Ks[st][r][c], k_from + (size_t)(t0 + r) * work_ld + c);
+                cp_async16(&Qs[st][r][c], k_from + (size_t)(t0 + r) * work_ld + keys + c);
+            } else {
+                *reinterpret_cast<uint4*>(&Ks[st][r][c]) = none;
+                *reinterpret_cast<uint4*>(&Qs[st][r][c]) = none;
+            }
+        }
+        for (int i = tid; i < C * (VT / 8); i += WARPS * 32) {
+            int r = i / (VT / 8), c = i % (VT / 8) * 8;
+            if (r < count && v0 + c < V) cp_async16(&Vs[st][r][c], v_from + (size_t)(t0 + r) * work_ld + c);
+            else *reinterpret_cast<uint4*>(&Vs[st][r][c]) = none;
+        }
+        cp_async_commit();
+    };
+    const int n_chunks = (n_new + C - 1) / C;
+    const int mt = warp & 3, nh = warp >> 2;                 // this warp's rows and columns of the results
+    request(0);
+    for (int chunk = 0; chunk < n_chunks; ++chunk) {
+        int st = chunk & 1, t0 = chunk * C, count = min(C, n_new - t0);
+        cp_async_wait<0>();
+        __syncthreads();                                     // the chunk landed; everyone is done with the one before and its parts
+        if (chunk + 1 < n_chunks) request(chunk + 1);
+        // ---- the parts: the state before the chunk, and the values as the state after the chunk wants them
+        if (owns) {
+#pragma unroll
+            for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+                for (int f = 0; f < 2; ++f) {
+                    uint32_t part[3];
+                    split_pair(s[nt][2 * f], s[nt][2 * f + 1], part);
+#pragma unroll
+                    for (int p = 0; p < 3; ++p)
+                        *reinterpret_cast<uint32_t*>(&Sp[p][warp * 16 + g + f * 8][nt * 8 + 2 * t4]) = part[p];
+                }
+        }
+        for (int i = tid; i < C * VT / 2; i += WARPS * 32) {
+            int r = i / (VT / 2), c = i % (VT / 2) * 2;
+            float fade = r < count ? power[count - 1 - r] : 0.f;
+            uint32_t part[3];
+            split_pair(to_float(Vs[st][r][c]) * fade, to_float(Vs[st][r][c + 1]) * fade, part);
+#pragma unroll
+            for (int p = 0; p < 3; ++p) *reinterpret_cast<uint32_t*>(&Vp[p][r][c]) = part[p];
+        }
+        __syncthreads();
+        // ---- results: what the state gives (16 rows x 16 columns a warp)
+        if (mt * 16 < count) {
+            float acc[2][4] = {}, w[8][4] = {};              // w: q_i . k_j for this warp's rows, 8 keys a block
+            const int blocks = 2 * (mt + 1);                 // keys up to the last row's own
+#pragma unroll
+            for (int k = 0; k < D; k += 16) {
+                uint32_t a[4];
+                ldmatrix_x4(a, &Qs[st][mt * 16 + (lane & 15)][k + (lane >> 4) * 8]);
+#pragma unroll
+                for (int p = 0; p < 3; ++p) {
+                    uint32_t b[4];
+                    ldmatrix_x4_trans(b, &Sp[p][k + ((lane >> 3) & 1) * 8 + (lane & 7)][nh * 16 + (lane >> 4) * 8]);
+                    mma_bf16(acc[0], a[0], a[1], a[2], a[3], b[0], b[1]);
+                    mma_bf16(acc[1], a[0], a[1], a[2], a[3], b[2], b[3]);
+                }
+#pragma unroll
+                for (int nb = 0; nb < 8; nb += 2) {
+                    if (nb >= blocks) break;
+                    uint32_t b[4];
+                    ldmatrix_x4(b, &Ks[st][nb * 8 + (lane >> 4) * 8 + (lane & 7)][k + ((lane >> 3) & 1) * 8]);
+                    mma_bf16(w[nb], a[0], a[1], a[2], a[3], b[0], b[1]);
+                    mma_bf16(w[nb + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
+                }
+            }
+            int row0 = mt * 16 + g, row1 = row0 + 8;
+            float fade0 = power[row0 + 1], fade1 = power[row1 + 1];
+#pragma unroll
+            for (int n = 0; n < 2; ++n) { acc[n][0] *= fade0; acc[n][1] *= fade0; acc[n][2] *= fade1; acc[n][3] *= fade1; }
+            // ---- and what the chunk's own tokens give
+#pragma unroll
+            for (int kk = 0; kk < 4; ++kk) {
+                if (kk > mt) break;
+                uint32_t a[4][3];                            // the four registers of the operand, in parts
+#pragma unroll
+                for (int h = 0; h < 2; ++h) {
+                    int nb = 2 * kk + h, j = nb * 8 + 2 * t4;
+                    float x[4];
+#pragma unroll
+                    for (int f = 0; f < 4; ++f) {
+                        int back = (f < 2 ? row0 : row1) - (j + (f & 1));
+                        x[f] = back >= 0 ? w[nb][f] * power[back] : 0.f;
+                    }
+                    split_pair(x[0], x[1], a[2 * h]);
+                    split_pair(x[2], x[3], a[2 * h + 1]);
+                }
+                uint32_t b[4];
+                ldmatrix_x4_trans(b, &Vs[st][kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)][nh * 16 + (lane >> 4) * 8]);
+#pragma unroll
+                for (int p = 0; p < 3; ++p) {
+                    mma_bf16(acc[0], a[0][p], a[1][p], a[2][p], a[3][p], b[0], b[1]);
+                    mma_bf16(acc[1], a[0][p], a[1][p], a[2][p], a[3][p], b[2], b[3]);
+                }
+            }
+#pragma unroll
+            for (int n = 0; n < 2; ++n)
+#pragma unroll
+                for (int f = 0; f < 2; ++f) {
+                    int r = f ? row1 : row0, v = v0 + nh * 16 + n * 8 + 2 * t4;
+                    if (r < count && v < V)
+                        *reinterpret_cast<float2*>(o + (size_t)(first + t0 + r) * H * V + head * V + v) = make_float2(acc[n][2 * f], acc[n][2 * f + 1]);
+                }
+        }
+        // ---- the state after the chunk
+        if (owns) {
+            float fade = power[count];
+#pragma unroll
+            for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+                for (int f = 0; f < 4; ++f) s[nt][f] *= fade;
+#pragma unroll
+            for (int k = 0; k < C; k += 16) {
+                if (k >= count) break;
+                uint32_t a[4];                               // rows of k as columns: the operand is K^T
+                ldmatrix_x4_trans(a, &Ks[st][k + ((lane >> 4) & 1) * 8 + (lane & 7)][warp * 16 + ((lane >> 3) & 1) * 8]);
+#pragma unroll
+                for (int p = 0; p < 3; ++p)
+#pragma unroll
+                    for (int n = 0; n < 4; n += 2) {
+                        uint32_t b[4];
+                        ldmatrix_x4_trans(b, &Vp[p][k + ((lane >> 3) & 1) * 8 + (lane & 7)][n * 8 + (lane >> 4) * 8]);
+                        mma_bf16(s[n], a[0], a[1], a[2], a[3], b[0], b[1]);
+                        mma_bf16(s[n + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
+                    }
+            }
+        }
+    }
+    if (!owns) return;
+#pragma unroll
+    for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+        for (int f = 0; f < 4; ++f) {
+            int d = warp * 16 + g + (f >> 1) * 8, v = v0 + nt * 8 + 2 * t4 + (f & 1);
+            if (v < V) S[(size_t)v * D + d] = s[nt][f];
+        }
+}
+
+}  // namespace chunk
 
 // One block per token: the factor of the norm over all heads, then weight and gate.
 template <typename T>
@@ -139,14 +365,19 @@ decay_step_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ 
     if ((lane & 3) == 0 && v0 + (lane >> 2) < V) o[t * H * V + head * V + v0 + (lane >> 2)] = total;
 }
 
+// Whether a step of these sizes takes the chunked form.
+LLMB_EXPORT int llmb_decay_recurrence_chunked(int dtype, int n_tokens, int n_seqs, int D, int V) {
+    return dtype == LLMB_DTYPE_BF16 && (D == 32 || D == 64 || D == 96 || D == 128) && V % 8 == 0 && n_tokens >= 16LL * n_seqs;
+}
+
 // proj [T, ld >= 2 H D + 2 H V] in `dtype`; decays float32 [H]; state float32 [slots, state_stride >= H D V]; weight
 // float32 [H V]; work float32 [T, work_ld >= 2 H D + H V] (scratch; not touched where the step takes its own kernel), o
 // float32 [T, H V] (scratch); mixed [T, mixed_ld] in `dtype` receives the H V result columns. single: every sequence
-// brings one token.
+// brings one token. chunks: whether steps that can may take the chunked form.
 LLMB_EXPORT int llmb_decay_recurrence(const void* proj, int ld, int dtype, const float* decays, float* state,
                                       long long state_stride, const int* cu_seqlens, const int* slot_ids, const float* weight,
                                       float eps, float* work, int work_ld, float* o, void* mixed, int mixed_ld, int n_tokens,
-                                      int n_seqs, int H, int D, int V, int single, cudaStream_t stream) {
+                                      int n_seqs, int H, int D, int V, int single, int chunks, cudaStream_t stream) {
     if (n_tokens == 0) return LLMB_OK;
     LLMB_REQUIRE(H > 0 && D > 0 && V > 0 && D <= 512, "decay_recurrence: %d heads with states of %d x %d (up to 512 rows are built)", H, D, V);
     LLMB_REQUIRE(n_seqs > 0 && n_seqs <= 65535 && H <= 65535, "decay_recurrence: bad sizes");
@@ -173,11 +404,32 @@ LLMB_EXPORT int llmb_decay_recurrence(const void* proj, int ld, int dtype, const
         if (dtype == LLMB_DTYPE_F32) LLMB_STEP(float); else LLMB_STEP(B);
 #undef LLMB_STEP
 #undef LLMB_STEP_AS
+    } else if (chunks && llmb_decay_recurrence_chunked(dtype, n_tokens, n_seqs, D, V) && ld % 4 == 0 && work_ld % 4 == 0 &&
+               (((size_t)proj | (size_t)work) % 16) == 0 && ((size_t)o % 8) == 0) {
+        LLMB_CUDA(llmb::launch(decay_prepare_kernel<B, 4, B>, dim3(n_tokens), dim3(THREADS), 0, stream, true, (const B*)proj, ld,
+                               (B*)work, 2 * work_ld, keys, values));
+        dim3 grid(ceil_div(V, chunk::VT), H, n_seqs);
+#define LLMB_CHUNK(DD)                                                                                                    \
+        do {                                                                                                              \
+            static bool configured = false;                                                                               \
+            if (!configured) {                                                                                            \
+                LLMB_CUDA(cudaFuncSetAttribute(chunk::decay_chunk_kernel<DD>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                               (int)chunk::smem_bytes<DD>()));                                            \
+                configured = true;                                                                                        \
+            }                                                                                                             \
+            LLMB_CUDA(llmb::launch(chunk::decay_chunk_kernel<DD>, grid, dim3(chunk::WARPS * 32), chunk::smem_bytes<DD>(), stream, true, \
+                                   (const B*)work, 2 * work_ld, state, state_stride, cu_seqlens, slot_ids, decays, o, H, V)); \
+        } while (0)
+        if (D == 32) LLMB_CHUNK(32);
+        else if (D == 64) LLMB_CHUNK(64);
+        else if (D == 96) LLMB_CHUNK(96);
+        else LLMB_CHUNK(128);
+#undef LLMB_CHUNK
     } else {
         bool wide_loads = keys % 4 == 0 && values % 4 == 0 && ld % 4 == 0 && work_ld % 4 == 0 && ((size_t)proj % (4 * esize)) == 0 &&
                           ((size_t)work % 16) == 0;
 #define LLMB_PREPARE(T, VEC)                                                                                              \
-        LLMB_CUDA(llmb::launch(decay_prepare_kernel<T, VEC>, dim3(n_tokens), dim3(THREADS), 0, stream, true, (const T*)proj, \
+        LLMB_CUDA(llmb::launch(decay_prepare_kernel<T, VEC, float>, dim3(n_tokens), dim3(THREADS), 0, stream, true, (const T*)proj, \
                                ld, work, work_ld, keys, values))
         if (dtype == LLMB_DTYPE_F32) { if (wide_loads) LLMB_PREPARE(float, 4); else LLMB_PREPARE(float, 1); }
         else { if (wide_loads) LLMB_PREPARE(B, 4); else LLMB_PREPARE(B, 1); }

@@ -1,6 +1,7 @@
 // A residual of several streams x_1 .. x_S per token (Zhu et al., "Hyper-Connections"), X [T, S, width] in 32-bit.
 //
-// streams_embed   every stream of a token is its row of the embedding table.
+// streams_embed   every stream of a token is its row of the embedding table. A pass's first kernel: it starts behind
+//                 everything before it, so that kernels of the pass may read states of sequences before their own wait.
 // streams_update  behind a part: y = the sum of a token's result rows (`terms` rows in index order), then, from the old
 //                 streams, x_t <- sum_s mix[s, t] x_s + out[t] y; and in the same launch, where `read` is given, the next
 //                 part's input: u = sum_s read[s] x_s (of the new streams), h = u / sqrt(mean(u^2) + eps) * gain.
@@ -178,7 +179,7 @@ LLMB_EXPORT int llmb_streams_embed(const int* tokens, const void* table, int dty
     LLMB_REQUIRE(S >= 1 && S <= MAX_STREAMS && width > 0 && vocab > 0, "streams_embed: %d streams (up to %d) of %d", S, MAX_STREAMS, width);
     bool vector = width % 4 == 0 && aligned16(table) && aligned16(X);
 #define LLMB_STREAMS_EMBED(T, VEC)                                                                                         \
-    LLMB_CUDA(llmb::launch(streams_embed_kernel<T, VEC>, dim3(n_tokens), dim3(256), 0, stream, true, tokens, (const T*)table, X, \
+    LLMB_CUDA(llmb::launch(streams_embed_kernel<T, VEC>, dim3(n_tokens), dim3(256), 0, stream, false, tokens, (const T*)table, X, \
                            S, width, vocab, scale))
     if (dtype == LLMB_DTYPE_F32) { if (vector) LLMB_STREAMS_EMBED(float, 4); else LLMB_STREAMS_EMBED(float, 1); }
     else if (dtype == LLMB_DTYPE_BF16) { if (vector) LLMB_STREAMS_EMBED(__nv_bfloat16, 4); else LLMB_STREAMS_EMBED(__nv_bfloat16, 1); }

@@ -843,7 +843,8 @@ def decay_recurrence(proj, decays, state, cu_seqlens, slot_ids, norm_weight, eps
     o / sqrt(mean(o^2) + eps) * norm_weight * sigmoid(gate) (norm_weight float32 [H V]) into `mixed` [T, H V] (run dtype).
     `state` float32 [slots, H V D]: S as [H, V, D], read and updated for the slots of the step. `work` float32
     [T, decay_recurrence_work_width], `o` float32 [T, H V]: scratch. `single_tokens`: every sequence brings exactly one
-    token (token b is sequence b's)."""
+    token (token b is sequence b's). Long bfloat16 steps of the sizes that have it take a chunked form on tensor cores
+    (q, k and v rounded behind silu; switched off by disabling 'decay_recurrence_chunks')."""
     _require_cuda(proj, decays, state, cu_seqlens, slot_ids, norm_weight, work, o, mixed)
     n, H, D, V = proj.shape[0], n_heads, dim, vdim
     if proj.dim() != 2 or proj.shape[1] < 2 * H * (D + V) or proj.stride(1) != 1:
@@ -863,8 +864,8 @@ def decay_recurrence(proj, decays, state, cu_seqlens, slot_ids, norm_weight, eps
     _call("decay_recurrence", "llmb_decay_recurrence", _ptr(proj), _c_int(proj.stride(0)), _c_int(_code(proj.dtype)),
           _ptr(decays), _ptr(state), ctypes.c_longlong(state.stride(0)), _ptr(cu_seqlens), _ptr(slot_ids),
           _ptr(norm_weight), _c_float(eps), _ptr(work), _c_int(work.shape[1]), _ptr(o), _ptr(mixed), _c_int(mixed.stride(0)),
-          _c_int(n), _c_int(n_seqs), _c_int(H), _c_int(D), _c_int(V), _c_int(1 if single_tokens else 0), _stream(),
-          kernels=2 if one else 3)
+          _c_int(n), _c_int(n_seqs), _c_int(H), _c_int(D), _c_int(V), _c_int(1 if single_tokens else 0),
+          _c_int(0 if tactics.is_disabled("decay_recurrence_chunks") else 1), _stream(), kernels=2 if one else 3)
     return mixed
 
 

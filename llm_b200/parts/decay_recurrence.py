@@ -19,8 +19,8 @@ class DecayRecurrenceMixer(ProjectedMixer):
 
     One product [q; k; v; gate] (rows padded to a multiple of 8), then ops.decay_recurrence (silu, the scan over each
     sequence's tokens, norm and gate: two launches in a decode step, three else), then the output product. Per sequence
-    the cache holds S as one float32 row [heads, value_dim, head_dim]; zeroed when a slot is taken. Everything behind the
-    projection is 32-bit in every run."""
+    the cache holds S as one float32 row [heads, value_dim, head_dim]; zeroed when a slot is taken. Behind the silu
+    everything is 32-bit in every run; long bfloat16 steps round q, k and v there and take the tokens of a chunk together."""
     libraries = ("elementwise", "gemm_simt", "gemm_skinny", "gemm_tc", "decay_recurrence")
 
     def __init__(self, spec):

@@ -138,6 +138,35 @@ def test_decay_recurrence(dtype, case):
         assert float((states[0] - states[1]).abs().max()) <= (3e-6 if dtype == torch.float32 else 1e-2) * top, (case, lengths)
 
 
+@pytest.mark.parametrize("case", [(3, 32, 48), (2, 64, 64), (1, 96, 40), (4, 128, 128), (2, 128, 8)])
+def test_chunks_of_tokens_agree_with_the_scan_to_32_bit(case):
+    """The chunked form beside the scan on inputs whose silu is exact in bfloat16 (0 and whole numbers of 20 and more), with
+    a state of 32-bit numbers: what is left is the order of the sums. Steps that end inside a chunk, on its edge and just
+    beyond; sequences of one token beside long ones; small and large decays, zero and one."""
+    ops = _ops()
+    H, D, V = case
+    for lengths, new in (([64], [64]), ([65, 63, 300], [65, 63, 300]), ([200, 9, 1, 129], [130, 2, 1, 128]), ([17], [17]), ([700, 1], [640, 1])):
+        batch = Batch(lengths, new, seed=1)
+        gen = torch.Generator().manual_seed(D + len(new))
+        n, width = batch.n_tokens, 2 * H * (D + V)
+        whole = torch.randint(20, 40, (n, width), generator=gen).float() * (torch.rand((n, width), generator=gen) < 0.3)
+        proj = whole.to(torch.bfloat16).to(DEV)
+        decays = torch.tensor([0.999, 0.6, 0.0, 1.0][:H], device=DEV)
+        state = (1e4 * torch.randn((len(lengths) + 1, H * D * V), generator=gen)).abs().to(DEV)
+        results = []
+        for without in ((), ("decay_recurrence_chunks",)):
+            held, o = state.clone(), torch.zeros((n, H * V), device=DEV)
+            work = torch.zeros((n, ops.decay_recurrence_work_width(H, D, V)), device=DEV)
+            mixed = torch.zeros((n, H * V), dtype=torch.bfloat16, device=DEV)
+            with off(*without):
+                ops.decay_recurrence(proj, decays, held, batch.cu, batch.slots, torch.ones(H * V, device=DEV), 1e-5, work, o, mixed,
+                                     H, D, V, single_tokens=False)
+            results.append((o, held))
+        assert float(results[1][0].abs().max()) > 0.0
+        for got, want in zip(*results):
+            assert torch.allclose(got, want, rtol=3e-6, atol=0.0), (case, new, float(((got - want).abs() / want.abs().clamp_min(1e-20)).max()))
+
+
 @pytest.mark.parametrize("case", [(2, 12, 10), (1, 128, 128), (2, 100, 36)])
 def test_decay_recurrence_carries_its_state_across_any_cut(case):
     """A sequence in one step, and the same cut into two (the second also token by token, in the launch of its own for
