@@ -44,7 +44,11 @@ decay_prepare_kernel(const T* __restrict__ proj, int ld, TWork* __restrict__ wor
         else raw[0] = in[c];
         int to = c < keys ? keys + c : c < 2 * keys ? c - keys : c;          // k in front of q
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) r[i] = silu(to_float(raw[i]));
+        for (int i = 0; i < VEC; ++i) {
+            float z = to_float(raw[i]);
+            // (what is rounded to bfloat16 next takes the hardware's exponential and quotient)
+            r[i] = sizeof(TWork) == 2 ? __fdividef(z, 1.0f + __expf(-z)) : silu(z);
+        }
         if constexpr (VEC == 4 && sizeof(TWork) == 2) *reinterpret_cast<uint2*>(out + to) = make_uint2(pack_bf16(r[0], r[1]), pack_bf16(r[2], r[3]));
         else if constexpr (VEC == 4) *reinterpret_cast<float4*>(out + to) = make_float4(r[0], r[1], r[2], r[3]);
         else out[to] = from_float<TWork>(r[0]);
@@ -55,14 +59,15 @@ decay_prepare_kernel(const T* __restrict__ proj, int ld, TWork* __restrict__ wor
 
 // With b = decay, for the token i of a chunk that starts from the state S:
 //     o_i = b^(i + 1) S^T q_i + sum_{j <= i} b^(i - j) (q_i . k_j) v_j,      S' = b^n S + sum_j b^(n - 1 - j) k_j v_j^T
-// (n tokens in the chunk). A block takes 32 columns of a head's state for one sequence, eight warps (mma.sync, 32-bit
-// accumulation): warp w holds the state's rows 16 w .. in registers as 32-bit accumulators of the second formula, and works on
-// the rows 16 (w % 4) .. and columns 16 (w / 4) .. of the chunk's results. q, k and v are bfloat16 as they are; the state, the
-// weights b^(i - j) (q_i . k_j) and the faded values are split into three bfloat16 parts. The chunks' rows come by
+// (n tokens in the chunk). A block takes 32 columns of a head's state for one sequence, sixteen warps (mma.sync, 32-bit
+// accumulation). The state lives in registers, as the 32-bit accumulators of the second formula: 16 rows and 16 columns a warp.
+// q, k and v are bfloat16 as they are; the state, the weights b^(i - j) (q_i . k_j) and the faded values b^(n - 1 - j) v_j are
+// split into three bfloat16 parts each in shared memory. Per chunk: first all parts (16 rows and 16 keys of the weights a
+// warp), then, behind one barrier, the results (16 rows and 8 columns a warp) and the new state. The chunks' rows come by
 // cp.async, the next under the current.
 namespace chunk {
 
-constexpr int C = 64, VT = 32, WARPS = 8, LDV = VT + 8;
+constexpr int C = 64, VT = 32, WARPS = 16, LDV = VT + 8, LDW = C + 8;
 
 __device__ __forceinline__ void split3(float x, float& a, float& b, float& c) {
     a = __bfloat162float(__float2bfloat16_rn(x));
@@ -80,10 +85,14 @@ __device__ __forceinline__ void split_pair(float lo, float hi, uint32_t (&part)[
     part[2] = pack_bf16(c0, c1);
 }
 
+// bfloat16 elements in front of each part of shared memory
 template <int D>
-constexpr size_t smem_bytes() {
-    return sizeof(__nv_bfloat16) * (2 * 2 * C * (D + 8) + 2 * C * LDV + 3 * D * LDV + 3 * C * LDV) + sizeof(float) * (C + 4);
-}
+struct Place {
+    static constexpr int LDD = D + 8;
+    static constexpr int K = 0, Q = K + 2 * C * LDD, V = Q + 2 * C * LDD, S = V + 2 * C * LDV, F = S + 3 * D * LDV, W = F + 3 * C * LDV,
+                         END = W + 3 * C * LDW;
+    static constexpr size_t bytes = sizeof(__nv_bfloat16) * END + sizeof(float) * (C + 4);
+};
 
 template <int D>
 __global__ void __launch_bounds__(WARPS * 32, 1)
@@ -91,14 +100,16 @@ decay_chunk_kernel(const __nv_bfloat16* __restrict__ work, int work_ld, float* _
                    const int* __restrict__ cu_seqlens, const int* __restrict__ slot_ids, const float* __restrict__ decays,
                    float* __restrict__ o, int H, int V) {
     typedef __nv_bfloat16 B;
-    constexpr int LDD = D + 8;
+    typedef Place<D> P;
     extern __shared__ __align__(16) unsigned char raw[];
-    auto Ks = reinterpret_cast<B (*)[C][LDD]>(raw);                                  // [2]
-    auto Qs = reinterpret_cast<B (*)[C][LDD]>(raw + sizeof(B) * 2 * C * LDD);        // [2]
-    auto Vs = reinterpret_cast<B (*)[C][LDV]>(raw + sizeof(B) * 4 * C * LDD);        // [2]
-    auto Sp = reinterpret_cast<B (*)[D][LDV]>(raw + sizeof(B) * (4 * C * LDD + 2 * C * LDV));                 // [3] the state's parts
-    auto Vp = reinterpret_cast<B (*)[C][LDV]>(raw + sizeof(B) * (4 * C * LDD + 2 * C * LDV + 3 * D * LDV));    // [3] the faded values'
-    float* power = reinterpret_cast<float*>(raw + sizeof(B) * (4 * C * LDD + 2 * C * LDV + 3 * D * LDV + 3 * C * LDV));   // [C + 1] b^n
+    B* base = reinterpret_cast<B*>(raw);
+    auto Ks = reinterpret_cast<B (*)[C][P::LDD]>(base + P::K);       // [2] stages
+    auto Qs = reinterpret_cast<B (*)[C][P::LDD]>(base + P::Q);
+    auto Vs = reinterpret_cast<B (*)[C][LDV]>(base + P::V);
+    auto Sp = reinterpret_cast<B (*)[D][LDV]>(base + P::S);          // [3] parts: the state before the chunk,
+    auto Vp = reinterpret_cast<B (*)[C][LDV]>(base + P::F);          // the faded values,
+    auto Wp = reinterpret_cast<B (*)[C][LDW]>(base + P::W);          // the weights
+    float* power = reinterpret_cast<float*>(base + P::END);          // [C + 1] b^n
     griddep_launch();
     int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
     int head = blockIdx.y, seq = blockIdx.z, v0 = blockIdx.x * VT;
@@ -108,13 +119,15 @@ decay_chunk_kernel(const __nv_bfloat16* __restrict__ work, int work_ld, float* _
         for (int n = 0; n <= C; ++n) { power[n] = (float)p; p *= b; }
     }
     float* S = state + (long long)slot_ids[seq] * state_stride + (size_t)head * D * V;   // [V, D]
-    const bool owns = warp * 16 < D;
-    float s[4][4];                                           // rows warp * 16 + g, + 8; columns nt * 8 + 2 t4, + 1
+    // this warp's part of the state: rows d0 + g, + 8; columns c0 + 8 nt + 2 t4, + 1 of the block's
+    const int d0 = (warp & 7) * 16, c0 = (warp >> 3) * 16;
+    const bool owns = d0 < D;
+    float s[2][4];
 #pragma unroll
-    for (int nt = 0; nt < 4; ++nt)
+    for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
         for (int f = 0; f < 4; ++f) {
-            int d = warp * 16 + g + (f >> 1) * 8, v = v0 + nt * 8 + 2 * t4 + (f & 1);
+            int d = d0 + g + (f >> 1) * 8, v = v0 + c0 + nt * 8 + 2 * t4 + (f & 1);
             s[nt][f] = owns && n_new > 0 && v < V ? S[(size_t)v * D + d] : 0.f;
         }
     griddep_wait();
@@ -144,24 +157,25 @@ decay_chunk_kernel(const __nv_bfloat16* __restrict__ work, int work_ld, float* _
         cp_async_commit();
     };
     const int n_chunks = (n_new + C - 1) / C;
-    const int mt = warp & 3, nh = warp >> 2;                 // this warp's rows and columns of the results
+    const int mt = warp & 3, nq = warp >> 2;                 // rows 16 mt .. of the results; keys 16 nq .., columns 8 nq ..
+    const int row0 = mt * 16 + g, row1 = row0 + 8;
     request(0);
     for (int chunk = 0; chunk < n_chunks; ++chunk) {
         int st = chunk & 1, t0 = chunk * C, count = min(C, n_new - t0);
         cp_async_wait<0>();
         __syncthreads();                                     // the chunk landed; everyone is done with the one before and its parts
         if (chunk + 1 < n_chunks) request(chunk + 1);
-        // ---- the parts: the state before the chunk, and the values as the state after the chunk wants them
+        // ---- the parts
         if (owns) {
 #pragma unroll
-            for (int nt = 0; nt < 4; ++nt)
+            for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
                 for (int f = 0; f < 2; ++f) {
                     uint32_t part[3];
                     split_pair(s[nt][2 * f], s[nt][2 * f + 1], part);
 #pragma unroll
                     for (int p = 0; p < 3; ++p)
-                        *reinterpret_cast<uint32_t*>(&Sp[p][warp * 16 + g + f * 8][nt * 8 + 2 * t4]) = part[p];
+                        *reinterpret_cast<uint32_t*>(&Sp[p][d0 + g + f * 8][c0 + nt * 8 + 2 * t4]) = part[p];
                 }
         }
         for (int i = tid; i < C * VT / 2; i += WARPS * 32) {
@@ -172,107 +186,115 @@ decay_chunk_kernel(const __nv_bfloat16* __restrict__ work, int work_ld, float* _
 #pragma unroll
             for (int p = 0; p < 3; ++p) *reinterpret_cast<uint32_t*>(&Vp[p][r][c]) = part[p];
         }
-        __syncthreads();
-        // ---- results: what the state gives (16 rows x 16 columns a warp)
-        if (mt * 16 < count) {
-            float acc[2][4] = {}, w[8][4] = {};              // w: q_i . k_j for this warp's rows, 8 keys a block
-            const int blocks = 2 * (mt + 1);                 // keys up to the last row's own
+        const bool rows_live = mt * 16 < count;
+        if (rows_live && nq <= mt) {
+            float w[2][4] = {};
 #pragma unroll
             for (int k = 0; k < D; k += 16) {
-                uint32_t a[4];
+                uint32_t a[4], b[4];
                 ldmatrix_x4(a, &Qs[st][mt * 16 + (lane & 15)][k + (lane >> 4) * 8]);
-#pragma unroll
-                for (int p = 0; p < 3; ++p) {
-                    uint32_t b[4];
-                    ldmatrix_x4_trans(b, &Sp[p][k + ((lane >> 3) & 1) * 8 + (lane & 7)][nh * 16 + (lane >> 4) * 8]);
-                    mma_bf16(acc[0], a[0], a[1], a[2], a[3], b[0], b[1]);
-                    mma_bf16(acc[1], a[0], a[1], a[2], a[3], b[2], b[3]);
-                }
-#pragma unroll
-                for (int nb = 0; nb < 8; nb += 2) {
-                    if (nb >= blocks) break;
-                    uint32_t b[4];
-                    ldmatrix_x4(b, &Ks[st][nb * 8 + (lane >> 4) * 8 + (lane & 7)][k + ((lane >> 3) & 1) * 8]);
-                    mma_bf16(w[nb], a[0], a[1], a[2], a[3], b[0], b[1]);
-                    mma_bf16(w[nb + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
-                }
-            }
-            int row0 = mt * 16 + g, row1 = row0 + 8;
-            float fade0 = power[row0 + 1], fade1 = power[row1 + 1];
-#pragma unroll
-            for (int n = 0; n < 2; ++n) { acc[n][0] *= fade0; acc[n][1] *= fade0; acc[n][2] *= fade1; acc[n][3] *= fade1; }
-            // ---- and what the chunk's own tokens give
-#pragma unroll
-            for (int kk = 0; kk < 4; ++kk) {
-                if (kk > mt) break;
-                uint32_t a[4][3];                            // the four registers of the operand, in parts
-#pragma unroll
-                for (int h = 0; h < 2; ++h) {
-                    int nb = 2 * kk + h, j = nb * 8 + 2 * t4;
-                    float x[4];
-#pragma unroll
-                    for (int f = 0; f < 4; ++f) {
-                        int back = (f < 2 ? row0 : row1) - (j + (f & 1));
-                        x[f] = back >= 0 ? w[nb][f] * power[back] : 0.f;
-                    }
-                    split_pair(x[0], x[1], a[2 * h]);
-                    split_pair(x[2], x[3], a[2 * h + 1]);
-                }
-                uint32_t b[4];
-                ldmatrix_x4_trans(b, &Vs[st][kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)][nh * 16 + (lane >> 4) * 8]);
-#pragma unroll
-                for (int p = 0; p < 3; ++p) {
-                    mma_bf16(acc[0], a[0][p], a[1][p], a[2][p], a[3][p], b[0], b[1]);
-                    mma_bf16(acc[1], a[0][p], a[1][p], a[2][p], a[3][p], b[2], b[3]);
-                }
+                ldmatrix_x4(b, &Ks[st][nq * 16 + (lane >> 4) * 8 + (lane & 7)][k + ((lane >> 3) & 1) * 8]);
+                mma_bf16(w[0], a[0], a[1], a[2], a[3], b[0], b[1]);
+                mma_bf16(w[1], a[0], a[1], a[2], a[3], b[2], b[3]);
             }
 #pragma unroll
             for (int n = 0; n < 2; ++n)
 #pragma unroll
                 for (int f = 0; f < 2; ++f) {
-                    int r = f ? row1 : row0, v = v0 + nh * 16 + n * 8 + 2 * t4;
-                    if (r < count && v < V)
-                        *reinterpret_cast<float2*>(o + (size_t)(first + t0 + r) * H * V + head * V + v) = make_float2(acc[n][2 * f], acc[n][2 * f + 1]);
+                    int r = f ? row1 : row0, j = nq * 16 + n * 8 + 2 * t4, back = r - j;
+                    uint32_t part[3];
+                    split_pair(back >= 0 ? w[n][2 * f] * power[back] : 0.f, back >= 1 ? w[n][2 * f + 1] * power[back - 1] : 0.f, part);
+#pragma unroll
+                    for (int p = 0; p < 3; ++p) *reinterpret_cast<uint32_t*>(&Wp[p][r][j]) = part[p];
                 }
+        }
+        __syncthreads();
+        // ---- results: what the state gives, faded, and what the chunk's own tokens give
+        if (rows_live) {
+            float acc[3][4] = {};                            // a sum per part: their products do not wait for one another
+#pragma unroll
+            for (int k = 0; k < D; k += 32) {
+                uint32_t a[2][4];
+                ldmatrix_x4(a[0], &Qs[st][mt * 16 + (lane & 15)][k + (lane >> 4) * 8]);
+                ldmatrix_x4(a[1], &Qs[st][mt * 16 + (lane & 15)][k + 16 + (lane >> 4) * 8]);
+#pragma unroll
+                for (int p = 0; p < 3; ++p) {
+                    uint32_t b[4];
+                    ldmatrix_x4_trans(b, &Sp[p][k + lane][nq * 8]);
+                    mma_bf16(acc[p], a[0][0], a[0][1], a[0][2], a[0][3], b[0], b[1]);
+                    mma_bf16(acc[p], a[1][0], a[1][1], a[1][2], a[1][3], b[2], b[3]);
+                }
+            }
+            float fade0 = power[row0 + 1], fade1 = power[row1 + 1];
+#pragma unroll
+            for (int p = 0; p < 3; ++p) { acc[p][0] *= fade0; acc[p][1] *= fade0; acc[p][2] *= fade1; acc[p][3] *= fade1; }
+#pragma unroll
+            for (int pair = 0; pair < 2; ++pair) {
+                if (2 * pair > mt) break;
+                uint32_t b[4];
+                ldmatrix_x4_trans(b, &Vs[st][pair * 32 + lane][nq * 8]);
+#pragma unroll
+                for (int h = 0; h < 2; ++h) {
+                    if (2 * pair + h > mt) break;
+#pragma unroll
+                    for (int p = 0; p < 3; ++p) {
+                        uint32_t a[4];
+                        ldmatrix_x4(a, &Wp[p][mt * 16 + (lane & 15)][pair * 32 + h * 16 + (lane >> 4) * 8]);
+                        mma_bf16(acc[p], a[0], a[1], a[2], a[3], b[2 * h], b[2 * h + 1]);
+                    }
+                }
+            }
+            int v = v0 + nq * 8 + 2 * t4;
+            float* to = o + (size_t)(first + t0) * H * V + head * V + v;
+#pragma unroll
+            for (int f = 0; f < 4; ++f) acc[0][f] += acc[1][f] + acc[2][f];
+            if (v < V) {
+                if (row0 < count) *reinterpret_cast<float2*>(to + (size_t)row0 * H * V) = make_float2(acc[0][0], acc[0][1]);
+                if (row1 < count) *reinterpret_cast<float2*>(to + (size_t)row1 * H * V) = make_float2(acc[0][2], acc[0][3]);
+            }
         }
         // ---- the state after the chunk
         if (owns) {
             float fade = power[count];
 #pragma unroll
-            for (int nt = 0; nt < 4; ++nt)
+            for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
                 for (int f = 0; f < 4; ++f) s[nt][f] *= fade;
+            float low[2][2][4] = {};                         // what the second and third parts add
 #pragma unroll
             for (int k = 0; k < C; k += 16) {
                 if (k >= count) break;
                 uint32_t a[4];                               // rows of k as columns: the operand is K^T
-                ldmatrix_x4_trans(a, &Ks[st][k + ((lane >> 4) & 1) * 8 + (lane & 7)][warp * 16 + ((lane >> 3) & 1) * 8]);
+                ldmatrix_x4_trans(a, &Ks[st][k + ((lane >> 4) & 1) * 8 + (lane & 7)][d0 + ((lane >> 3) & 1) * 8]);
 #pragma unroll
-                for (int p = 0; p < 3; ++p)
-#pragma unroll
-                    for (int n = 0; n < 4; n += 2) {
-                        uint32_t b[4];
-                        ldmatrix_x4_trans(b, &Vp[p][k + ((lane >> 3) & 1) * 8 + (lane & 7)][n * 8 + (lane >> 4) * 8]);
-                        mma_bf16(s[n], a[0], a[1], a[2], a[3], b[0], b[1]);
-                        mma_bf16(s[n + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
-                    }
+                for (int p = 0; p < 3; ++p) {
+                    uint32_t b[4];
+                    ldmatrix_x4_trans(b, &Vp[p][k + ((lane >> 3) & 1) * 8 + (lane & 7)][c0 + (lane >> 4) * 8]);
+                    mma_bf16(p == 0 ? s[0] : low[p - 1][0], a[0], a[1], a[2], a[3], b[0], b[1]);
+                    mma_bf16(p == 0 ? s[1] : low[p - 1][1], a[0], a[1], a[2], a[3], b[2], b[3]);
+                }
             }
+#pragma unroll
+            for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+                for (int f = 0; f < 4; ++f) s[nt][f] += low[0][nt][f] + low[1][nt][f];
         }
     }
     if (!owns) return;
 #pragma unroll
-    for (int nt = 0; nt < 4; ++nt)
+    for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
         for (int f = 0; f < 4; ++f) {
-            int d = warp * 16 + g + (f >> 1) * 8, v = v0 + nt * 8 + 2 * t4 + (f & 1);
+            int d = d0 + g + (f >> 1) * 8, v = v0 + c0 + nt * 8 + 2 * t4 + (f & 1);
             if (v < V) S[(size_t)v * D + d] = s[nt][f];
         }
 }
 
 }  // namespace chunk
 
-// One block per token: the factor of the norm over all heads, then weight and gate.
-template <typename T>
+// One block per token: the factor of the norm over all heads, then weight and gate. VEC: elements a thread takes together (a
+// property of the model, so a token's sum has one order in every step).
+template <typename T, int VEC>
 __global__ void __launch_bounds__(THREADS)
 decay_finish_kernel(const float* __restrict__ o, const T* __restrict__ gate, int ld, const float* __restrict__ weight, float eps,
                     T* __restrict__ mixed, int mixed_ld, int values) {
@@ -284,7 +306,14 @@ decay_finish_kernel(const float* __restrict__ o, const T* __restrict__ gate, int
     size_t t = blockIdx.x;
     const float* row = o + t * values;
     float sq = 0.f;
-    for (int d = threadIdx.x; d < values; d += THREADS) sq = fmaf(row[d], row[d], sq);
+#pragma unroll 4
+    for (int d = threadIdx.x * VEC; d < values; d += THREADS * VEC) {
+        float x[VEC];
+        if constexpr (VEC == 4) *reinterpret_cast<float4*>(x) = *reinterpret_cast<const float4*>(row + d);
+        else x[0] = row[d];
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) sq = fmaf(x[i], x[i], sq);
+    }
     sq = warp_sum(sq);
     if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = sq;
     __syncthreads();
@@ -292,9 +321,29 @@ decay_finish_kernel(const float* __restrict__ o, const T* __restrict__ gate, int
 #pragma unroll
     for (int w = 0; w < THREADS / 32; ++w) total += scratch[w];
     float factor = 1.0f / sqrtf(total / (float)values + eps);
-    for (int d = threadIdx.x; d < values; d += THREADS) {
-        float g = to_float(gate[t * ld + d]);
-        mixed[t * mixed_ld + d] = from_float<T>(row[d] * factor * weight[d] / (1.0f + expf(-g)));
+#pragma unroll 4
+    for (int d = threadIdx.x * VEC; d < values; d += THREADS * VEC) {
+        float x[VEC], g[VEC], w[VEC];
+        if constexpr (VEC == 4) {
+            *reinterpret_cast<float4*>(x) = *reinterpret_cast<const float4*>(row + d);
+            *reinterpret_cast<float4*>(w) = *reinterpret_cast<const float4*>(weight + d);
+            if constexpr (sizeof(T) == 2) {
+                T raw[4];
+                *reinterpret_cast<uint2*>(raw) = *reinterpret_cast<const uint2*>(gate + t * ld + d);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) g[i] = to_float(raw[i]);
+            } else {
+                *reinterpret_cast<float4*>(g) = *reinterpret_cast<const float4*>(gate + t * ld + d);
+            }
+        } else {
+            x[0] = row[d]; w[0] = weight[d]; g[0] = to_float(gate[t * ld + d]);
+        }
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) x[i] = x[i] * factor * w[i] / (1.0f + expf(-g[i]));
+        T* to = mixed + t * mixed_ld + d;
+        if constexpr (VEC == 4 && sizeof(T) == 2) *reinterpret_cast<uint2*>(to) = make_uint2(pack_bf16(x[0], x[1]), pack_bf16(x[2], x[3]));
+        else if constexpr (VEC == 4) *reinterpret_cast<float4*>(to) = make_float4(x[0], x[1], x[2], x[3]);
+        else to[0] = from_float<T>(x[0]);
     }
 }
 
@@ -414,10 +463,10 @@ LLMB_EXPORT int llmb_decay_recurrence(const void* proj, int ld, int dtype, const
             static bool configured = false;                                                                               \
             if (!configured) {                                                                                            \
                 LLMB_CUDA(cudaFuncSetAttribute(chunk::decay_chunk_kernel<DD>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
-                                               (int)chunk::smem_bytes<DD>()));                                            \
+                                               (int)chunk::Place<DD>::bytes));                                            \
                 configured = true;                                                                                        \
             }                                                                                                             \
-            LLMB_CUDA(llmb::launch(chunk::decay_chunk_kernel<DD>, grid, dim3(chunk::WARPS * 32), chunk::smem_bytes<DD>(), stream, true, \
+            LLMB_CUDA(llmb::launch(chunk::decay_chunk_kernel<DD>, grid, dim3(chunk::WARPS * 32), chunk::Place<DD>::bytes, stream, true, \
                                    (const B*)work, 2 * work_ld, state, state_stride, cu_seqlens, slot_ids, decays, o, H, V)); \
         } while (0)
         if (D == 32) LLMB_CHUNK(32);
@@ -461,13 +510,15 @@ LLMB_EXPORT int llmb_decay_recurrence(const void* proj, int ld, int dtype, const
 #undef LLMB_SCAN
 #undef LLMB_SCAN_AS
     }
-    int gate_at = 2 * keys + values;
-    if (dtype == LLMB_DTYPE_F32)
-        LLMB_CUDA(llmb::launch(decay_finish_kernel<float>, dim3(n_tokens), dim3(THREADS), 0, stream, true, (const float*)o,
-                               (const float*)proj + gate_at, ld, weight, eps, (float*)mixed, mixed_ld, values));
-    else
-        LLMB_CUDA(llmb::launch(decay_finish_kernel<B>, dim3(n_tokens), dim3(THREADS), 0, stream, true, (const float*)o,
-                               (const B*)proj + gate_at, ld, weight, eps, (B*)mixed, mixed_ld, values));
+    const char* gate = (const char*)proj + (size_t)(2 * keys + values) * esize;
+    bool wide_rows = values % 4 == 0 && ld % 4 == 0 && mixed_ld % 4 == 0 && ((size_t)gate % (4 * esize)) == 0 &&
+                     ((size_t)mixed % (4 * esize)) == 0 && (((size_t)o | (size_t)weight) % 16) == 0;
+#define LLMB_FINISH(T, VEC)                                                                                               \
+    LLMB_CUDA(llmb::launch(decay_finish_kernel<T, VEC>, dim3(n_tokens), dim3(THREADS), 0, stream, true, (const float*)o,  \
+                           (const T*)gate, ld, weight, eps, (T*)mixed, mixed_ld, values))
+    if (dtype == LLMB_DTYPE_F32) { if (wide_rows) LLMB_FINISH(float, 4); else LLMB_FINISH(float, 1); }
+    else { if (wide_rows) LLMB_FINISH(B, 4); else LLMB_FINISH(B, 1); }
+#undef LLMB_FINISH
     return check_launch("decay_recurrence");
 }
 LLMB_PACKED(llmb_decay_recurrence)
